@@ -8,7 +8,8 @@
 // per query head where `head_scale` is given; with `softcap` c > 0 a score s
 // becomes c * tanh(s / c).  With `keep_first` n > 0 the keys at positions
 // below n stay visible behind a window (le::key_visible): their tiles are
-// visited before the window's.
+// visited before the window's.  With `sink` (one number per query head) the
+// softmax's denominator has one more term exp(sink[head]).
 //
 // One block per (tile of 16 query tokens of one request, query head).  Keys
 // are visited in tiles of 32 from position 0 (or the window's start) with a
@@ -50,7 +51,7 @@ attention_generic_kernel(T *__restrict__ out, int64_t out_stride, const T *__res
                          const int32_t *__restrict__ ctx_before, const int32_t *__restrict__ tile_request,
                          const int32_t *__restrict__ tile_q0, int num_heads, int num_kv_heads, int page_size,
                          int num_pages, int reach, float scale, const float *__restrict__ head_scale,
-                         int keep_first, float softcap, int *__restrict__ status) {
+                         int keep_first, float softcap, const float *__restrict__ sink, int *__restrict__ status) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   GenericSmem &sm = *reinterpret_cast<GenericSmem *>(smem_raw);
 
@@ -156,7 +157,12 @@ attention_generic_kernel(T *__restrict__ out, int64_t out_stride, const T *__res
   }
 
   if (row < rows) {
-    const float inv = l_run > 0.0f ? 1.0f / l_run : 0.0f;
+    float inv = l_run > 0.0f ? 1.0f / l_run : 0.0f;
+    if (sink) {                                  // one more term in the denominator
+      const float top = fmaxf(m_run, sink[head]);
+      const float a = expf(m_run - top);
+      inv = a / fmaf(l_run, a, expf(sink[head] - top));
+    }
     T *o = out + (tok0 + row) * out_stride + head * HD;
 #pragma unroll
     for (int j = 0; j < HD / 8; ++j) o[sub + 8 * j] = le::from_f32<T>(acc[j] * inv);
@@ -174,13 +180,13 @@ LE_API const char *le_last_error() { return le::error_buffer(); }
 // q_stride holding num_heads * HD query values; caches [pages, kv_heads,
 // page, HD].  tile_request / tile_q0 list the tiles of 16 query tokens.
 // `reach`: see le::first_visible_key; `head_scale`: num_heads floats or null; `keep_first`: see le::key_visible;
-// `softcap`: 0 for none.
+// `softcap`: 0 for none; `sink`: num_heads floats or null.
 LE_API int le_attention_generic(void *out, int64_t out_stride, const void *q, int64_t q_stride, const void *k_cache,
                                 const void *v_cache, int dtype, const int32_t *block_table, int max_blocks,
                                 const int32_t *cu_q, const int32_t *ctx_before, const int32_t *tile_request,
                                 const int32_t *tile_q0, int num_tiles, int num_heads, int num_kv_heads, int page_size,
                                 int num_pages, int reach, float scale, const float *head_scale, int keep_first,
-                                float softcap, int *status, cudaStream_t stream) {
+                                float softcap, const float *sink, int *status, cudaStream_t stream) {
   if (num_tiles <= 0) return 0;
   if (num_kv_heads <= 0 || num_heads % num_kv_heads) return le::invalid("le_attention_generic: %d heads do not divide into %d groups", num_heads, num_kv_heads);
   if (num_heads > 65535) return le::invalid("le_attention_generic: too many heads for one launch");
@@ -197,7 +203,7 @@ LE_API int le_attention_generic(void *out, int64_t out_stride, const void *q, in
                                             static_cast<const T *>(k_cache), static_cast<const T *>(v_cache),          \
                                             block_table, max_blocks, cu_q, ctx_before, tile_request, tile_q0,          \
                                             num_heads, num_kv_heads, page_size, num_pages, reach, scale, head_scale,   \
-                                            keep_first, softcap, status);                                                                \
+                                            keep_first, softcap, sink, status);                                        \
   } while (0)
   if (dtype == LE_F32) LE_GO(float);
   else if (dtype == LE_BF16) LE_GO(__nv_bfloat16);

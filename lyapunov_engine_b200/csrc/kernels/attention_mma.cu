@@ -15,6 +15,8 @@
 // flight, so any page size works and a page's rows need not be adjacent.
 // One formula for every cut: the query at absolute position p sees keys
 // le::first_visible_key(p, reach) .. p of its own request (all keys, a window, or its own chunk).
+// With `sink` (one number per query head) the softmax's denominator has one more term exp(sink[head]); it enters where
+// the last division is made (le::sink_inverse), after every split and warp has been added up.
 //
 // Reference: flash_attn_v2.cu:13-212 (contiguous keys, scalar dot products,
 // top-left mask), flash_decoding.cu:13-147 (contiguous keys, every thread
@@ -236,7 +238,7 @@ attention_prefill_kernel(bf16 *__restrict__ out, int64_t out_stride, const bf16 
                          const int32_t *__restrict__ ctx_before, const int32_t *__restrict__ tile_request,
                          const int32_t *__restrict__ tile_q0, int num_heads, int num_kv_heads, int page_size,
                          int page_shift, int num_pages, int reach, float scale, const float *__restrict__ head_scale,
-                         int keep_first, float softcap, int *__restrict__ status) {
+                         int keep_first, float softcap, const float *__restrict__ sink, int *__restrict__ status) {
   extern __shared__ __align__(128) unsigned char smem_raw[];
   bf16 *q_tile = reinterpret_cast<bf16 *>(smem_raw);
   bf16 *k_tiles = q_tile + PF_BM * HD;
@@ -400,7 +402,12 @@ attention_prefill_kernel(bf16 *__restrict__ out, int64_t out_stride, const bf16 
     l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 1);
     l_run[r] += __shfl_xor_sync(0xffffffffu, l_run[r], 2);
   }
-  const float inv[2] = {l_run[0] > 0.0f ? 1.0f / l_run[0] : 0.0f, l_run[1] > 0.0f ? 1.0f / l_run[1] : 0.0f};
+  float inv[2] = {l_run[0] > 0.0f ? 1.0f / l_run[0] : 0.0f, l_run[1] > 0.0f ? 1.0f / l_run[1] : 0.0f};
+  if (sink) {
+    const float sink2 = sink[head] * LOG2E;
+#pragma unroll
+    for (int r = 0; r < 2; ++r) inv[r] = le::sink_inverse(l_run[r], m_run[r] * sl2, sink2);
+  }
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
     if ((r ? row_hi : row_lo) >= rows) continue;
@@ -438,7 +445,8 @@ attention_decode_kernel(bf16 *__restrict__ out, int64_t out_stride, float *__res
                         const int32_t *__restrict__ cu_q, const int32_t *__restrict__ ctx_before,
                         const int32_t *__restrict__ requests, int num_heads, int num_kv_heads, int page_size,
                         int page_shift, int num_pages, int reach, float scale, const float *__restrict__ head_scale,
-                        int keep_first, float softcap, int num_splits, int cluster_merge, int *__restrict__ status) {
+                        int keep_first, float softcap, const float *__restrict__ sink, int num_splits, int cluster_merge,
+                        int *__restrict__ status) {
   extern __shared__ __align__(128) unsigned char smem_raw[];
   // (the kernel before this one wrote the queries and the newest key and value of every request; what is
   // read before wait_for_predecessor() below is older than that: the step's integers and keys of earlier steps)
@@ -680,7 +688,8 @@ attention_decode_kernel(bf16 *__restrict__ out, int64_t out_stride, float *__res
     }
     const int head = h0 + row;
     if (num_splits == 1) {
-      out[tok * out_stride + head * HD + d] = __float2bfloat16_rn(l > 0.0f ? acc / l : 0.0f);
+      const float y = sink ? acc * le::sink_inverse(l, m * sl2, sink[head] * LOG2E) : (l > 0.0f ? acc / l : 0.0f);
+      out[tok * out_stride + head * HD + d] = __float2bfloat16_rn(y);
     } else if (cluster_merge) {
       cl_o[row * HD + d] = acc;
       if (d == 0) {
@@ -723,7 +732,8 @@ attention_decode_kernel(bf16 *__restrict__ out, int64_t out_stride, float *__res
         acc += f * os[s2];
         l += f * ls[s2];
       }
-      out[tok * out_stride + (h0 + row) * HD + d] = __float2bfloat16_rn(l > 0.0f ? acc / l : 0.0f);
+      const float y = sink ? acc * le::sink_inverse(l, m, sink[h0 + row] * LOG2E) : (l > 0.0f ? acc / l : 0.0f);
+      out[tok * out_stride + (h0 + row) * HD + d] = __float2bfloat16_rn(y);
     }
     le::cluster_sync();                       // nobody leaves while another still reads its shared memory
   }
@@ -735,7 +745,8 @@ attention_decode_kernel(bf16 *__restrict__ out, int64_t out_stride, float *__res
 constexpr int MERGE_MAX_SPLITS = 1024;
 __global__ void attention_merge_kernel(bf16 *__restrict__ out, int64_t out_stride, const float *__restrict__ part_o,
                                        const float *__restrict__ part_ml, const int32_t *__restrict__ cu_q,
-                                       const int32_t *__restrict__ requests, int num_heads, int num_splits) {
+                                       const int32_t *__restrict__ requests, int num_heads, int num_splits,
+                                       const float *__restrict__ sink) {
   extern __shared__ float merge_weight[];          // [num_splits], then the reciprocal of the sum
   le::let_successor_start();
   le::wait_for_predecessor();
@@ -759,7 +770,8 @@ __global__ void attention_merge_kernel(bf16 *__restrict__ out, int64_t out_strid
     }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
-    if (lane == 0) merge_weight[num_splits] = l > 0.0f ? 1.0f / l : 0.0f;
+    if (lane == 0)
+      merge_weight[num_splits] = sink ? le::sink_inverse(l, m, sink[head] * LOG2E) : (l > 0.0f ? 1.0f / l : 0.0f);
   }
   __syncthreads();
   const float inv_l = merge_weight[num_splits];
@@ -801,7 +813,7 @@ LE_API int le_attention_prefill_bf16(void *out, int64_t out_stride, const void *
                                      const int32_t *ctx_before, const int32_t *tile_request, const int32_t *tile_q0,
                                      int num_tiles, int num_heads, int num_kv_heads, int page_size, int num_pages,
                                      int reach, float scale, const float *head_scale, int keep_first, float softcap,
-                                     int *status, cudaStream_t stream) {
+                                     const float *sink, int *status, cudaStream_t stream) {
   if (num_tiles <= 0) return 0;
   if (num_kv_heads <= 0 || num_heads % num_kv_heads) return le::invalid("le_attention_prefill_bf16: %d heads do not divide into %d groups", num_heads, num_kv_heads);
   if (num_heads > 65535) return le::invalid("le_attention_prefill_bf16: too many heads for one launch");
@@ -815,7 +827,8 @@ LE_API int le_attention_prefill_bf16(void *out, int64_t out_stride, const void *
   attention_prefill_kernel<<<grid, PF_THREADS, smem, stream>>>(
       static_cast<bf16 *>(out), out_stride, static_cast<const bf16 *>(q), q_stride, static_cast<const bf16 *>(k_cache),
       static_cast<const bf16 *>(v_cache), block_table, max_blocks, cu_q, ctx_before, tile_request, tile_q0, num_heads,
-      num_kv_heads, page_size, page_shift_of(page_size), num_pages, reach, scale, head_scale, keep_first, softcap, status);
+      num_kv_heads, page_size, page_shift_of(page_size), num_pages, reach, scale, head_scale, keep_first, softcap, sink,
+      status);
   return le::launched();
 }
 
@@ -917,7 +930,7 @@ struct DecodeForm {
                     const void *k_cache, const void *v_cache, const int32_t *block_table, int max_blocks, const int32_t *cu_q,
                     const int32_t *ctx_before, const int32_t *requests, int num_requests, int num_heads, int num_kv_heads,
                     int page_size, int num_pages, int reach, float scale, const float *head_scale, int keep_first, float softcap,
-                    int num_splits, int *status) {
+                    const float *sink, int num_splits, int *status) {
     if (!ready()) return le::invalid("le_attention_decode_bf16: cannot get %zu bytes of shared memory", smem());
     if (cluster_fits(num_splits)) {
       // the splits of a (request, kv head) as one cluster: merged through shared memory, no scratch, no second kernel
@@ -927,7 +940,7 @@ struct DecodeForm {
                                         static_cast<const bf16 *>(k_cache), static_cast<const bf16 *>(v_cache), block_table,
                                         max_blocks, cu_q, ctx_before, requests, num_heads, num_kv_heads, page_size,
                                         page_shift_of(page_size), num_pages, reach, scale, head_scale, keep_first, softcap,
-                                        num_splits, 1, status);
+                                        sink, num_splits, 1, status);
     }
     if (num_splits > 1 && scratch == nullptr) return le::invalid("le_attention_decode_bf16: splitting the keys %d ways needs scratch memory", num_splits);
     if (reinterpret_cast<uintptr_t>(scratch) % 8) return le::invalid("le_attention_decode_bf16: the scratch memory must start on an 8-byte boundary");
@@ -937,13 +950,13 @@ struct DecodeForm {
                                 part_o, part_ml, static_cast<const bf16 *>(q), q_stride, static_cast<const bf16 *>(k_cache),
                                 static_cast<const bf16 *>(v_cache), block_table, max_blocks, cu_q, ctx_before, requests, num_heads,
                                 num_kv_heads, page_size, page_shift_of(page_size), num_pages, reach, scale, head_scale, keep_first,
-                                softcap, num_splits, 0, status);
+                                softcap, sink, num_splits, 0, status);
     if (rc != 0 || num_splits == 1) return rc;
     dim3 mgrid(num_heads, num_requests);
     return le::launch_chained(attention_merge_kernel, mgrid, dim3(HD < 32 ? 32 : (HD > 128 ? 128 : HD)),
                               (static_cast<size_t>(num_splits) + 1) * sizeof(float), stream,
                               static_cast<bf16 *>(out), out_stride, static_cast<const float *>(part_o),
-                              static_cast<const float *>(part_ml), cu_q, requests, num_heads, num_splits);
+                              static_cast<const float *>(part_ml), cu_q, requests, num_heads, num_splits, sink);
   }
 };
 
@@ -973,7 +986,8 @@ LE_API int le_attention_decode_resident_blocks(int num_splits, int small) {
 // le_attention_decode_scratch_floats(...) floats; it is used when the keys are
 // cut into more splits than a thread-block cluster merges by itself.
 // `reach`: see le::first_visible_key; `head_scale`: one more factor per query head on its scores, or null;
-// `keep_first`: see le::key_visible; `softcap` c > 0: a score s becomes c * tanh(s / c).
+// `keep_first`: see le::key_visible; `softcap` c > 0: a score s becomes c * tanh(s / c); `sink`: one number per query
+// head, or null.
 // `form`: 0 lets the number of blocks decide between the usual form of the kernel and the one with 16-key tiles
 // (see small_form); 1 asks for the usual form, 2 for the small one where the head size has it (a caller that pads
 // the step with dummy requests knows how many of the blocks are real; the grid does not show it).
@@ -982,7 +996,7 @@ LE_API int le_attention_decode_bf16_form(void *out, int64_t out_stride, float *s
                                          const int32_t *cu_q, const int32_t *ctx_before, const int32_t *requests,
                                          int num_requests, int num_heads, int num_kv_heads, int page_size, int num_pages,
                                          int reach, float scale, const float *head_scale, int keep_first, float softcap,
-                                         int num_splits, int form, int *status, cudaStream_t stream) {
+                                         const float *sink, int num_splits, int form, int *status, cudaStream_t stream) {
   if (num_requests <= 0) return 0;
   if (num_kv_heads <= 0 || num_heads % num_kv_heads) return le::invalid("le_attention_decode_bf16: %d heads do not divide into %d groups", num_heads, num_kv_heads);
   if (num_splits < 1 || num_splits > MERGE_MAX_SPLITS) return le::invalid("le_attention_decode_bf16: %d splits (1..%d)", num_splits, MERGE_MAX_SPLITS);
@@ -995,10 +1009,11 @@ LE_API int le_attention_decode_bf16_form(void *out, int64_t out_stride, float *s
   if (small)
     return DecodeForm<16>::launch(grid, stream, out, out_stride, scratch, q, q_stride, k_cache, v_cache, block_table, max_blocks, cu_q,
                                   ctx_before, requests, num_requests, num_heads, num_kv_heads, page_size, num_pages, reach, scale,
-                                  head_scale, keep_first, softcap, num_splits, status);
+                                  head_scale, keep_first, softcap, sink, num_splits, status);
   return DecodeForm<DC_TILE_DEFAULT>::launch(grid, stream, out, out_stride, scratch, q, q_stride, k_cache, v_cache, block_table,
                                              max_blocks, cu_q, ctx_before, requests, num_requests, num_heads, num_kv_heads, page_size,
-                                             num_pages, reach, scale, head_scale, keep_first, softcap, num_splits, status);
+                                             num_pages, reach, scale, head_scale, keep_first, softcap, sink, num_splits,
+                                             status);
 }
 
 LE_API int le_attention_decode_bf16(void *out, int64_t out_stride, float *scratch, const void *q, int64_t q_stride,
@@ -1008,7 +1023,7 @@ LE_API int le_attention_decode_bf16(void *out, int64_t out_stride, float *scratc
                                     int window, float scale, int num_splits, int *status, cudaStream_t stream) {
   return le_attention_decode_bf16_form(out, out_stride, scratch, q, q_stride, k_cache, v_cache, block_table, max_blocks, cu_q,
                                        ctx_before, requests, num_requests, num_heads, num_kv_heads, page_size, num_pages, window,
-                                       scale, nullptr, 0, 0.0f, num_splits, 0, status, stream);
+                                       scale, nullptr, 0, 0.0f, nullptr, num_splits, 0, status, stream);
 }
 
 // ---------------------------------------------------------------- no allocation

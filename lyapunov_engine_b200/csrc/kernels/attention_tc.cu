@@ -35,7 +35,8 @@
 // The running maximum only moves when the tile's maximum exceeds it by more
 // than 2^8 in the exponent; until then probabilities up to 256 go into the
 // product and the sum (both 32-bit accumulations), which the final division
-// takes out again.  The accumulator in tensor memory is therefore rescaled
+// takes out again (a sink, one more term exp(sink[head]) of the denominator,
+// enters there).  The accumulator in tensor memory is therefore rescaled
 // rarely.  At the end every thread normalises its row and stores it.
 //
 // Every wait on an mbarrier is bounded in time; a block that gives up sets the
@@ -93,7 +94,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                     const int32_t *__restrict__ block_table, int max_blocks, const int32_t *__restrict__ cu_q,
                     const int32_t *__restrict__ ctx_before, const int32_t *__restrict__ tile_request,
                     const int32_t *__restrict__ tile_q0, int num_heads, int num_kv_heads, int page_size, int page_shift,
-                    int num_pages, int reach, float scale, const float *__restrict__ head_scale, int *__restrict__ status) {
+                    int num_pages, int reach, float scale, const float *__restrict__ head_scale,
+                    const float *__restrict__ sink, int *__restrict__ status) {
   extern __shared__ unsigned char smem_unaligned[];
   unsigned char *smem = reinterpret_cast<unsigned char *>((reinterpret_cast<uintptr_t>(smem_unaligned) + 1023) & ~uintptr_t(1023));
   unsigned char *q_smem = smem;                // [2 heads]
@@ -401,7 +403,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
       if (lane == 0) { *failed = 1; atomicOr(status, LE_STATUS_WAIT_TIMEOUT); }
     } else {
       tc_fence_after();
-      const float inv = l_run > 0.0f ? 1.0f / l_run : 0.0f;
+      float inv = l_run > 0.0f ? 1.0f / l_run : 0.0f;
+      if (sink) inv = le::sink_inverse(l_run, m_run, sink[head0 + g] * LOG2E);
       bf16 *dst = out + (tok0 + r) * out_stride + (head0 + g) * HD;
 #pragma unroll
       for (int c = 0; c < HD / 32; ++c) {
@@ -450,7 +453,8 @@ LE_API int le_attention_prefill_tc_bf16(void *out, int64_t out_stride, const voi
                                         int q_width, const void *k_cache, const void *v_cache, const int32_t *block_table,
                                         int max_blocks, const int32_t *cu_q, const int32_t *ctx_before,
                                         const int32_t *tile_request, const int32_t *tile_q0, int num_tiles, int num_heads,
-                                        int num_kv_heads, int page_size, int num_pages, int reach, float scale, const float *head_scale, int *status,
+                                        int num_kv_heads, int page_size, int num_pages, int reach, float scale, const float *head_scale,
+                                        const float *sink, int *status,
                                         cudaStream_t stream) {
   if (num_tiles <= 0) return 0;
   if (!le_attention_tc_available(page_size)) return le::invalid("le_attention_prefill_tc_bf16: pages of %d keys are not supported (8..128, a power of two)", page_size);
@@ -474,7 +478,7 @@ LE_API int le_attention_prefill_tc_bf16(void *out, int64_t out_stride, const voi
   dim3 grid(num_kv_heads * ((group + 1) / 2), num_tiles);   // two heads of a group per block
   return le::launch_chained(attention_tc_kernel, grid, dim3(THREADS), smem, stream, map_q, map_k, map_v, static_cast<bf16 *>(out),
                             out_stride, block_table, max_blocks, cu_q, ctx_before, tile_request, tile_q0, num_heads,
-                            num_kv_heads, page_size, tc_page_shift_of(page_size), num_pages, reach, scale, head_scale, status);
+                            num_kv_heads, page_size, tc_page_shift_of(page_size), num_pages, reach, scale, head_scale, sink, status);
 }
 
 #else

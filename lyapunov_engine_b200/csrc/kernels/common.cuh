@@ -199,6 +199,16 @@ __device__ __forceinline__ float exp_unbiased(float x) {
   return e * __int_as_float((static_cast<int>(k) + 127) << 23);
 }
 
+// A softmax whose denominator has one more term, 2^sink, that belongs to no key (a learned number per head times
+// log2 e).  `l` is the sum of 2^(s - m) over the keys and the weighted sum of values is in the same units: returns the
+// factor that makes it the output, 1 / (l + 2^(sink - m)), without overflow on either side.
+__device__ __forceinline__ float sink_inverse(float l, float m, float sink) {
+  const float top = fmaxf(m, sink);
+  if (top == -INFINITY) return 0.0f;
+  const float a = exp2f(m - top);
+  return a / fmaf(l, a, exp2f(sink - top));
+}
+
 // cap * tanh(x) with x = score / cap already: capped attention scores for the bfloat16 kernels.  tanh(x) = 1 -
 // 2 / (2^(2 x log2 e) + 1) with ex2.approx and a fast division: absolute error about 1e-7 over the whole range
 // (the exponential overflows to +inf, which gives 1, and underflows to 0, which gives -1).
@@ -221,6 +231,16 @@ struct GatedActivation {
   const float *bias = nullptr;
   int inter = 0;
 };
+// An activation of a product that has no gate beside it, applied by the ungated forms of the product kernels to their
+// 32-bit sums.  kind 3: max(v, 0)^2; every other kind leaves the product as it is.
+constexpr int ACT_RELU_SQUARED = 3;
+__device__ __forceinline__ float ungated_activation(float v, const GatedActivation &a) {
+  if (a.kind == ACT_RELU_SQUARED) {
+    const float r = fmaxf(v, 0.0f);
+    return r * r;
+  }
+  return v;
+}
 __device__ __forceinline__ void gated_bias(float &g, float &u, int n, const GatedActivation &a) {
   if (a.bias != nullptr) g += a.bias[n], u += a.bias[a.inter + n];
 }

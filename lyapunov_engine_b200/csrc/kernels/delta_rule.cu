@@ -349,6 +349,65 @@ head_norm_gate_kernel(T *__restrict__ out, int64_t out_stride, const float *__re
 
 namespace {
 
+// The same for few wide heads: a block per (token, head), four values a thread at a time, kept in registers between
+// the sum of squares and the result (V groups of 1024 values; everything on 16-byte addresses for floats, 8 for bfloat16).
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+head_norm_gate_wide_kernel(T *__restrict__ out, int64_t out_stride, const float *__restrict__ o, int64_t o_stride,
+                           const T *__restrict__ gate, int64_t gate_stride, const float *__restrict__ weight, float eps,
+                           int heads, int vdim, int weight_per_head, int gate_kind, float out_scale) {
+  __shared__ float scratch[33];
+  le::let_successor_start();
+  le::wait_for_predecessor();
+  const int64_t t = blockIdx.x / heads;
+  const int h = static_cast<int>(blockIdx.x - t * heads);
+  const float *x = o + t * o_stride + static_cast<int64_t>(h) * vdim;
+  const T *gr = gate + t * gate_stride + static_cast<int64_t>(h) * vdim;
+  T *dst = out + t * out_stride + static_cast<int64_t>(h) * vdim;
+  if (weight_per_head) weight += static_cast<int64_t>(h) * vdim;
+  float4 xv[V];
+  float g[V][4];
+  float ss = 0.0f;
+#pragma unroll
+  for (int v = 0; v < V; ++v) {
+    const int i = (threadIdx.x + v * 256) * 4;
+    xv[v] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    if (i < vdim) {
+      xv[v] = *reinterpret_cast<const float4 *>(x + i);
+      if constexpr (sizeof(T) == 2) {
+        const uint2 r = *reinterpret_cast<const uint2 *>(gr + i);
+        g[v][0] = __uint_as_float(r.x << 16), g[v][1] = __uint_as_float(r.x & 0xffff0000u);
+        g[v][2] = __uint_as_float(r.y << 16), g[v][3] = __uint_as_float(r.y & 0xffff0000u);
+      } else {
+        const float4 r = *reinterpret_cast<const float4 *>(gr + i);
+        g[v][0] = r.x, g[v][1] = r.y, g[v][2] = r.z, g[v][3] = r.w;
+      }
+    }
+    ss = fmaf(xv[v].x, xv[v].x, fmaf(xv[v].y, xv[v].y, fmaf(xv[v].z, xv[v].z, fmaf(xv[v].w, xv[v].w, ss))));
+  }
+  const float inv = rsqrtf(le::block_sum(ss, scratch) / static_cast<float>(vdim) + eps) * out_scale;
+#pragma unroll
+  for (int v = 0; v < V; ++v) {
+    const int i = (threadIdx.x + v * 256) * 4;
+    if (i >= vdim) continue;
+    const float4 w = *reinterpret_cast<const float4 *>(weight + i);
+    float y[4] = {xv[v].x * inv * w.x, xv[v].y * inv * w.y, xv[v].z * inv * w.z, xv[v].w * inv * w.w};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float s = 1.0f / (1.0f + expf(-g[v][e]));
+      y[e] *= gate_kind == 0 ? g[v][e] * s : s;
+    }
+    if constexpr (sizeof(T) == 2) {
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(y[0], y[1]), hi = __floats2bfloat162_rn(y[2], y[3]);
+      uint2 r;
+      r.x = *reinterpret_cast<const uint32_t *>(&lo), r.y = *reinterpret_cast<const uint32_t *>(&hi);
+      *reinterpret_cast<uint2 *>(dst + i) = r;
+    } else {
+      *reinterpret_cast<float4 *>(dst + i) = make_float4(y[0], y[1], y[2], y[3]);
+    }
+  }
+}
+
 // How a column of the state is shared out for heads of `dim` entries: `rows` entries a thread, `lanes` threads a
 // column (a power of two, rows * lanes >= dim); false: dim is too large.  Heads of 128 to 256 entries may be held 8 or
 // 16 rows a thread (LYAPUNOV_DELTA_ROWS=8|16; the default is the one measured faster).
@@ -441,6 +500,21 @@ LE_API int le_head_norm_gate(void *out, int64_t out_stride, const float *o, int6
                              int vdim, int weight_per_head, int gate_kind, float out_scale, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
   const int64_t items = static_cast<int64_t>(num_tokens) * heads;
+  const auto on16 = [](const void *p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+  if (vdim >= 512 && vdim <= 8192 && vdim % 4 == 0 && out_stride % 4 == 0 && o_stride % 4 == 0 && gate_stride % 4 == 0 &&
+      on16(o) && on16(weight) && (reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(out)) % (dtype == LE_BF16 ? 8 : 16) == 0) {
+#define LE_WIDE(V)                                                                                                        \
+  LE_DISPATCH_DTYPE(dtype, T,                                                                                             \
+                    return le::launch_chained(head_norm_gate_wide_kernel<T, V>, dim3(static_cast<unsigned>(items)),       \
+                                              dim3(256), 0, stream, static_cast<T *>(out), out_stride, o, o_stride,       \
+                                              static_cast<const T *>(gate), gate_stride, weight, eps, heads, vdim,        \
+                                              weight_per_head, gate_kind, out_scale))
+    if (vdim <= 1024) LE_WIDE(1);
+    if (vdim <= 2048) LE_WIDE(2);
+    if (vdim <= 4096) LE_WIDE(4);
+    LE_WIDE(8);
+#undef LE_WIDE
+  }
   const dim3 grid(static_cast<unsigned>((items + 3) / 4));
   LE_DISPATCH_DTYPE(dtype, T,
                     return le::launch_chained(head_norm_gate_kernel<T>, grid, dim3(128), 0, stream, static_cast<T *>(out),

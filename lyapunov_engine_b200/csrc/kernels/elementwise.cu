@@ -126,6 +126,37 @@ __global__ void sigmoid_gate_kernel(T *__restrict__ out, int64_t out_stride, con
   }
 }
 
+// out[t, i] = act(x[t, i]) (kind 0: silu, le::ACT_RELU_SQUARED: max(x, 0)^2); 32-bit, rounded once.
+template <typename T>
+__device__ __forceinline__ T activated(T x, int kind) {
+  const float v = le::to_f32(x);
+  if (kind == le::ACT_RELU_SQUARED) {
+    const float r = fmaxf(v, 0.0f);
+    return le::from_f32<T>(r * r);
+  }
+  return le::from_f32<T>(v / (1.0f + expf(-v)));
+}
+template <typename T, int VEC>
+__global__ void activate_kernel(T *__restrict__ out, int64_t out_stride, const T *__restrict__ x, int64_t x_stride,
+                                int num_tokens, int width, int kind) {
+  le::let_successor_start();
+  le::wait_for_predecessor();
+  const int per_row = width / VEC;
+  const int64_t idx = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x;
+  if (idx >= static_cast<int64_t>(num_tokens) * per_row) return;
+  const int64_t t = idx / per_row;
+  const int i = static_cast<int>(idx - t * per_row) * VEC;
+  if constexpr (VEC == 1) {
+    out[t * out_stride + i] = activated<T>(x[t * x_stride + i], kind);
+  } else {
+    uint4 raw = *reinterpret_cast<const uint4 *>(x + t * x_stride + i);
+    T *e = reinterpret_cast<T *>(&raw);
+#pragma unroll
+    for (int v = 0; v < VEC; ++v) e[v] = activated<T>(e[v], kind);
+    *reinterpret_cast<uint4 *>(out + t * out_stride + i) = raw;
+  }
+}
+
 // out[t, i] = silu(gu[t, i]) * gu[t, I + i], in 32-bit, rounded once.
 template <typename T>
 __global__ void swiglu_kernel(T *__restrict__ out, const T *__restrict__ gu, int64_t total, int inter) {
@@ -305,6 +336,26 @@ LE_API int le_sigmoid_gate(void *out, int64_t out_stride, const void *x, int64_t
   if (dtype == LE_F32) { if (wide) LE_GO(float, 4); LE_GO(float, 1); }
 #undef LE_GO
   return le::invalid("le_sigmoid_gate: unknown dtype code %d", dtype);
+}
+
+// out, x: [T, width] with row strides of their own (column ranges of wider rows are fine; out may be x).
+LE_API int le_activate(void *out, int64_t out_stride, const void *x, int64_t x_stride, int dtype, int num_tokens, int width,
+                       int kind, cudaStream_t stream) {
+  if (num_tokens <= 0 || width <= 0) return 0;
+  if (kind != 0 && kind != le::ACT_RELU_SQUARED) return le::invalid("le_activate: unknown activation %d", kind);
+  const int vec = dtype == LE_BF16 ? 8 : 4;
+  const bool wide = width % vec == 0 && out_stride % vec == 0 && x_stride % vec == 0 &&
+                    ((reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(x)) & 15) == 0;
+  const int64_t items = static_cast<int64_t>(num_tokens) * width / (wide ? vec : 1);
+  const int64_t blocks = (items + 255) / 256;
+  if (blocks > 2147483647LL) return le::invalid("le_activate: too many elements for one launch");
+#define LE_GO(T, V)                                                                                                   \
+  return le::launch_chained(activate_kernel<T, V>, dim3(static_cast<unsigned>(blocks)), dim3(256), 0, stream,         \
+                            static_cast<T *>(out), out_stride, static_cast<const T *>(x), x_stride, num_tokens, width, kind)
+  if (dtype == LE_BF16) { if (wide) LE_GO(__nv_bfloat16, 8); LE_GO(__nv_bfloat16, 1); }
+  if (dtype == LE_F32) { if (wide) LE_GO(float, 4); LE_GO(float, 1); }
+#undef LE_GO
+  return le::invalid("le_activate: unknown dtype code %d", dtype);
 }
 
 LE_API int le_swiglu(void *out, const void *gate_up, int dtype, int num_tokens, int inter, cudaStream_t stream) {

@@ -284,6 +284,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                 float up = __uint_as_float(u[j + i]);
                 if (col + i < n_limit) le::gated_bias(f[i], up, col + i, act);
                 f[i] = le::gated_activation<true>(f[i], up, act);
+              } else {
+                f[i] = le::ungated_activation(f[i], act);
               }
             }
             if (col + 8 <= n_limit && (reinterpret_cast<uintptr_t>(dst + col) & 15) == 0) {
@@ -410,7 +412,8 @@ int launch(void *out, const void *x, const void *w, int M, int N, int K, int64_t
 // gated = 0: out[M, N] (bfloat16 or float32) = x W^T.  gated = 1: W is
 // [N = 2 I, K] (gate rows, then up rows), out is bfloat16 [M, I] =
 // act(x Wg^T, x Wu^T) with the activation (act_kind, act_slope, act_limit) of
-// le::GatedActivation (0: silu(g) * u).  Needs K and the leading dimensions of x and W to
+// le::GatedActivation (0: silu(g) * u).  With gated = 0 act_kind
+// le::ACT_RELU_SQUARED puts that activation on the product.  Needs K and the leading dimensions of x and W to
 // be multiples of 8 and their base addresses 16-byte aligned (TMA).
 LE_API int le_gemm_tc_bias_bf16(void *out, int out_dtype, const void *x, const void *w, int M, int N, int K, int64_t ldx,
                                 int64_t ldw, int64_t ldo, int gated, int act_kind, float act_slope, float act_limit,
@@ -428,7 +431,7 @@ LE_API int le_gemm_tc_bias_bf16(void *out, int out_dtype, const void *x, const v
                                 int64_t ldw, int64_t ldo, int gated, int act_kind, float act_slope, float act_limit,
                                 const float *bias, int *status, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
-  if (act_kind < 0 || act_kind > 2) return le::invalid("le_gemm_tc_bf16: unknown activation %d", act_kind);
+  if (act_kind < 0 || act_kind > (gated ? 2 : le::ACT_RELU_SQUARED)) return le::invalid("le_gemm_tc_bf16: unknown activation %d", act_kind);
   const le::GatedActivation act{act_kind, act_slope, act_limit, gated ? bias : nullptr, N / 2};
   if (K <= 0 || K % 8 || ldx % 8 || ldw % 8) return le::invalid("le_gemm_tc_bf16: K (%d) and the leading dimensions must be multiples of 8", K);
   if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15) return le::invalid("le_gemm_tc_bf16: x and W must be 16-byte aligned");
@@ -451,14 +454,14 @@ LE_API int le_gemm_tc_bias_bf16(void *out, int out_dtype, const void *x, const v
   // of the SMs without a tile
   const int64_t tiles_m = (M + BM - 1) / BM;
   const bool wide = tiles_m * ((N + 255) / 256) >= 74;
-  if (pair && out_dtype == LE_BF16) return launch<256, false, bf16, true>(out, x, w, M, N, K, ldx, ldw, ldo, status, stream);
-  if (pair && out_dtype == LE_F32) return launch<256, false, float, true>(out, x, w, M, N, K, ldx, ldw, ldo, status, stream);
+  if (pair && out_dtype == LE_BF16) return launch<256, false, bf16, true>(out, x, w, M, N, K, ldx, ldw, ldo, status, stream, act);
+  if (pair && out_dtype == LE_F32) return launch<256, false, float, true>(out, x, w, M, N, K, ldx, ldw, ldo, status, stream, act);
   if (out_dtype == LE_BF16)
-    return wide ? launch<256, false, bf16>(out, x, w, M, N, K, ldx, ldw, ldo, status, stream)
-                : launch<128, false, bf16>(out, x, w, M, N, K, ldx, ldw, ldo, status, stream);
+    return wide ? launch<256, false, bf16>(out, x, w, M, N, K, ldx, ldw, ldo, status, stream, act)
+                : launch<128, false, bf16>(out, x, w, M, N, K, ldx, ldw, ldo, status, stream, act);
   if (out_dtype == LE_F32)
-    return wide ? launch<256, false, float>(out, x, w, M, N, K, ldx, ldw, ldo, status, stream)
-                : launch<128, false, float>(out, x, w, M, N, K, ldx, ldw, ldo, status, stream);
+    return wide ? launch<256, false, float>(out, x, w, M, N, K, ldx, ldw, ldo, status, stream, act)
+                : launch<128, false, float>(out, x, w, M, N, K, ldx, ldw, ldo, status, stream, act);
   return le::invalid("le_gemm_tc_bf16: unknown dtype code %d", out_dtype);
 }
 
@@ -470,7 +473,7 @@ LE_API int le_gemm_tc_grouped_bf16(void *out, int out_dtype, const void *x, cons
                                    const int32_t *tile_count, int gated, int act_kind, float act_slope, float act_limit,
                                    int *status, cudaStream_t stream) {
   if (M <= 0 || N <= 0 || experts <= 0) return 0;
-  if (act_kind < 0 || act_kind > 2) return le::invalid("le_gemm_tc_grouped_bf16: unknown activation %d", act_kind);
+  if (act_kind < 0 || act_kind > (gated ? 2 : le::ACT_RELU_SQUARED)) return le::invalid("le_gemm_tc_grouped_bf16: unknown activation %d", act_kind);
   const le::GatedActivation act{act_kind, act_slope, act_limit};
   if (M % BM) return le::invalid("le_gemm_tc_grouped_bf16: x holds whole tiles of %d rows, got %d rows", BM, M);
   if (K <= 0 || K % 8 || ldx % 8 || ldw % 8) return le::invalid("le_gemm_tc_grouped_bf16: K (%d) and the leading dimensions must be multiples of 8", K);

@@ -20,7 +20,11 @@
 //          with the pair's weight as a factor (float32 output).  In the gated
 //          form a pair's weight is the factor on the expert's input instead:
 //          both products are multiplied by it, in 32 bits, before the activation.
+//          Without a gate (W[expert] [F, K]) C = act(a W^T) with an ungated
+//          activation, or the plain product.
 // combine: out[t] = sum_j y[t * top + j] (+ gate[t] * shared[t]).
+// Identity experts: ids from the number of real experts on stand for experts whose output is their input.  The
+// grouping leaves their pairs out, and the combination adds weight * h[t] for them instead of a product's row.
 // Where experts have many rows each (prompt portions, bfloat16) the products run on the tcgen05 kernel of
 // gemm_tc.cu in its grouped form instead: the grouping pads every expert's slots to whole tiles of 128, the rows of
 // x are gathered into slot order, both products run over the sorted rows, and the weighted sum reads them back
@@ -123,10 +127,12 @@ moe_logits_kernel(const T *__restrict__ h, int64_t h_stride, const float *__rest
 }
 
 // The choice: a warp per token picks the `top` largest of its logits (ties: the lower index), writes their ids and
-// the softmax over them (`scoring` 0) or each one's own sigmoid (`scoring` 1), and the shared gate's sigmoid.  It
-// marks what it has picked in z.
+// the softmax over them (`scoring` 0) or each one's own sigmoid (`scoring` 1), and the shared gate's sigmoid.
+// `scoring` 2: scores s are the softmax over all logits, the choice goes by s + correction, and the weights are the
+// chosen scores over their sum (+ 1e-20).  It marks what it has picked in z.
 __global__ void moe_pick_kernel(float *__restrict__ z, int32_t *__restrict__ ids, float *__restrict__ weights,
-                                float *__restrict__ gate, int tokens, int experts, int top, int with_gate, int scoring) {
+                                float *__restrict__ gate, const float *__restrict__ correction, int tokens, int experts, int top,
+                                int with_gate, int scoring) {
   le::let_successor_start();
   le::wait_for_predecessor();
   const int t = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
@@ -134,11 +140,20 @@ __global__ void moe_pick_kernel(float *__restrict__ z, int32_t *__restrict__ ids
   float *zt = z + static_cast<int64_t>(t) * (experts + 1);
   if (with_gate && lane == 0) gate[t] = 1.0f / (1.0f + expf(-zt[experts]));
   float first = 0.0f, total = 0.0f;
+  if (scoring == 2) {
+    float m = -INFINITY, sum = 0.0f;
+    for (int e = lane; e < experts; e += 32) m = fmaxf(m, zt[e]);
+    m = le::warp_max(m);
+    for (int e = lane; e < experts; e += 32) sum += expf(zt[e] - m);
+    sum = le::warp_sum(sum);
+    for (int e = lane; e < experts; e += 32) zt[e] = expf(zt[e] - m) / sum;      // (a lane reads and writes its own entries)
+    __syncwarp();
+  }
   for (int j = 0; j < top; ++j) {
     float best = -INFINITY;
     int at = 0x7fffffff;
     for (int e = lane; e < experts; e += 32) {
-      const float v = zt[e];
+      const float v = scoring == 2 && correction != nullptr ? zt[e] + correction[e] : zt[e];
       if (v > best || (v == best && e < at)) { best = v; at = e; }
     }
 #pragma unroll
@@ -150,7 +165,8 @@ __global__ void moe_pick_kernel(float *__restrict__ z, int32_t *__restrict__ ids
     if (at == 0x7fffffff) at = 0;   // (no finite logit left: cannot happen with top <= experts)
     if (j == 0) first = best;
     // scoring 1: the weight is the chosen logit's sigmoid by itself (the largest logits are the largest scores)
-    const float p = scoring == 1 ? 1.0f / (1.0f + expf(-best)) : expf(best - first);
+    const float p = scoring == 1 ? 1.0f / (1.0f + expf(-best)) : (scoring == 2 ? zt[at] : expf(best - first));
+    __syncwarp();                   // (every lane has read the score before it is marked)
     total += p;
     if (lane == 0) {
       ids[static_cast<int64_t>(t) * top + j] = at;
@@ -160,7 +176,7 @@ __global__ void moe_pick_kernel(float *__restrict__ z, int32_t *__restrict__ ids
     __syncwarp();
   }
   if (scoring == 1) return;
-  for (int j = lane; j < top; j += 32) weights[static_cast<int64_t>(t) * top + j] /= total;
+  for (int j = lane; j < top; j += 32) weights[static_cast<int64_t>(t) * top + j] /= (scoring == 2 ? total + 1e-20f : total);
 }
 
 template <typename T, int NT, int RB>
@@ -271,20 +287,24 @@ __global__ void moe_gather_kernel(T *__restrict__ out, const T *__restrict__ x, 
 }
 
 // out[t] = sum_j share[t, j] * y[pair_slot[t * top + j]] (+ gate[t] * shared[t]): the weighted sum over rows that
-// lie in slot order.
+// lie in slot order.  ids (or nullptr): pairs of an identity expert (id >= experts) add share * h[t] instead.
 template <typename T, typename TY>
 __global__ void moe_combine_sorted_kernel(T *__restrict__ out, const TY *__restrict__ y, const int32_t *__restrict__ pair_slot,
                                           const float *__restrict__ share, const T *__restrict__ shared_out,
-                                          const float *__restrict__ gate, int64_t n, int width, int top) {
+                                          const float *__restrict__ gate, const int32_t *__restrict__ ids,
+                                          const T *__restrict__ h, int64_t h_stride, int experts, int64_t n, int width, int top) {
   le::let_successor_start();
   le::wait_for_predecessor();
   const int64_t i = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x;
   if (i >= n) return;
   const int64_t t = i / width, c = i - t * width;
   float acc = 0.0f;
-  for (int j = 0; j < top; ++j)
-    acc = fmaf(share != nullptr ? share[t * top + j] : 1.0f,
-               le::to_f32(y[static_cast<int64_t>(pair_slot[t * top + j]) * width + c]), acc);
+  for (int j = 0; j < top; ++j) {
+    const bool identity = ids != nullptr && ids[t * top + j] >= experts;
+    const float v = identity ? le::to_f32(h[t * h_stride + c])
+                             : le::to_f32(y[static_cast<int64_t>(pair_slot[t * top + j]) * width + c]);
+    acc = fmaf(share != nullptr ? share[t * top + j] : 1.0f, v, acc);
+  }
   if (shared_out != nullptr) acc = fmaf(gate != nullptr ? gate[t] : 1.0f, le::to_f32(shared_out[i]), acc);
   out[i] = le::from_f32<T>(acc);
 }
@@ -368,7 +388,7 @@ __global__ void moe_grouped_kernel(TOut *__restrict__ out, int64_t out_stride, c
         v = le::gated_activation(v * row_factor[m], acc_up[i][j] * row_factor[m], act);
         o[n] = le::from_f32<TOut>(v);
       } else {
-        o[n] = le::from_f32<TOut>(v * row_factor[m]);
+        o[n] = le::from_f32<TOut>(le::ungated_activation(v, act) * row_factor[m]);
       }
     }
   }
@@ -532,7 +552,7 @@ moe_grouped_mma_kernel(TOut *__restrict__ out, int64_t out_stride, const __nv_bf
             v = le::gated_activation(v * f, acc[1][mt][nt][half * 2 + j] * f, act);
             o[n] = le::from_f32<TOut>(v);
           } else {
-            o[n] = le::from_f32<TOut>(v * f);
+            o[n] = le::from_f32<TOut>(le::ungated_activation(v, act) * f);
           }
         }
     }
@@ -556,14 +576,20 @@ int launch_grouped_mma(int N, int max_tiles, cudaStream_t stream, Args... args) 
 
 template <typename T>
 __global__ void moe_combine_kernel(T *__restrict__ out, const float *__restrict__ y, const T *__restrict__ shared_out,
-                                   const float *__restrict__ gate, int64_t n, int width, int top) {
+                                   const float *__restrict__ gate, const int32_t *__restrict__ ids,
+                                   const float *__restrict__ share, const T *__restrict__ h, int64_t h_stride, int experts,
+                                   int64_t n, int width, int top) {
   le::let_successor_start();
   le::wait_for_predecessor();
   const int64_t i = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x;
   if (i >= n) return;
   const int64_t t = i / width, c = i - t * width;
   float acc = 0.0f;
-  for (int j = 0; j < top; ++j) acc += y[(t * top + j) * width + c];
+  for (int j = 0; j < top; ++j) {
+    const int64_t p = t * top + j;
+    if (ids != nullptr && ids[p] >= experts) acc = fmaf(share != nullptr ? share[p] : 1.0f, le::to_f32(h[t * h_stride + c]), acc);
+    else acc += y[p * width + c];
+  }
   if (shared_out != nullptr) acc = fmaf(gate != nullptr ? gate[t] : 1.0f, le::to_f32(shared_out[i]), acc);
   out[i] = le::from_f32<T>(acc);
 }
@@ -572,10 +598,11 @@ __global__ void moe_combine_kernel(T *__restrict__ out, const float *__restrict_
 
 LE_API int le_moe_tile_rows(int wide) { return wide ? TILE_M_WIDE : TILE_M; }
 
-// `z`: float32 scratch [tokens, experts + 1] (the logits; the picked ones are overwritten).
+// `z`: float32 scratch [tokens, experts + 1] (the logits; the picked ones are overwritten).  `correction`: scoring 2
+// only, [experts] or null.
 LE_API int le_moe_route(const void *h, int64_t h_stride, int dtype, const float *w_router, const float *b_router,
-                        const float *w_gate, float *z, int32_t *ids, float *weights, float *gate, int tokens, int width,
-                        int experts, int top, int scoring, cudaStream_t stream) {
+                        const float *w_gate, const float *correction, float *z, int32_t *ids, float *weights, float *gate,
+                        int tokens, int width, int experts, int top, int scoring, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (top < 1 || top > experts) return le::invalid("le_moe_route: %d of %d experts", top, experts);
   // tokens a block takes: up to 8, fewer where the step has fewer or a row is wide
@@ -602,9 +629,10 @@ LE_API int le_moe_route(const void *h, int64_t h_stride, int dtype, const float 
   }
 #undef LE_LOGITS
   if (rc != 0) return rc;
-  if (scoring != 0 && scoring != 1) return le::invalid("le_moe_route: scoring %d is neither 0 (softmax over the chosen) nor 1 (sigmoid)", scoring);
-  return le::launch_chained(moe_pick_kernel, dim3((tokens + 7) / 8), dim3(256), 0, stream, z, ids, weights, gate, tokens, experts,
-                            top, w_gate != nullptr ? 1 : 0, scoring);
+  if (scoring < 0 || scoring > 2)
+    return le::invalid("le_moe_route: scoring %d is none of 0 (softmax over the chosen), 1 (sigmoid), 2 (softmax over all)", scoring);
+  return le::launch_chained(moe_pick_kernel, dim3((tokens + 7) / 8), dim3(256), 0, stream, z, ids, weights, gate, correction,
+                            tokens, experts, top, w_gate != nullptr ? 1 : 0, scoring);
 }
 
 LE_API int le_moe_group(const int32_t *ids, int pairs, int experts, int tile_m, int padded, int max_tiles, int slots_cap,
@@ -634,8 +662,10 @@ LE_API int le_moe_gather(void *out, const void *x, int64_t x_stride, int dtype, 
                             static_cast<const float *>(x), x_stride, slot_pair, src_div, tile_m, meta, width, pair_weight);
 }
 
+// ids null: no identity experts; else ids [tokens, top], h [tokens, width] (row stride h_stride, the type of out).
 LE_API int le_moe_combine_sorted(void *out, int dtype, const void *y, int y_dtype, const int32_t *pair_slot,
-                                 const float *share, const void *shared_out, const float *gate, int tokens, int width, int top,
+                                 const float *share, const void *shared_out, const float *gate, const int32_t *ids,
+                                 const void *h, int64_t h_stride, int experts, int tokens, int width, int top,
                                  cudaStream_t stream) {
   const int64_t n = static_cast<int64_t>(tokens) * width;
   if (n <= 0) return 0;
@@ -643,15 +673,17 @@ LE_API int le_moe_combine_sorted(void *out, int dtype, const void *y, int y_dtyp
   if (dtype == LE_BF16 && y_dtype == LE_F32)
     return le::launch_chained(moe_combine_sorted_kernel<__nv_bfloat16, float>, grid, block, 0, stream,
                               static_cast<__nv_bfloat16 *>(out), static_cast<const float *>(y), pair_slot, share,
-                              static_cast<const __nv_bfloat16 *>(shared_out), gate, n, width, top);
+                              static_cast<const __nv_bfloat16 *>(shared_out), gate, ids, static_cast<const __nv_bfloat16 *>(h),
+                              h_stride, experts, n, width, top);
   if (dtype == LE_BF16 && y_dtype == LE_BF16)
     return le::launch_chained(moe_combine_sorted_kernel<__nv_bfloat16, __nv_bfloat16>, grid, block, 0, stream,
                               static_cast<__nv_bfloat16 *>(out), static_cast<const __nv_bfloat16 *>(y), pair_slot, share,
-                              static_cast<const __nv_bfloat16 *>(shared_out), gate, n, width, top);
+                              static_cast<const __nv_bfloat16 *>(shared_out), gate, ids, static_cast<const __nv_bfloat16 *>(h),
+                              h_stride, experts, n, width, top);
   if (dtype == LE_F32 && y_dtype == LE_F32)
     return le::launch_chained(moe_combine_sorted_kernel<float, float>, grid, block, 0, stream, static_cast<float *>(out),
-                              static_cast<const float *>(y), pair_slot, share, static_cast<const float *>(shared_out), gate, n,
-                              width, top);
+                              static_cast<const float *>(y), pair_slot, share, static_cast<const float *>(shared_out), gate,
+                              ids, static_cast<const float *>(h), h_stride, experts, n, width, top);
   return le::invalid("le_moe_combine_sorted: no form for output type %d and rows of type %d", dtype, y_dtype);
 }
 
@@ -710,14 +742,18 @@ LE_API int le_moe_grouped(void *out, int out_dtype, int64_t out_stride, const vo
   return le::invalid("le_moe_grouped: no form for input type %d, output type %d, gated %d", dtype, out_dtype, gated);
 }
 
-LE_API int le_moe_combine(void *out, int dtype, const float *y, const void *shared_out, const float *gate, int tokens,
-                          int width, int top, cudaStream_t stream) {
+// y holds weighted rows; ids null: no identity experts; else as le_moe_combine_sorted, with the pairs' weights `share`.
+LE_API int le_moe_combine(void *out, int dtype, const float *y, const void *shared_out, const float *gate, const int32_t *ids,
+                          const float *share, const void *h, int64_t h_stride, int experts, int tokens, int width, int top,
+                          cudaStream_t stream) {
   const int64_t n = static_cast<int64_t>(tokens) * width;
   if (n <= 0) return 0;
   const dim3 grid(static_cast<unsigned>((n + 255) / 256)), block(256);
   if (dtype == LE_BF16)
     return le::launch_chained(moe_combine_kernel<__nv_bfloat16>, grid, block, 0, stream, static_cast<__nv_bfloat16 *>(out), y,
-                              static_cast<const __nv_bfloat16 *>(shared_out), gate, n, width, top);
+                              static_cast<const __nv_bfloat16 *>(shared_out), gate, ids, share,
+                              static_cast<const __nv_bfloat16 *>(h), h_stride, experts, n, width, top);
   return le::launch_chained(moe_combine_kernel<float>, grid, block, 0, stream, static_cast<float *>(out), y,
-                            static_cast<const float *>(shared_out), gate, n, width, top);
+                            static_cast<const float *>(shared_out), gate, ids, share, static_cast<const float *>(h), h_stride,
+                            experts, n, width, top);
 }

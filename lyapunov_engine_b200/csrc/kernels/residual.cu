@@ -7,7 +7,8 @@
 //
 // rmsnorm_pair_kernel: one row of the stream, an optional addend y that
 // enters first, either plainly (x += y) or normed, x += y / sqrt(mean(y^2) +
-// eps_y) * wy, then up to two norms of the same x with weights of their own,
+// eps_y) * wy (a plain addend may have a second one beside it, x += y + y2: two
+// sub-layers that read the same norm), then up to two norms of the same x with weights of their own,
 // out_i = x / sqrt(mean(x^2) + eps) * w_i.  With a row list only those rows
 // are normed and the stream is left as it is.
 //
@@ -68,7 +69,7 @@ __device__ __forceinline__ float4 addend4(const Addend &a, int64_t at) {
 // keeps V pieces of four values in registers, and the row is read once.
 template <typename T, int V>
 __global__ void __launch_bounds__(256)
-rmsnorm_pair_wide_kernel(T *__restrict__ out1, T *__restrict__ out2, float *__restrict__ resid, Addend y,
+rmsnorm_pair_wide_kernel(T *__restrict__ out1, T *__restrict__ out2, float *__restrict__ resid, Addend y, Addend y2,
                          const float *__restrict__ wy, float eps_y, const float *__restrict__ w1,
                          const float *__restrict__ w2, float eps, const int32_t *__restrict__ rows, int width) {
   __shared__ float scratch[33];
@@ -85,6 +86,10 @@ rmsnorm_pair_wide_kernel(T *__restrict__ out1, T *__restrict__ out2, float *__re
     if (i < n4) {
       xv[v] = load4(x + 4 * i);
       if (y.data != nullptr) yv[v] = addend4(y, r * width + 4 * i);
+      if (y2.data != nullptr) {
+        const float4 w = addend4(y2, r * width + 4 * i);
+        yv[v].x += w.x, yv[v].y += w.y, yv[v].z += w.z, yv[v].w += w.w;
+      }
     }
   }
   if (y.data != nullptr) {
@@ -160,7 +165,7 @@ residual_add_wide_kernel(float *__restrict__ resid, T *__restrict__ copy, Addend
 
 template <typename T>
 __global__ void __launch_bounds__(256)
-rmsnorm_pair_kernel(T *__restrict__ out1, T *__restrict__ out2, float *__restrict__ resid, Addend y,
+rmsnorm_pair_kernel(T *__restrict__ out1, T *__restrict__ out2, float *__restrict__ resid, Addend y, Addend y2,
                     const float *__restrict__ wy, float eps_y, const float *__restrict__ w1,
                     const float *__restrict__ w2, float eps, const int32_t *__restrict__ rows, int width) {
   extern __shared__ float xs[];          // the row
@@ -173,7 +178,7 @@ rmsnorm_pair_kernel(T *__restrict__ out1, T *__restrict__ out2, float *__restric
   if (y.data != nullptr) {
     float yy = 0.0f;
     for (int i = threadIdx.x; i < width; i += blockDim.x) {
-      const float v = addend_at(y, r * width + i);
+      const float v = addend_at(y, r * width + i) + (y2.data != nullptr ? addend_at(y2, r * width + i) : 0.0f);
       xs[i] = v;
       yy = fmaf(v, v, yy);
     }
@@ -278,19 +283,22 @@ int blocks_for(int64_t total) {
 
 // out1 / out2: [n, width] (out2 null: one norm; out1 null too: the addend enters and nothing is normed); resid
 // [rows, width] float32; y: an addend or null, y_parts partial sums y_stride elements apart; wy null: y enters plainly.
+// y2 (only beside a plain y): a second addend, x += y + y2, or null.
 LE_API int le_rmsnorm_pair(void *out1, void *out2, int out_dtype, float *resid, const void *y, int y_dtype, int y_parts,
-                           int64_t y_stride, const float *wy, float eps_y, const float *w1, const float *w2, float eps,
-                           const int32_t *rows, int n, int width, cudaStream_t stream) {
+                           int64_t y_stride, const void *y2, int y2_dtype, int y2_parts, int64_t y2_stride, const float *wy,
+                           float eps_y, const float *w1, const float *w2, float eps, const int32_t *rows, int n, int width,
+                           cudaStream_t stream) {
   if (n <= 0) return 0;
   if (width < 1 || width > 32 * 1024) return le::invalid("le_rmsnorm_pair: rows of %d values (at most 32768)", width);
   if (out1 == nullptr && (out2 != nullptr || rows != nullptr)) return le::invalid("le_rmsnorm_pair: nothing to write");
-  const Addend add{y, y_dtype, y_parts < 1 ? 1 : y_parts, y_stride};
-  if (width % 4 == 0 && width <= 8192 && y_stride % 4 == 0 && on16(out1) && on16(out2) && on16(resid) && on16(y) &&
+  if (y2 != nullptr && (y == nullptr || wy != nullptr)) return le::invalid("le_rmsnorm_pair: a second addend stands beside a plain first one");
+  const Addend add{y, y_dtype, y_parts < 1 ? 1 : y_parts, y_stride}, add2{y2, y2_dtype, y2_parts < 1 ? 1 : y2_parts, y2_stride};
+  if (width % 4 == 0 && width <= 8192 && y_stride % 4 == 0 && y2_stride % 4 == 0 && on16(out1) && on16(out2) && on16(resid) && on16(y) && on16(y2) &&
       on16(wy) && on16(w1) && on16(w2)) {
 #define LE_GO(V)                                                                                                        \
   LE_DISPATCH_DTYPE(out_dtype, T,                                                                                       \
                     return le::launch_chained(rmsnorm_pair_wide_kernel<T, V>, dim3(n), dim3(256), 0, stream,            \
-                                              static_cast<T *>(out1), static_cast<T *>(out2), resid, add, wy, eps_y, w1, \
+                                              static_cast<T *>(out1), static_cast<T *>(out2), resid, add, add2, wy, eps_y, w1, \
                                               w2, eps, rows, width))
     if (width <= 1024) LE_GO(1);
     if (width <= 2048) LE_GO(2);
@@ -302,7 +310,7 @@ LE_API int le_rmsnorm_pair(void *out1, void *out2, int out_dtype, float *resid, 
   LE_DISPATCH_DTYPE(out_dtype, T,
                     if (smem > 40 * 1024) cudaFuncSetAttribute(rmsnorm_pair_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
                     return le::launch_chained(rmsnorm_pair_kernel<T>, dim3(n), dim3(256), smem, stream,
-                                              static_cast<T *>(out1), static_cast<T *>(out2), resid, add, wy, eps_y, w1, w2,
+                                              static_cast<T *>(out1), static_cast<T *>(out2), resid, add, add2, wy, eps_y, w1, w2,
                                               eps, rows, width));
 }
 

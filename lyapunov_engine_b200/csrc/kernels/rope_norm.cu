@@ -9,9 +9,14 @@
 // angle position * rates[i]: (a, b) -> (a cos - b sin, b cos + a sin).  With
 // `unit` set the turned head is then divided by sqrt(mean(head^2) + eps) over
 // its first norm_dim entries (the entries behind them are padding and zero).
+// With weights of head_dim entries (one set for queries, one for keys, shared by
+// the heads) the result is multiplied by them, and with a query temperature
+// (coef, every) queries at position p are multiplied by
+// 1 + coef * ln(floor((p + 1) / every) + 1).
 // Queries are rewritten in place; keys go to the key pool; the value pool
 // receives the keys as projected (before turn and norm) when
-// `values_are_keys`, else nothing.  A warp takes a head, a lane up to eight
+// `values_are_keys`, the value heads [kv_heads][head_dim] behind the keys as
+// they are when `store_values`, else nothing.  A warp takes a head, a lane up to eight
 // pairs of it; a token's sines and cosines are made once per block.  Angle,
 // sine, cosine, turn and norm are 32-bit; the result is rounded once.
 //
@@ -27,6 +32,17 @@
 namespace {
 
 constexpr int RN_MAX_PAIRS = 8;      // pairs a lane holds: heads of up to 512 entries
+
+// What a caller may add to the turn and the norm.
+struct HeadExtras {
+  const float *w_q, *w_k;      // [head_dim] each, or null
+  float temp_coef;             // temp_every 0: no query temperature
+  int temp_every;
+  int store_values;            // the rows' value heads go to the value pool
+};
+__device__ __forceinline__ float query_temperature(int pos, const HeadExtras &x) {
+  return x.temp_every > 0 ? fmaf(x.temp_coef, logf(static_cast<float>((pos + 1) / x.temp_every + 1)), 1.0f) : 1.0f;
+}
 
 // Two neighbouring entries at once where the address allows it.
 template <typename T>
@@ -65,7 +81,7 @@ rope_norm_store_kernel(T *__restrict__ rows, int64_t row_stride, T *__restrict__
                        const int32_t *__restrict__ request_of_token, const int32_t *__restrict__ block_table,
                        int max_blocks, int heads, int kv_heads, int head_dim, int rot_col, int rot, int unit, float eps,
                        int norm_dim, int page_size, int num_pages, int write_kv, int values_are_keys, int heads_per_block,
-                       int together, int *__restrict__ status) {
+                       int together, HeadExtras extras, int *__restrict__ status) {
   extern __shared__ float turn[];            // [rot / 2][2]: sine, cosine
   le::let_successor_start();
   le::wait_for_predecessor();
@@ -85,19 +101,22 @@ rope_norm_store_kernel(T *__restrict__ rows, int64_t row_stride, T *__restrict__
   }
   __syncthreads();
   const int pairs = head_dim >> 1;
-  const int all = heads + (write_kv ? kv_heads : 0);
+  const int all = heads + (write_kv ? kv_heads * (extras.store_values ? 2 : 1) : 0);
+  const float temperature = query_temperature(pos, extras);
   const int h_end = min(all, (static_cast<int>(blockIdx.y) + 1) * heads_per_block);
   for (int h = blockIdx.y * heads_per_block + warp; h < h_end; h += warps) {
     T *x = row + static_cast<int64_t>(h) * head_dim;
-    const bool is_key = h >= heads;
-    if (is_key && bad) continue;
+    const bool is_value = h >= heads + kv_heads;
+    const bool is_key = h >= heads && !is_value;
+    if ((is_key || is_value) && bad) continue;
     float a[RN_MAX_PAIRS], b[RN_MAX_PAIRS];
     float ss = 0.0f;
     T *k_dst = nullptr, *v_dst = nullptr;
-    if (is_key) {
-      const int64_t at = ((static_cast<int64_t>(page) * kv_heads + (h - heads)) * page_size + pos % page_size) * head_dim;
-      k_dst = k_cache + at;
-      v_dst = values_are_keys ? v_cache + at : nullptr;
+    if (is_key || is_value) {
+      const int kvh = is_value ? h - heads - kv_heads : h - heads;
+      const int64_t at = ((static_cast<int64_t>(page) * kv_heads + kvh) * page_size + pos % page_size) * head_dim;
+      k_dst = is_value ? v_cache + at : k_cache + at;
+      v_dst = values_are_keys && is_key ? v_cache + at : nullptr;
     }
 #pragma unroll
     for (int i = 0; i < RN_MAX_PAIRS; ++i) {
@@ -107,7 +126,7 @@ rope_norm_store_kernel(T *__restrict__ rows, int64_t row_stride, T *__restrict__
         load_pair(x + 2 * p, together, u, v);
         if (v_dst != nullptr) store_pair(v_dst + 2 * p, together, u, v);     // (as projected: the same bits)
         const int j = 2 * p - rot_col;
-        if (j >= 0 && j + 1 < rot) {
+        if (j >= 0 && j + 1 < rot && !is_value) {
           const float s = turn[j], c = turn[j + 1];
           const float nu = u * c - v * s, nv = v * c + u * s;
           u = nu, v = nv;
@@ -117,12 +136,17 @@ rope_norm_store_kernel(T *__restrict__ rows, int64_t row_stride, T *__restrict__
       }
     }
     float inv = 1.0f;
-    if (unit) inv = rsqrtf(le::warp_sum(ss) / static_cast<float>(norm_dim) + eps);
-    T *dst = is_key ? k_dst : x;
+    if (unit && !is_value) inv = rsqrtf(le::warp_sum(ss) / static_cast<float>(norm_dim) + eps);
+    const float *w = is_value ? nullptr : (is_key ? extras.w_k : extras.w_q);
+    if (!is_key && !is_value) inv *= temperature;
+    T *dst = is_key || is_value ? k_dst : x;
 #pragma unroll
     for (int i = 0; i < RN_MAX_PAIRS; ++i) {
       const int p = lane + 32 * i;
-      if (p < pairs) store_pair(dst + 2 * p, together, a[i] * inv, b[i] * inv);
+      if (p < pairs) {
+        if (w != nullptr) a[i] *= w[2 * p], b[i] *= w[2 * p + 1];
+        store_pair(dst + 2 * p, together, a[i] * inv, b[i] * inv);
+      }
     }
   }
 }
@@ -168,7 +192,7 @@ rope_norm_store_pieces_kernel(T *__restrict__ rows, int64_t row_stride, T *__res
                               const int32_t *__restrict__ request_of_token, const int32_t *__restrict__ block_table,
                               int max_blocks, int heads, int kv_heads, int head_dim, int rot_col, int rot, int unit, float eps,
                               int norm_dim, int page_size, int num_pages, int write_kv, int values_are_keys,
-                              int heads_per_block, int lph, int *__restrict__ status) {
+                              int heads_per_block, int lph, HeadExtras extras, int *__restrict__ status) {
   constexpr int N = Piece<T>::N;
   constexpr int HELD = 2 * RN_MAX_PAIRS / N;          // pieces a lane holds at most
   extern __shared__ float turn[];                     // [rot / 2][2]: sine, cosine
@@ -191,18 +215,21 @@ rope_norm_store_pieces_kernel(T *__restrict__ rows, int64_t row_stride, T *__res
   __syncthreads();
   const int at_once = 32 / lph, sub = lane % lph, mine = lane / lph;
   const int pieces = head_dim / N;
-  const int all = heads + (write_kv ? kv_heads : 0);
+  const int all = heads + (write_kv ? kv_heads * (extras.store_values ? 2 : 1) : 0);
+  const float temperature = query_temperature(pos, extras);
   const int h_end = min(all, (static_cast<int>(blockIdx.y) + 1) * heads_per_block);
   for (int h0 = blockIdx.y * heads_per_block + warp * at_once; h0 < h_end; h0 += warps * at_once) {
     const int h = h0 + mine;
-    const bool is_key = h >= heads;
-    const bool live = h < h_end && !(is_key && bad);
+    const bool is_value = h >= heads + kv_heads;
+    const bool is_key = h >= heads && !is_value;
+    const bool live = h < h_end && !((is_key || is_value) && bad);
     T *x = row + static_cast<int64_t>(h) * head_dim;
     T *k_dst = nullptr, *v_dst = nullptr;
-    if (live && is_key) {
-      const int64_t at = ((static_cast<int64_t>(page) * kv_heads + (h - heads)) * page_size + pos % page_size) * head_dim;
-      k_dst = k_cache + at;
-      v_dst = values_are_keys ? v_cache + at : nullptr;
+    if (live && (is_key || is_value)) {
+      const int kvh = is_value ? h - heads - kv_heads : h - heads;
+      const int64_t at = ((static_cast<int64_t>(page) * kv_heads + kvh) * page_size + pos % page_size) * head_dim;
+      k_dst = is_value ? v_cache + at : k_cache + at;
+      v_dst = values_are_keys && is_key ? v_cache + at : nullptr;
     }
     float val[HELD][N];
     float ss = 0.0f;
@@ -217,7 +244,7 @@ rope_norm_store_pieces_kernel(T *__restrict__ rows, int64_t row_stride, T *__res
         for (int e = 0; e < N; e += 2) {
           const int j = c * N + e - rot_col;
           float u = val[i][e], v = val[i][e + 1];
-          if (j >= 0 && j + 1 < rot) {
+          if (j >= 0 && j + 1 < rot && !is_value) {
             const float sn = turn[j], cs = turn[j + 1];
             const float nu = u * cs - v * sn, nv = v * cs + u * sn;
             u = nu, v = nv;
@@ -230,12 +257,18 @@ rope_norm_store_pieces_kernel(T *__restrict__ rows, int64_t row_stride, T *__res
     float inv = 1.0f;
     if (unit) {
       for (int o = 1; o < lph; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-      inv = rsqrtf(ss / static_cast<float>(norm_dim) + eps);
+      if (!is_value) inv = rsqrtf(ss / static_cast<float>(norm_dim) + eps);
     }
-    T *dst = is_key ? k_dst : x;
+    const float *w = is_value ? nullptr : (is_key ? extras.w_k : extras.w_q);
+    if (!is_key && !is_value) inv *= temperature;
+    T *dst = is_key || is_value ? k_dst : x;
 #pragma unroll
     for (int i = 0; i < HELD; ++i) {
       const int c = sub + i * lph;
+      if (live && c < pieces && w != nullptr) {
+#pragma unroll
+        for (int e = 0; e < N; ++e) val[i][e] *= w[c * N + e];
+      }
       if (live && c < pieces) *reinterpret_cast<uint4 *>(dst + c * N) = Piece<T>::close(val[i], inv);
     }
   }
@@ -311,17 +344,21 @@ latent_rope_store_kernel(const T *__restrict__ src, int64_t src_stride, int col,
 
 // rows: [tokens] rows of row_stride elements, queries then keys, heads of head_dim entries (even, at most 512).
 // k_cache / v_cache: [pages, kv_heads, page, head_dim].  write_kv 0: queries only (the keys' columns are not read).
+// w_q / w_k: float32 [head_dim] or null; temp_every 0: no query temperature; store_values: value heads lie behind the keys.
 LE_API int le_rope_norm_store(void *rows, int64_t row_stride, int dtype, void *k_cache, void *v_cache, const float *rates,
                               const int32_t *positions, const int32_t *request_of_token, const int32_t *block_table,
                               int max_blocks, int num_tokens, int heads, int kv_heads, int head_dim, int rot_col, int rot,
                               int unit, float eps, int norm_dim, int page_size, int num_pages, int write_kv,
-                              int values_are_keys, int *status, cudaStream_t stream) {
+                              int values_are_keys, const float *w_q, const float *w_k, float temp_coef, int temp_every,
+                              int store_values, int *status, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
+  if (temp_every < 0 || (values_are_keys && store_values)) return le::invalid("le_rope_norm_store: bad options");
+  const HeadExtras extras{w_q, w_k, temp_coef, temp_every, store_values};
   if (head_dim < 2 || head_dim % 2 || head_dim > 64 * RN_MAX_PAIRS)
     return le::invalid("le_rope_norm_store: heads of %d entries (even, at most %d)", head_dim, 64 * RN_MAX_PAIRS);
   if (rot < 0 || rot % 2 || rot_col < 0 || rot_col % 2 || rot_col + rot > head_dim)
     return le::invalid("le_rope_norm_store: %d turned entries from column %d of a head of %d", rot, rot_col, head_dim);
-  const int all = heads + (write_kv ? kv_heads : 0);
+  const int all = heads + (write_kv ? kv_heads * (store_values ? 2 : 1) : 0);
   const int per_block = num_tokens >= 512 ? 16 : 4;       // few tokens: more blocks; many: the sines serve more heads
   const dim3 grid(num_tokens, (all + per_block - 1) / per_block);
   if (grid.y > 65535) return le::invalid("le_rope_norm_store: %d heads are too many for one launch", all);
@@ -339,14 +376,14 @@ LE_API int le_rope_norm_store(void *rows, int64_t row_stride, int dtype, void *k
                                                 static_cast<T *>(rows), row_stride, static_cast<T *>(k_cache),
                                                 static_cast<T *>(v_cache), rates, positions, request_of_token, block_table,
                                                 max_blocks, heads, kv_heads, head_dim, rot_col, rot, unit, eps, norm_dim,
-                                                page_size, num_pages, write_kv, values_are_keys, per_block, lph, status));
+                                                page_size, num_pages, write_kv, values_are_keys, per_block, lph, extras, status));
   }
   LE_DISPATCH_DTYPE(dtype, T,
                     return le::launch_chained(rope_norm_store_kernel<T>, grid, dim3(128), smem, stream,
                                               static_cast<T *>(rows), row_stride, static_cast<T *>(k_cache),
                                               static_cast<T *>(v_cache), rates, positions, request_of_token, block_table,
                                               max_blocks, heads, kv_heads, head_dim, rot_col, rot, unit, eps, norm_dim,
-                                              page_size, num_pages, write_kv, values_are_keys, per_block, together, status));
+                                              page_size, num_pages, write_kv, values_are_keys, per_block, together, extras, status));
 }
 
 // cache: [pages, 1, page, padded] or null (nothing is stored); out2 null: no second latent.

@@ -92,12 +92,12 @@ _CORE_SIGNATURES = {
                           c_int, c_int, c_int, c_float, c_void_p],
     "le_rope_norm_store": [c_void_p, c_int64, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                            c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_int, c_int,
-                           c_void_p, c_void_p],
+                           c_void_p, c_void_p, c_float, c_int, c_int, c_void_p, c_void_p],
     "le_latent_rope_store": [c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p,
                              c_int, c_int, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                              c_int, c_void_p, c_void_p],
-    "le_rmsnorm_pair": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int64, c_void_p, c_float, c_void_p,
-                        c_void_p, c_float, c_void_p, c_int, c_int, c_void_p],
+    "le_rmsnorm_pair": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int64, c_void_p, c_int, c_int, c_int64,
+                        c_void_p, c_float, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_void_p],
     "le_residual_add": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int64, c_void_p, c_int, c_int, c_int64,
                         c_void_p, c_int, c_int, c_void_p],
     "le_gate_rows": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int64, c_int, c_void_p, c_int, c_int, c_int, c_void_p,
@@ -107,6 +107,13 @@ _CORE_SIGNATURES = {
     "le_ssm_scan": [c_void_p, c_int, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_void_p, c_int64, c_void_p,
                     c_int64, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                     c_int, c_int, c_int, c_float, c_void_p],
+    "le_activate": [c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_void_p],
+    "le_lightning_segment": [],
+    "le_lightning_chunk": [],
+    "le_lightning_scan": [c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
+                          c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "le_lightning_chunks": [c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int,
+                            c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "le_mlstm_rows": [c_int, c_int],
     "le_mlstm_scan": [c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
                       c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p],
@@ -146,19 +153,20 @@ _CORE_SIGNATURES = {
                         c_float, c_void_p],
     "le_softcap": [c_void_p, c_int64, c_float, c_void_p],
     "le_moe_tile_rows": [c_int],
-    "le_moe_route": [c_void_p, c_int64, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+    "le_moe_route": [c_void_p, c_int64, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                      c_int, c_int, c_int, c_int, c_void_p],
     "le_moe_group": [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                      c_void_p, c_void_p],
     "le_moe_gather": [c_void_p, c_void_p, c_int64, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p],
-    "le_moe_combine_sorted": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                              c_void_p],
+    "le_moe_combine_sorted": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                              c_int64, c_int, c_int, c_int, c_int, c_void_p],
     "le_gemm_tc_grouped_bf16": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int64, c_int64, c_int64, c_int,
                                 c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_void_p, c_void_p],
     "le_moe_grouped": [c_void_p, c_int, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_int64, c_int, c_void_p, c_int,
                        c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                        c_float, c_float, c_void_p],
-    "le_moe_combine": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+    "le_moe_combine": [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_int, c_int, c_int,
+                       c_int, c_void_p],
     "le_argmax": [c_void_p, c_void_p, c_int, c_int, c_int64, c_void_p, c_void_p],
     "le_sample": [c_void_p, c_void_p, c_int, c_int, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                   c_void_p, c_void_p],
@@ -166,7 +174,7 @@ _CORE_SIGNATURES = {
 _ATTENTION_SIGNATURES = {
     "le_attention_generic": [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_void_p, c_int,
                              c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
-                             c_float, c_void_p, c_int, c_float, c_void_p, c_void_p],
+                             c_float, c_void_p, c_int, c_float, c_void_p, c_void_p, c_void_p],
 }
 
 
@@ -208,16 +216,16 @@ def attention_lib(head_dim: int):
 _EXTRA_ATTENTION_SIGNATURES: dict[str, list] = {
     "le_attention_prefill_bf16": [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                                   c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-                                  c_void_p, c_int, c_float, c_void_p, c_void_p],
+                                  c_void_p, c_int, c_float, c_void_p, c_void_p, c_void_p],
     "le_attention_prefill_tc_bf16": [c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_void_p, c_void_p, c_void_p,
                                      c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                                     c_int, c_float, c_void_p, c_void_p, c_void_p],
+                                     c_int, c_float, c_void_p, c_void_p, c_void_p, c_void_p],
     "le_attention_decode_bf16": [c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int,
                                  c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
                                  c_int, c_void_p, c_void_p],
     "le_attention_decode_bf16_form": [c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int,
                                       c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-                                      c_void_p, c_int, c_float, c_int, c_int, c_void_p, c_void_p],
+                                      c_void_p, c_int, c_float, c_void_p, c_int, c_int, c_void_p, c_void_p],
 }
 
 
@@ -318,6 +326,8 @@ def swiglu(out: torch.Tensor, gate_up: torch.Tensor) -> None:
 
 
 GLU_SILU, GLU_CLAMPED, GLU_RELU = 0, 1, 2
+# activations of a product without a gate (as the second-to-last numbers of the products' ``activation``): max(v, 0)^2
+ACT_SILU, ACT_RELU_SQUARED = 0, 3
 
 
 def glu(out: torch.Tensor, gate_up: torch.Tensor, kind: int = GLU_SILU, alpha: float = 1.0, limit: float = 0.0,
@@ -332,6 +342,17 @@ def glu(out: torch.Tensor, gate_up: torch.Tensor, kind: int = GLU_SILU, alpha: f
     assert bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == 2 * I)
     _check(core().le_glu_bias(_ptr(out), _ptr(gate_up), dtype_code(out.dtype), T, I, int(kind), float(alpha), float(limit),
                               _ptr(bias), _stream()), "le_glu_bias")
+
+
+def activate(out: torch.Tensor, x: torch.Tensor, kind: int) -> None:
+    """out[t, i] = silu(x[t, i]) (ACT_SILU) or max(x[t, i], 0)^2
+    (ACT_RELU_SQUARED); column ranges of wider rows are fine, and ``out`` may
+    be ``x``."""
+    _need_cuda(out, x)
+    T, W = x.shape
+    assert out.shape == x.shape and out.dtype == x.dtype and out.stride(1) == 1 and x.stride(1) == 1
+    _check(core().le_activate(_ptr(out), out.stride(0), _ptr(x), x.stride(0), dtype_code(x.dtype), T, W, int(kind), _stream()),
+           "le_activate")
 
 
 def embed_sinusoid(out_resid, table, ids, positions, rates, status) -> None:
@@ -590,7 +611,9 @@ def gemm_skinny(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, splits: int
     inputs).  ``splits`` > 1: ``out`` is float32 [splits, M, N] partial sums.
     ``gated``: ``w`` is [2 I, K] (gate rows, then up rows), out = act(gate, up)
     with ``activation`` = (kind, slope, limit) as glu() takes them (silu(gate) * up by default), and
-    ``bias`` (float32 [2 I] or None) added to the product's columns before it."""
+    ``bias`` (float32 [2 I] or None) added to the product's columns before it.
+    Without a gate and with one split, the kind ACT_RELU_SQUARED puts that
+    activation on the product."""
     _need_cuda(out, a, w, bias)
     M, K = a.shape
     N = w.shape[0]
@@ -648,7 +671,8 @@ def gemm_tc(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, gated: bool = F
     out = a @ w^T (bfloat16 or float32), or with ``gated`` out = act(a Wg^T,
     a Wu^T) for w = [Wg; Wu], ``activation`` = (kind, slope, limit) as glu()
     takes them (silu(g) * u by default), and ``bias`` (float32 [2 I] or None)
-    added to the product's columns before it."""
+    added to the product's columns before it.  Without a gate the kind
+    ACT_RELU_SQUARED puts that activation on the product."""
     _need_cuda(out, a, w, bias)
     M, K = a.shape
     N = w.shape[0]
@@ -737,6 +761,21 @@ def gated_linear(out: torch.Tensor, a: torch.Tensor, w_gate_up: torch.Tensor, wo
     glu(out, gu, *activation)
 
 
+def activated_linear(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, kind: int, status=None) -> None:
+    """out = act(a @ w^T) for an activation without a gate (``kind``:
+    ACT_RELU_SQUARED).  bfloat16: one kernel of the package (weight-streaming
+    for few rows, tcgen05 for many) with the activation in its epilogue, on
+    the 32-bit sums; else the product, then the activation's kernel."""
+    if skinny_applies(a, w):
+        gemm_skinny(out, a, w, activation=(kind, 1.0, 0.0))
+        return
+    if tc_applies(a, w):
+        gemm_tc(out, a, w, status=status, activation=(kind, 1.0, 0.0))
+        return
+    linear(out, a, w, status)
+    activate(out, out, kind)
+
+
 FUSE_GATED_BIAS = os.environ.get("LYAPUNOV_FUSE_GATED_BIAS", "1") not in ("0", "")
 
 
@@ -819,11 +858,12 @@ def _head_scale(head_scale, num_heads):
 
 def attention_generic(out, q, q_stride, k_cache, v_cache, block_table, cu_q, ctx_before, tile_request, tile_q0,
                       num_tiles, num_heads, num_kv_heads, head_dim, page_size, reach, scale, status, head_scale=None,
-                      keep_first: int = 0, softcap: float = 0.0) -> None:
+                      keep_first: int = 0, softcap: float = 0.0, sink=None) -> None:
     """``reach``: see reach_code.  ``head_scale`` (float32 [num_heads] or None):
     one more factor per query head on its scores.  ``keep_first`` n: the keys
     at positions below n stay visible behind a window.  ``softcap`` c > 0: a
-    score s becomes c * tanh(s / c)."""
+    score s becomes c * tanh(s / c).  ``sink`` (float32 [num_heads] or None):
+    the softmax's denominator has one more term exp(sink) per head."""
     _need_cuda(out, q, k_cache, v_cache, block_table)
     lib = attention_lib(head_dim)
     assert out.is_contiguous() and out.shape[1] == num_heads * head_dim
@@ -832,8 +872,8 @@ def attention_generic(out, q, q_stride, k_cache, v_cache, block_table, cu_q, ctx
                                     dtype_code(out.dtype), _ptr(block_table), block_table.shape[1], _ptr(cu_q),
                                     _ptr(ctx_before), _ptr(tile_request), _ptr(tile_q0), num_tiles, num_heads,
                                     num_kv_heads, page_size, k_cache.shape[0], int(reach or 0), float(scale),
-                                    _head_scale(head_scale, num_heads), int(keep_first), float(softcap), _ptr(status),
-                                    _stream()), "le_attention_generic", lib)
+                                    _head_scale(head_scale, num_heads), int(keep_first), float(softcap),
+                                    _head_scale(sink, num_heads), _ptr(status), _stream()), "le_attention_generic", lib)
 
 
 def attention_mma_available(head_dim: int) -> bool:
@@ -844,9 +884,9 @@ def attention_mma_available(head_dim: int) -> bool:
 
 def attention_prefill_bf16(out, q, q_stride, k_cache, v_cache, block_table, cu_q, ctx_before, tile_request, tile_q0,
                            num_tiles, num_heads, num_kv_heads, head_dim, page_size, reach, scale, status,
-                           head_scale=None, keep_first: int = 0, softcap: float = 0.0) -> None:
+                           head_scale=None, keep_first: int = 0, softcap: float = 0.0, sink=None) -> None:
     """Tensor-core attention for requests that bring several tokens; the tiles
-    list 128 query tokens each.  ``keep_first``, ``softcap``: as attention_generic."""
+    list 128 query tokens each.  ``keep_first``, ``softcap``, ``sink``: as attention_generic."""
     _need_cuda(out, q, k_cache, v_cache, block_table)
     lib = attention_lib(head_dim)
     assert out.dtype == torch.bfloat16 and out.is_contiguous() and out.shape[1] == num_heads * head_dim
@@ -855,8 +895,8 @@ def attention_prefill_bf16(out, q, q_stride, k_cache, v_cache, block_table, cu_q
                                          _ptr(block_table), block_table.shape[1], _ptr(cu_q), _ptr(ctx_before),
                                          _ptr(tile_request), _ptr(tile_q0), num_tiles, num_heads, num_kv_heads,
                                          page_size, k_cache.shape[0], int(reach or 0), float(scale),
-                                         _head_scale(head_scale, num_heads), int(keep_first), float(softcap), _ptr(status),
-                                         _stream()),
+                                         _head_scale(head_scale, num_heads), int(keep_first), float(softcap),
+                                         _head_scale(sink, num_heads), _ptr(status), _stream()),
            "le_attention_prefill_bf16", lib)
 
 
@@ -867,11 +907,12 @@ def attention_tc_available(head_dim: int, page_size: int) -> bool:
 
 def attention_prefill_tc_bf16(out, q, q_stride, k_cache, v_cache, block_table, cu_q, ctx_before, tile_request, tile_q0,
                               num_tiles, num_heads, num_kv_heads, head_dim, page_size, reach, scale, status,
-                              head_scale=None) -> None:
+                              head_scale=None, sink=None) -> None:
     """tcgen05 / TMA attention for requests that bring several tokens (head
     sizes 64 and 128, pages of 8..128 keys); the tiles list 128 query tokens
     each.  ``q`` is the [T, width] buffer whose rows start with the query heads.
-    ``head_scale`` must be positive here (the kernel folds it into the exponent's scale)."""
+    ``head_scale`` must be positive here (the kernel folds it into the exponent's scale).
+    ``sink``: as attention_generic."""
     _need_cuda(out, q, k_cache, v_cache, block_table)
     lib = attention_lib(head_dim)
     assert out.dtype == torch.bfloat16 and out.is_contiguous() and out.shape[1] == num_heads * head_dim
@@ -881,7 +922,8 @@ def attention_prefill_tc_bf16(out, q, q_stride, k_cache, v_cache, block_table, c
                                             _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1],
                                             _ptr(cu_q), _ptr(ctx_before), _ptr(tile_request), _ptr(tile_q0), num_tiles,
                                             num_heads, num_kv_heads, page_size, k_cache.shape[0], int(reach or 0),
-                                            float(scale), _head_scale(head_scale, num_heads), _ptr(status), _stream()),
+                                            float(scale), _head_scale(head_scale, num_heads), _head_scale(sink, num_heads),
+                                            _ptr(status), _stream()),
            "le_attention_prefill_tc_bf16", lib)
 
 
@@ -913,9 +955,9 @@ def attention_decode_resident_blocks(head_dim: int, num_splits: int, small: bool
 
 def attention_decode_bf16(out, scratch, q, q_stride, k_cache, v_cache, block_table, cu_q, ctx_before, requests,
                           num_requests, num_heads, num_kv_heads, head_dim, page_size, reach, scale, num_splits,
-                          status, small_form=None, head_scale=None, keep_first: int = 0, softcap: float = 0.0) -> None:
+                          status, small_form=None, head_scale=None, keep_first: int = 0, softcap: float = 0.0, sink=None) -> None:
     """Split-key tensor-core attention for requests that bring one token
-    (``keep_first``, ``softcap``: as attention_generic).
+    (``keep_first``, ``softcap``, ``sink``: as attention_generic).
     ``scratch``: float32, attention_decode_scratch_floats(...) elements.
     ``small_form``: None lets the launcher choose between the kernel's usual
     form and the one with 16-key tiles by the number of blocks; a caller that
@@ -932,8 +974,8 @@ def attention_decode_bf16(out, scratch, q, q_stride, k_cache, v_cache, block_tab
                                              _ptr(v_cache), _ptr(block_table), block_table.shape[1], _ptr(cu_q),
                                              _ptr(ctx_before), _ptr(requests), num_requests, num_heads, num_kv_heads,
                                              page_size, k_cache.shape[0], int(reach or 0), float(scale),
-                                             _head_scale(head_scale, num_heads), int(keep_first), float(softcap), num_splits,
-                                             form, _ptr(status), _stream()),
+                                             _head_scale(head_scale, num_heads), int(keep_first), float(softcap),
+                                             _head_scale(sink, num_heads), num_splits, form, _ptr(status), _stream()),
            "le_attention_decode_bf16", lib,
            launches=2 if num_splits > 1 else 1)       # the attention kernel and the merge
 
@@ -1092,20 +1134,25 @@ def moe_max_tiles(pairs: int, experts: int, wide: bool = False) -> int:
     return pairs // moe_tile_rows(wide) + min(experts, pairs)
 
 
-MOE_SOFTMAX_CHOSEN, MOE_SIGMOID = 0, 1
+MOE_SOFTMAX_CHOSEN, MOE_SIGMOID, MOE_SOFTMAX_ALL = 0, 1, 2
 
 
-def moe_route(ids, weights, gate, h, w_router, b_router, w_gate, top: int, scratch=None, scoring: int = MOE_SOFTMAX_CHOSEN) -> None:
+def moe_route(ids, weights, gate, h, w_router, b_router, w_gate, top: int, scratch=None, scoring: int = MOE_SOFTMAX_CHOSEN,
+              correction=None) -> None:
     """Per row of ``h``: router logits W h + b in 32 bits, the ``top`` largest
     (``ids`` int32 [T, top], best first), softmax over the chosen logits
     (``weights`` float32 [T, top]; ``scoring`` MOE_SIGMOID: each chosen
-    logit's own sigmoid instead, not renormalized); with ``w_gate`` (float32 [W]) also
+    logit's own sigmoid instead, not renormalized; MOE_SOFTMAX_ALL: scores s
+    are the softmax over all logits, the choice goes by s + ``correction``
+    (float32 [experts] or None) and the weights are the chosen s over their
+    sum + 1e-20); with ``w_gate`` (float32 [W]) also
     ``gate`` [T] = sigmoid(w_gate . h).  ``scratch``: float32, T * (experts +
     1) elements, for the logits (made here when not given: a caller whose
     steps are captured passes its own)."""
-    _need_cuda(ids, weights, gate, h, w_router, b_router, w_gate, scratch)
+    _need_cuda(ids, weights, gate, h, w_router, b_router, w_gate, scratch, correction)
     T, W = h.shape
     E = w_router.shape[0]
+    assert correction is None or (scoring == MOE_SOFTMAX_ALL and correction.dtype == torch.float32 and correction.numel() == E)
     assert w_router.dtype == torch.float32 and w_router.is_contiguous() and w_router.shape[1] == W and h.stride(1) == 1
     assert b_router is None or (b_router.dtype == torch.float32 and b_router.numel() == E)
     assert ids.dtype == torch.int32 and ids.is_contiguous() and tuple(ids.shape) == (T, top)
@@ -1116,13 +1163,14 @@ def moe_route(ids, weights, gate, h, w_router, b_router, w_gate, top: int, scrat
         scratch = torch.empty(T * (E + 1), dtype=torch.float32, device=h.device)
     assert scratch.dtype == torch.float32 and scratch.is_contiguous() and scratch.numel() >= T * (E + 1)
     _check(core().le_moe_route(_ptr(h), h.stride(0), dtype_code(h.dtype), _ptr(w_router), _ptr(b_router), _ptr(w_gate),
-                               _ptr(scratch), _ptr(ids), _ptr(weights), _ptr(gate), T, W, E, top, int(scoring), _stream()),
+                               _ptr(correction), _ptr(scratch), _ptr(ids), _ptr(weights), _ptr(gate), T, W, E, top, int(scoring), _stream()),
            "le_moe_route",
            launches=2)
 
 
 def moe_group(ids, experts: int, slot_pair, tiles, meta, wide: bool = False, padded: bool = False, pair_slot=None) -> None:
-    """Sorts the pairs (entries of ``ids``) by expert: ``slot_pair`` int32
+    """Sorts the pairs (entries of ``ids``) by expert (ids from ``experts`` on,
+    which stand for experts without a product, are left out): ``slot_pair`` int32
     lists the pairs expert by expert; ``tiles`` int32 [3, max tiles] (expert,
     first slot, rows of each row tile; unused entries zero); ``meta[0]`` the
     tile count.  ``padded``: every expert's slots start at a multiple of the
@@ -1154,16 +1202,30 @@ def moe_gather(out, x, slot_pair, meta, src_div: int, wide: bool = True, pair_we
            "le_moe_gather")
 
 
-def moe_combine_sorted(out, y, pair_slot, share, top: int, shared_out=None, gate=None) -> None:
-    """out[t] = sum_j share[t, j] * y[pair_slot[t * top + j]] (+ gate[t] * shared_out[t]); ``share`` None: plain sum."""
+def _identity(identity, out, top: int):
+    """(ids, h, h's row stride, experts) of moe_combine's ``identity``."""
+    if identity is None:
+        return None, None, 0, 0
+    ids, h, experts = identity
+    _need_cuda(ids, h)
+    assert ids.dtype == torch.int32 and ids.is_contiguous() and tuple(ids.shape) == (out.shape[0], top)
+    assert h.shape == out.shape and h.dtype == out.dtype and h.stride(1) == 1
+    return _ptr(ids), _ptr(h), h.stride(0), int(experts)
+
+
+def moe_combine_sorted(out, y, pair_slot, share, top: int, shared_out=None, gate=None, identity=None) -> None:
+    """out[t] = sum_j share[t, j] * y[pair_slot[t * top + j]] (+ gate[t] * shared_out[t]); ``share`` None: plain sum.
+    ``identity`` = (ids, h, experts): a pair whose id is ``experts`` or more adds share[t, j] * h[t] instead."""
     _need_cuda(out, y, pair_slot, share, shared_out, gate)
+    ids_p, h_p, h_stride, experts = _identity(identity, out, top)
     T, W = out.shape
     assert y.is_contiguous() and y.shape[1] == W and out.is_contiguous()
     assert share is None or (share.dtype == torch.float32 and share.is_contiguous() and share.numel() == T * top)
     assert pair_slot.dtype == torch.int32 and pair_slot.numel() >= T * top
     assert shared_out is None or (shared_out.dtype == out.dtype and shared_out.is_contiguous() and shared_out.shape == out.shape)
     _check(core().le_moe_combine_sorted(_ptr(out), dtype_code(out.dtype), _ptr(y), dtype_code(y.dtype), _ptr(pair_slot),
-                                        _ptr(share), _ptr(shared_out), _ptr(gate), T, W, top, _stream()),
+                                        _ptr(share), _ptr(shared_out), _ptr(gate), ids_p, h_p, h_stride, experts, T, W, top,
+                                        _stream()),
            "le_moe_combine_sorted")
 
 
@@ -1194,7 +1256,8 @@ def moe_grouped(out, a, w, slot_pair, tiles, meta, max_tiles: int, src_div: int,
     src_div of ``a`` (``src_div`` 0: row slot).  Output row: the slot, or with
     ``scatter`` the pair, times ``pair_weight[pair]`` where given (in the
     gated form the weight multiplies both products before the activation: the
-    weight on the expert's input).  bfloat16
+    weight on the expert's input).  Without a gate the kind ACT_RELU_SQUARED
+    puts that activation on the product.  bfloat16
     with rows in 16-byte pieces: tensor cores (``wide``: the tiles moe_group
     made are the wide ones); else the FP32 pipes."""
     _need_cuda(out, a, w, slot_pair, tiles, meta, pair_weight)
@@ -1210,13 +1273,16 @@ def moe_grouped(out, a, w, slot_pair, tiles, meta, max_tiles: int, src_div: int,
                                  float(activation[2]), _stream()), "le_moe_grouped")
 
 
-def moe_combine(out, y, top: int, shared_out=None, gate=None) -> None:
-    """out[t] = sum_j y[t * top + j] (+ gate[t] * shared_out[t]); ``y`` float32 [T * top, W]."""
-    _need_cuda(out, y, shared_out, gate)
+def moe_combine(out, y, top: int, shared_out=None, gate=None, identity=None, share=None) -> None:
+    """out[t] = sum_j y[t * top + j] (+ gate[t] * shared_out[t]); ``y`` float32 [T * top, W].
+    ``identity``: as moe_combine_sorted, with the pairs' weights ``share`` (None: 1)."""
+    _need_cuda(out, y, shared_out, gate, share)
+    ids_p, h_p, h_stride, experts = _identity(identity, out, top)
     T, W = out.shape
     assert y.dtype == torch.float32 and y.is_contiguous() and tuple(y.shape) == (T * top, W) and out.is_contiguous()
     assert shared_out is None or (shared_out.dtype == out.dtype and shared_out.is_contiguous() and shared_out.shape == out.shape)
-    _check(core().le_moe_combine(_ptr(out), dtype_code(out.dtype), _ptr(y), _ptr(shared_out), _ptr(gate), T, W, top, _stream()),
+    _check(core().le_moe_combine(_ptr(out), dtype_code(out.dtype), _ptr(y), _ptr(shared_out), _ptr(gate), ids_p, _ptr(share),
+                                 h_p, h_stride, experts, T, W, top, _stream()),
            "le_moe_combine")
 
 
@@ -1302,31 +1368,41 @@ def head_norm_gate(out, o, gate, weight, eps, heads, vdim, sigmoid: bool = False
 
 # -------------------------------------------------------------------------- rotary pairs with a norm per head
 def rope_norm_store(rows, k_cache, v_cache, rates, positions, request_of_token, block_table, heads, kv_heads, head_dim,
-                    rot_col, rot, unit_eps, norm_dim, page_size, write_kv, values_are_keys, status) -> None:
+                    rot_col, rot, unit_eps, norm_dim, page_size, write_kv, values_are_keys, status, w_q=None, w_k=None,
+                    temperature=None, store_values: bool = False) -> None:
     """Rows hold query heads, then key heads, ``head_dim`` entries each.  The
     entries (rot_col + 2i, rot_col + 2i + 1) below rot_col + ``rot`` of every
     head turn by position * rates[i]; with ``unit_eps`` not None the head is
     then divided by sqrt(mean over its first ``norm_dim`` entries of x^2 +
     unit_eps).  Queries are rewritten in place, keys go to ``k_cache``, and
     ``v_cache`` receives the keys as they were projected when
-    ``values_are_keys``.  ``write_kv`` False: the queries only."""
-    _need_cuda(rows, k_cache, v_cache, rates, positions, block_table)
+    ``values_are_keys``.  ``write_kv`` False: the queries only.  ``w_q`` /
+    ``w_k`` (float32 [head_dim] or None): what the result is multiplied by in
+    every head.  ``temperature`` = (coef, every): queries at position p times
+    1 + coef * ln(floor((p + 1) / every) + 1).  ``store_values``: value heads
+    lie behind the keys and go to ``v_cache`` as they are."""
+    _need_cuda(rows, k_cache, v_cache, rates, positions, block_table, w_q, w_k)
     T = rows.shape[0]
-    assert rows.stride(1) == 1 and rows.shape[1] >= (heads + (kv_heads if write_kv else 0)) * head_dim
-    assert rates.dtype == torch.float32 and rates.is_contiguous() and rates.numel() >= rot // 2
+    assert rows.stride(1) == 1
+    assert rows.shape[1] >= (heads + (kv_heads * (2 if store_values else 1) if write_kv else 0)) * head_dim
+    assert rot == 0 or (rates.dtype == torch.float32 and rates.is_contiguous() and rates.numel() >= rot // 2)
+    for w in (w_q, w_k):
+        assert w is None or (w.dtype == torch.float32 and w.is_contiguous() and w.numel() == head_dim)
+    coef, every = temperature if temperature is not None else (0.0, 0)
     pages = 0
     if write_kv:
         assert k_cache.dtype == rows.dtype and k_cache.is_contiguous()
         assert tuple(k_cache.shape[1:]) == (kv_heads, page_size, head_dim)
-        assert not values_are_keys or (v_cache.shape == k_cache.shape and v_cache.is_contiguous())
+        assert not (values_are_keys or store_values) or (v_cache.shape == k_cache.shape and v_cache.is_contiguous())
         pages = k_cache.shape[0]
     _check(core().le_rope_norm_store(_ptr(rows), rows.stride(0), dtype_code(rows.dtype), _ptr(k_cache) if write_kv else None,
-                                     _ptr(v_cache) if write_kv and values_are_keys else None, _ptr(rates), _ptr(positions),
+                                     _ptr(v_cache) if write_kv and (values_are_keys or store_values) else None, _ptr(rates),
+                                     _ptr(positions),
                                      _ptr(request_of_token), _ptr(block_table), block_table.shape[1], T, heads, kv_heads,
                                      head_dim, rot_col, rot, 0 if unit_eps is None else 1,
                                      0.0 if unit_eps is None else float(unit_eps), norm_dim, page_size, pages,
-                                     1 if write_kv else 0, 1 if values_are_keys else 0, _ptr(status), _stream()),
-           "le_rope_norm_store")
+                                     1 if write_kv else 0, 1 if values_are_keys else 0, _ptr(w_q), _ptr(w_k), float(coef),
+                                     int(every), 1 if store_values else 0, _ptr(status), _stream()), "le_rope_norm_store")
 
 
 def latent_rope_store(src, col, rank, rot, padded, weight, eps, rates, cache, positions, request_of_token, block_table,
@@ -1368,13 +1444,16 @@ def _addend(t, rows: int, width: int):
     return t.data_ptr(), dtype_code(t.dtype), 1, 0
 
 
-def rmsnorm_pair(out1, out2, resid, w1, w2, eps, addend=None, addend_weight=None, addend_eps: float = 0.0, rows=None) -> None:
+def rmsnorm_pair(out1, out2, resid, w1, w2, eps, addend=None, addend_weight=None, addend_eps: float = 0.0, rows=None,
+                 addend2=None) -> None:
     """``addend`` first enters the 32-bit stream ``resid`` [T, W]: plainly, or,
     with ``addend_weight`` [W], as addend / sqrt(mean(addend^2) + addend_eps) *
-    addend_weight.  Then out1 = rmsnorm(resid) * w1 and (``out2`` given) out2 =
+    addend_weight; ``addend2`` beside a plain addend: resid += addend +
+    addend2.  Then out1 = rmsnorm(resid) * w1 and (``out2`` given) out2 =
     rmsnorm(resid) * w2.  ``out1`` None: only the addend enters.  With ``rows``
     only those rows are normed and ``resid`` is left as it is."""
-    _need_cuda(out1, out2, resid, w1, w2, addend, addend_weight, rows)
+    _need_cuda(out1, out2, resid, w1, w2, addend, addend2, addend_weight, rows)
+    assert addend2 is None or (addend is not None and addend_weight is None)
     T, W = resid.shape
     assert resid.dtype == torch.float32 and resid.is_contiguous()
     n = T if rows is None else (out1.shape[0] if out1 is not None else 0)
@@ -1382,9 +1461,10 @@ def rmsnorm_pair(out1, out2, resid, w1, w2, eps, addend=None, addend_weight=None
         if o is not None:
             assert o.is_contiguous() and o.shape == (n, W) and w.dtype == torch.float32 and w.numel() == W
     ptr, code, parts, stride = _addend(addend, T, W)
+    ptr2, code2, parts2, stride2 = _addend(addend2, T, W)
     out_code = dtype_code(out1.dtype) if out1 is not None else F32
     _check(core().le_rmsnorm_pair(_ptr(out1), _ptr(out2), out_code, _ptr(resid), ptr, code, parts, stride,
-                                  _ptr(addend_weight), float(addend_eps), _ptr(w1), _ptr(w2), float(eps), _ptr(rows), n, W,
+                                  ptr2, code2, parts2, stride2, _ptr(addend_weight), float(addend_eps), _ptr(w1), _ptr(w2), float(eps), _ptr(rows), n, W,
                                   _stream()), "le_rmsnorm_pair")
 
 
@@ -1468,6 +1548,78 @@ def ssm_scan(out, x, bc, b_col: int, c_col: int, dt, z, dt_bias, a_log, d_skip, 
                               dtype_code(x.dtype), _ptr(dt_bias), _ptr(a_log), _ptr(d_skip), _ptr(state), state.shape[0],
                               _ptr(state_slots), _ptr(cu_q), int(num_requests), T, rows, int(n_state), int(rows_per_head),
                               int(rows_per_group), 1 if per_row else 0, float(out_scale), _stream()), "le_ssm_scan")
+
+
+LIGHTNING_MAX_DIM = 512
+LIGHTNING_CHUNK_MAX_DIM = 128      # of the form over chunks
+_lightning_sizes: dict[str, int] = {}
+
+
+def lightning_segment() -> int:
+    """Tokens per segment of lightning_chunks()."""
+    if "segment" not in _lightning_sizes:
+        _lightning_sizes["segment"] = int(core().le_lightning_segment())
+        _lightning_sizes["chunk"] = int(core().le_lightning_chunk())
+    return _lightning_sizes["segment"]
+
+
+def lightning_tables(decay, device):
+    """What the two forms of lightning attention need of the decays (one
+    64-bit number per head): (their high and low float32 parts [2, heads],
+    their powers 0 .. chunk as float32 [heads, chunk + 1], the decays as float64)."""
+    lightning_segment()
+    d = torch.as_tensor([float(x) for x in decay], dtype=torch.float64)
+    high = d.to(torch.float32)
+    parts = torch.stack([high, (d - high.to(torch.float64)).to(torch.float32)])
+    powers = d[:, None] ** torch.arange(_lightning_sizes["chunk"] + 1, dtype=torch.float64)[None, :]
+    return (parts.to(device).contiguous(), powers.to(torch.float32).to(device).contiguous(), d.to(device).contiguous())
+
+
+def _lightning_checks(out, rows, state, heads, dim, vdim):
+    T = out.shape[0]
+    assert out.dtype == torch.float32 and out.stride(1) == 1 and rows.stride(1) == 1 and rows.shape[0] == T
+    assert out.shape[1] == heads * vdim and state.dtype == torch.float32 and state.is_contiguous()
+    assert tuple(state.shape[1:]) == (heads, vdim, dim)
+
+
+def lightning_scan(out, rows, q_col: int, k_col: int, v_col: int, decay_parts, state, state_slots, cu_q, num_requests: int,
+                   heads: int, dim: int, vdim: int, activated: bool = False, requests=None, single: bool = False) -> None:
+    """Lightning attention token by token, from each request's state row
+    (``state`` float32 [rows, heads, vdim, dim]) and back into it: S <- decay S
+    + k v^T, ``out`` (float32 [T, heads * vdim]) = S^T q.  ``rows``: q [heads,
+    dim] at column ``q_col``, k at ``k_col``, v [heads, vdim] at ``v_col``, each
+    before its silu (``activated``: after it).  ``requests``: indices of the
+    ``num_requests`` requests to run (None: all, in order); ``single``: each
+    brings one token."""
+    _need_cuda(out, rows, decay_parts, state, state_slots, cu_q, requests)
+    _lightning_checks(out, rows, state, heads, dim, vdim)
+    assert decay_parts.dtype == torch.float32 and tuple(decay_parts.shape) == (2, heads) and decay_parts.is_contiguous()
+    _check(core().le_lightning_scan(_ptr(out), out.stride(0), _ptr(rows), rows.stride(0), q_col, k_col, v_col,
+                                    dtype_code(rows.dtype), 1 if activated else 0, _ptr(decay_parts), _ptr(state),
+                                    state.shape[0], _ptr(state_slots), _ptr(cu_q), _ptr(requests), num_requests, heads, dim,
+                                    vdim, 1 if single else 0, _stream()), "le_lightning_scan")
+
+
+def lightning_chunks(out, rows, q_col: int, k_col: int, v_col: int, powers, decay, state, scratch, state_slots, cu_q,
+                     tile_request, tile_q0, num_segments: int, heads: int, dim: int, vdim: int) -> None:
+    """The same over chunks on the tensor cores, for the requests whose
+    segments (lightning_segment() tokens each, a request's one after the
+    other) the first ``num_segments`` entries of the tile lists name.  ``rows``
+    bfloat16, after silu.  ``powers``, ``decay``: see lightning_tables().
+    ``scratch``: float32 [num_segments, heads, vdim, dim] where a request has
+    several segments, else None."""
+    _need_cuda(out, rows, powers, decay, state, scratch, state_slots, cu_q, tile_request, tile_q0)
+    _lightning_checks(out, rows, state, heads, dim, vdim)
+    lightning_segment()
+    assert rows.dtype == torch.bfloat16 and dim <= LIGHTNING_CHUNK_MAX_DIM
+    assert powers.dtype == torch.float32 and tuple(powers.shape) == (heads, _lightning_sizes["chunk"] + 1)
+    assert powers.is_contiguous() and decay.dtype == torch.float64 and decay.numel() == heads
+    assert scratch is None or (scratch.dtype == torch.float32 and scratch.is_contiguous()
+                               and scratch.numel() >= num_segments * heads * vdim * dim)
+    _check(core().le_lightning_chunks(_ptr(out), out.stride(0), _ptr(rows), rows.stride(0), q_col, k_col, v_col, _ptr(powers),
+                                      _ptr(decay), _ptr(state), state.shape[0], _ptr(scratch), _ptr(state_slots), _ptr(cu_q),
+                                      _ptr(tile_request), _ptr(tile_q0), num_segments, heads, dim, vdim, _stream()),
+           "le_lightning_chunks", launches=1 if scratch is None else 3)
 
 
 def mlstm_rows(dim: int, vdim: int) -> int:

@@ -29,6 +29,8 @@ What a description may choose beyond the reference's Llama layer:
   visible to every later query, with their true positions; their pages are
   never given back;
 * ``softcap`` c: a score s (after the scale) becomes c * tanh(s / c);
+* ``sink_name``: a tensor [nh]; the softmax's denominator has one more term
+  exp(sink_h) (it has no key and no value, and neither scale nor cap);
 * ``v_name`` None: there is no value projection, the values are the keys as
   projected (before any position encoding or norm of the keys); the position
   encoding then fills the value pool itself (it is built with
@@ -84,7 +86,7 @@ class AttentionMixer(Mixer):
                  q_name: str, k_name: str, v_name: str | None, o_name: str, window: int | None = None,
                  chunk: int | None = None, scale: float | None = None, value_dim: int | None = None,
                  head_scale_name: str | None = None, gate_name: str | None = None, gate_per_entry: bool = False,
-                 keep_first: int = 0, softcap: float | None = None):
+                 keep_first: int = 0, softcap: float | None = None, sink_name: str | None = None):
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} heads do not divide into {num_kv_heads} groups")
         self.qk_dim = int(head_dim)
@@ -120,13 +122,13 @@ class AttentionMixer(Mixer):
             raise ValueError(f"a cap on the scores must be positive, got {softcap}")
         self.scale = float(scale) if scale is not None else 1.0 / (self.qk_dim ** 0.5)
         self.names = (q_name, k_name, v_name, o_name)
-        self.head_scale_name, self.gate_name = head_scale_name, gate_name
+        self.head_scale_name, self.gate_name, self.sink_name = head_scale_name, gate_name, sink_name
         self.gate_per_entry = bool(gate_per_entry) and bool(gate_name)
         # rows of the projection stay 16-byte multiples
         self.gate_rows = 0
         if gate_name:
             self.gate_rows = self.num_heads * self.head_dim if self.gate_per_entry else (self.num_heads + 7) // 8 * 8
-        self.w_qkv = self.w_o = self.head_scale = None
+        self.w_qkv = self.w_o = self.head_scale = self.sink = None
         self.head_scale_positive = True
         self.runtime = None
 
@@ -151,6 +153,8 @@ class AttentionMixer(Mixer):
             decls.insert(2, TensorDecl(v, (nkv * self.value_dim, H)))
         if self.head_scale_name:
             decls.append(TensorDecl(self.head_scale_name, (nh,), role="vector", init="ones_jitter"))
+        if self.sink_name:
+            decls.append(TensorDecl(self.sink_name, (nh,), role="vector", init="zeros"))
         if self.gate_name:
             decls.append(TensorDecl(self.gate_name, (nh * self.value_dim if self.gate_per_entry else nh, H)))
         return decls + (self.position.tensors() if self.position is not None else [])
@@ -172,6 +176,7 @@ class AttentionMixer(Mixer):
         self.runtime = runtime
         head_scale = get(self.head_scale_name).to(torch.float32) if self.head_scale_name else None
         self.kernel_scale, self.head_scale, self.head_scale_positive = signed_scale(self.scale, head_scale, nh, runtime.device)
+        self.sink = get(self.sink_name).contiguous() if self.sink_name else None
         if self.position is not None:
             self.position.bind(get, runtime)
         attention_kernels.prepare(self.head_dim)
@@ -209,7 +214,7 @@ class AttentionMixer(Mixer):
                              ctx.block_tables[cache.kv.group], nkv, hd, cache.kv.page_size, ctx.status)
         attn = ws.get("attn", (T, nh * hd), rt.dtype)
         attention_kernels.run(attn, qkv, ctx, cache.kv, nh, nkv, hd, self.reach, self.kernel_scale, self.head_scale,
-                              self.head_scale_positive, keep_first=self.keep_first, softcap=self.softcap)
+                              self.head_scale_positive, keep_first=self.keep_first, softcap=self.softcap, sink=self.sink)
         if self.gate_per_entry:
             target = out if out is not None else attn
             ops.sigmoid_gate(target, attn, qkv[:, width:width + nh * hd], scale)

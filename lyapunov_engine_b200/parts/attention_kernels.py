@@ -135,7 +135,7 @@ def decode_variant(fill: int, num_heads: int, num_kv_heads: int, head_dim: int, 
 
 def run(out, qkv, ctx, kv, num_heads, num_kv_heads, head_dim, reach, scale, head_scale=None,
         head_scale_positive: bool = True, max_splits: int = DECODE_MAX_SPLITS, keep_first: int = 0,
-        softcap: float = 0.0) -> None:
+        softcap: float = 0.0, sink=None) -> None:
     """``reach``: which keys a query sees (ops.reach_code); ``head_scale``: one
     more factor per query head on its scores (float32 [num_heads]) or None.
     The tcgen05 kernel folds that factor into its exponent's scale and so takes
@@ -143,7 +143,9 @@ def run(out, qkv, ctx, kv, num_heads, num_kv_heads, head_dim, reach, scale, head
     ``keep_first`` n: the keys at positions below n stay visible behind a
     window; ``softcap`` c > 0: a score s becomes c * tanh(s / c).  The tcgen05
     kernel has neither (its keys are one unbroken run and its scores stay raw
-    products until the exponent): prompts of such a mixer take the mma.sync kernel."""
+    products until the exponent): prompts of such a mixer take the mma.sync kernel.
+    ``sink`` (float32 [num_heads] or None): one more term exp(sink) per head in
+    the softmax's denominator; every kernel has it."""
     table = ctx.block_tables[kv.group]
     window = reach
     if out.dtype == torch.bfloat16 and ops.attention_mma_available(head_dim):
@@ -153,11 +155,12 @@ def run(out, qkv, ctx, kv, num_heads, num_kv_heads, head_dim, reach, scale, head
                     and ops.attention_tc_available(head_dim, kv.page_size)):
                 ops.attention_prefill_tc_bf16(out, qkv, qkv.stride(0), kv.k, kv.v, table, ctx.cu_q, ctx.ctx_before, req, q0,
                                               n_multi, num_heads, num_kv_heads, head_dim, kv.page_size, window, scale,
-                                              ctx.status, head_scale=head_scale)
+                                              ctx.status, head_scale=head_scale, sink=sink)
             else:
                 ops.attention_prefill_bf16(out, qkv, qkv.stride(0), kv.k, kv.v, table, ctx.cu_q, ctx.ctx_before, req, q0,
                                            n_multi, num_heads, num_kv_heads, head_dim, kv.page_size, window, scale,
-                                           ctx.status, head_scale=head_scale, keep_first=keep_first, softcap=softcap)
+                                           ctx.status, head_scale=head_scale, keep_first=keep_first, softcap=softcap,
+                                           sink=sink)
         if ctx.num_decode:
             real = min(ctx.decode_fill, ctx.num_decode) if SPLITS_BY_FILL else 0     # dummy requests finish at once
             splits = min(max_splits, decode_splits(real or ctx.num_decode, num_heads, num_kv_heads,
@@ -169,9 +172,9 @@ def run(out, qkv, ctx, kv, num_heads, num_kv_heads, head_dim, reach, scale, head
             ops.attention_decode_bf16(out, scratch, qkv, qkv.stride(0), kv.k, kv.v, table, ctx.cu_q, ctx.ctx_before,
                                       requests, ctx.num_decode, num_heads, num_kv_heads, head_dim, kv.page_size,
                                       window, scale, splits, ctx.status, small_form=small, head_scale=head_scale,
-                                      keep_first=keep_first, softcap=softcap)
+                                      keep_first=keep_first, softcap=softcap, sink=sink)
         return
     req, q0, n_tiles, _ = ctx.tiles[GENERIC_TILE]
     ops.attention_generic(out, qkv, qkv.stride(0), kv.k, kv.v, table, ctx.cu_q, ctx.ctx_before, req, q0, n_tiles,
                           num_heads, num_kv_heads, head_dim, kv.page_size, window, scale, ctx.status, head_scale=head_scale,
-                          keep_first=keep_first, softcap=softcap)
+                          keep_first=keep_first, softcap=softcap, sink=sink)

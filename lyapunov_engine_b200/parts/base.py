@@ -258,6 +258,17 @@ class ScaledAddend:
         self.weight = weight
 
 
+class SecondAddend:
+    """How a pending output enters the stream when another sub-layer's output
+    enters beside it: resid += pending + other (``other`` as a pending output:
+    a tensor or float32 partial sums); the norm that reads the stream adds both
+    in its own kernel."""
+    __slots__ = ("other",)
+
+    def __init__(self, other):
+        self.other = other
+
+
 class Block(Part):
     mixer: Mixer
 
@@ -283,7 +294,8 @@ class ResidualStream:
     a ``StreamLink`` whose ``mix`` [copies, copies] and ``post`` [copies]
     give copy j <- sum_s mix[s, j] copy_s + post[j] * pending; a
     ``NormedAddend``: resid += pending normed with a weight; a
-    ``ScaledAddend``: resid += weight * pending."""
+    ``ScaledAddend``: resid += weight * pending; a ``SecondAddend``: resid +=
+    pending + its ``other``."""
     __slots__ = ("resid", "pending", "update", "copies")
 
     def __init__(self, resid, pending=None):

@@ -21,7 +21,7 @@ from __future__ import annotations
 
 from .. import ops
 from .base import (BLOCKS, FEED_FORWARDS, INPUT_FILTERS, MIXERS, NORMS, STREAM_INPUTS, Block, PartSpec, ScaledAddend,
-                   TensorDecl, register_block)
+                   SecondAddend, TensorDecl, register_block)
 
 
 @register_block("prenorm")
@@ -111,11 +111,18 @@ class ParallelBlock(Block):
     (one kernel makes both norms; one adds both outputs, and the feed-forward's
     output bias, in 32 bits).  ``after``: a stream input that runs on the new
     h, after the sub-layers (an embedding per token behind a gate, say); what
-    it leaves pending enters in the next norm's kernel."""
+    it leaves pending enters in the next norm's kernel.
+
+    ``shared_norm``: there is one norm and both sub-layers read its output,
+        n = norm1(h);  h = h + (mixer(n) + feed_forward(n));
+    both outputs are left pending, and the next norm's kernel adds them."""
 
     def __init__(self, mixer: PartSpec, feed_forward: PartSpec | None, mixer_norm: PartSpec,
-                 feed_forward_norm: PartSpec | None, after: PartSpec | None = None):
-        if (feed_forward is None) != (feed_forward_norm is None):
+                 feed_forward_norm: PartSpec | None = None, after: PartSpec | None = None, shared_norm: bool = False):
+        self.shared_norm = bool(shared_norm)
+        if self.shared_norm and (feed_forward_norm is not None or after is not None):
+            raise ValueError("sub-layers that share one norm have no second one, and nothing runs after them")
+        if not self.shared_norm and (feed_forward is None) != (feed_forward_norm is None):
             raise ValueError("a block has a feed-forward and its norm, or neither")
         self.mixer = MIXERS.build(mixer)
         self.feed_forward = FEED_FORWARDS.build(feed_forward) if feed_forward is not None else None
@@ -137,7 +144,16 @@ class ParallelBlock(Block):
         for p in self.parts():
             p.bind(get, runtime)
 
+    def _forward_shared(self, stream, ctx, cache) -> None:
+        n = self.mixer_norm.apply_stream(stream, workspace=ctx.workspace)
+        stream.pending = self.mixer.forward(n, ctx, cache)
+        if self.feed_forward is not None:
+            stream.update = SecondAddend(self.feed_forward.forward(n, ctx))
+
     def forward(self, stream, ctx, cache) -> None:
+        if self.shared_norm:
+            self._forward_shared(stream, ctx, cache)
+            return
         n1, n2 = self.mixer_norm.apply_pair(stream, self.feed_forward_norm, workspace=ctx.workspace)
         a = self.mixer.forward(n1, ctx, cache)
         f = bias = None

@@ -1,4 +1,8 @@
-"""Gated feed-forward: down(act(gate(x), up(x))).
+"""Feed-forward layers.
+
+"relu_squared", without a gate: down(max(up(x), 0)^2).
+
+Gated: down(act(gate(x), up(x))).
 
 "gated_silu" (SwiGLU): act(g, u) = silu(g) * u.  "gated_relu": act(g, u) =
 max(g, 0) * u.  "gated_clamped": with a limit
@@ -81,6 +85,42 @@ class GatedFeedForward(FeedForward):
         ops.linear(out, act, self.w_down, ctx.status)
         if self.output_bias is not None:
             raise NotImplementedError("a feed-forward with an output bias is added to the residual stream by its block")
+        return out
+
+
+@register_feed_forward("relu_squared")
+class PlainFeedForward(FeedForward):
+    """down(act(up x)) without a gate and without biases; the activation is
+    taken in 32 bits in the first product's epilogue and rounded once."""
+    activation = ops.ACT_RELU_SQUARED
+
+    def __init__(self, hidden_size: int, intermediate_size: int, up_name: str, down_name: str):
+        self.hidden_size, self.intermediate_size = int(hidden_size), int(intermediate_size)
+        self.names = (up_name, down_name)
+        self.w_up = self.w_down = None
+        self.runtime = None
+
+    def tensors(self):
+        u, d = self.names
+        return [TensorDecl(u, (self.intermediate_size, self.hidden_size)), TensorDecl(d, (self.hidden_size, self.intermediate_size))]
+
+    def bind(self, get, runtime):
+        self.w_up, self.w_down = (get(n) for n in self.names)
+        self.runtime = runtime
+
+    def _activated(self, x, ctx, key):
+        act = ctx.workspace.get(key, (x.shape[0], self.intermediate_size), self.runtime.dtype)
+        ops.activated_linear(act, x, self.w_up, self.activation, ctx.status)
+        return act
+
+    def forward(self, x, ctx):
+        return ops.linear_for_residual(self._activated(x, ctx, "ffn_act"), self.w_down, ctx.workspace, "ffn_out", ctx.status)
+
+    def forward_plain(self, x, ctx, key: str = "ffn_plain"):
+        """The same as one tensor [T, H] in the activations' type, in buffers
+        of its own (see GatedFeedForward.forward_plain)."""
+        out = ctx.workspace.get(key, (x.shape[0], self.hidden_size), self.runtime.dtype)
+        ops.linear(out, self._activated(x, ctx, key + "_act"), self.w_down, ctx.status)
         return out
 
 

@@ -9,7 +9,7 @@ are bare parameters of the decoder layer (python/lyapunov_engine/models/llama.py
 from __future__ import annotations
 
 from .. import ops
-from .base import Norm, NormedAddend, ScaledAddend, TensorDecl, register_norm
+from .base import Norm, NormedAddend, ScaledAddend, SecondAddend, TensorDecl, register_norm
 
 
 @register_norm("rmsnorm")
@@ -20,7 +20,7 @@ class RMSNorm(Norm):
     (made once at load, in 32 bits).
 
     It also reads a stream whose pending output enters normed
-    (``NormedAddend``), and two such norms of the same stream run as one kernel
+    (``NormedAddend``) or beside another's (``SecondAddend``), and two such norms of the same stream run as one kernel
     (``apply_pair``: sub-layers that read the stream side by side)."""
 
     def __init__(self, hidden_size: int, eps: float, weight_name: str, groups: int = 1, offset: float = 0.0):
@@ -59,7 +59,7 @@ class RMSNorm(Norm):
             if rows is None:
                 stream.pending = stream.update = None
             return out
-        if not isinstance(stream.update, NormedAddend):
+        if not isinstance(stream.update, (NormedAddend, SecondAddend)):
             return super().apply_stream(stream, read, rows, workspace, key)
         return self.apply_pair(stream, None, rows=rows, workspace=workspace, keys=(key, None))[0]
 
@@ -70,15 +70,17 @@ class RMSNorm(Norm):
         if stream.copies != 1 or self.groups != 1 or (other is not None and (other.groups != 1 or other.eps != self.eps)):
             raise ValueError("norms that run as a pair read one copy of the stream, whole rows, with one eps")
         update = stream.update
-        if update is not None and not isinstance(update, NormedAddend):
+        second = update.other if isinstance(update, SecondAddend) else None
+        normed = update if isinstance(update, NormedAddend) else None
+        if update is not None and second is None and normed is None:
             raise ValueError(f"{type(self).__name__} cannot apply a pending {type(update).__name__}")
         n = stream.resid.shape[0] if rows is None else rows.shape[0]
         ws = workspace or self.runtime.workspace
         out1 = ws.get(keys[0], (n, self.hidden_size), self.runtime.dtype)
         out2 = ws.get(keys[1], (n, self.hidden_size), self.runtime.dtype) if other is not None else None
         ops.rmsnorm_pair(out1, out2, stream.resid, self.weight, other.weight if other is not None else None, self.eps,
-                         addend=stream.pending, addend_weight=update.weight if update is not None else None,
-                         addend_eps=update.eps if update is not None else 0.0, rows=rows)
+                         addend=stream.pending, addend_weight=normed.weight if normed is not None else None,
+                         addend_eps=normed.eps if normed is not None else 0.0, rows=rows, addend2=second)
         if rows is None:
             stream.pending = stream.update = None
         return out1, out2

@@ -147,6 +147,53 @@ class RotaryPairsEncoding(PositionEncoding):
                          ctx.block_tables[kv.group], nkv, hd, kv.page_size, ctx.status)
 
 
+@register_position_encoding("head_norm")
+class HeadNormEncoding(PositionEncoding):
+    """No rotation: every head of queries and keys is divided by
+    sqrt(mean(head^2) + eps) and multiplied by a weight of the head's size that
+    all heads share (``q_norm_name``, ``k_norm_name``), and queries may have a
+    temperature that grows with their position p (``temperature`` = {"coef",
+    "every"}): q times 1 + coef * ln(floor((p + 1) / every) + 1).  One kernel
+    with the write of keys and values to their pages; 32-bit, rounded once.
+    ``head_dim`` is the real size of queries and keys; the heads the kernels
+    see may be padded with zeros behind it."""
+    padded_heads_ok = True
+    takes_gate_columns = True
+
+    def __init__(self, head_dim: int, eps: float, q_norm_name: str, k_norm_name: str, temperature: dict | None = None):
+        self.head_dim, self.eps = int(head_dim), float(eps)
+        self.names = (q_norm_name, k_norm_name)
+        self.temperature = None
+        if temperature is not None:
+            self.temperature = (float(temperature["coef"]), int(temperature["every"]))
+            if self.temperature[1] < 1:
+                raise ValueError(f"a query temperature steps every 1 or more positions, got {temperature['every']}")
+        self.padded = self.head_dim
+        self.w_q = self.w_k = None
+
+    def set_geometry(self, padded_head_dim: int) -> None:
+        self.padded = int(padded_head_dim)
+
+    def tensors(self):
+        from .base import TensorDecl
+        return [TensorDecl(name, (self.head_dim,), role="vector", init="ones_jitter") for name in self.names]
+
+    def bind(self, get, runtime):
+        def padded(t):
+            out = torch.zeros(self.padded, dtype=torch.float32, device=t.device)
+            out[:self.head_dim] = t
+            return out
+        self.w_q, self.w_k = (padded(get(name)) for name in self.names)
+
+    def encode_and_store(self, qkv, geometry, ctx, kv, write: bool) -> None:
+        nh, nkv, hd = geometry
+        write = write and kv is not None
+        ops.rope_norm_store(qkv, kv.k if write else None, kv.v if write else None, None, ctx.positions, ctx.request_of_token,
+                            ctx.block_tables[kv.group] if kv is not None else ctx.block_tables[0], nh, nkv, hd, 0, 0, self.eps,
+                            self.head_dim, kv.page_size if kv is not None else 1, write, False, ctx.status, w_q=self.w_q,
+                            w_k=self.w_k, temperature=self.temperature, store_values=True)
+
+
 def ramped_rates(rot: int, base: float, scaling: dict | None) -> tuple[torch.Tensor, float]:
     """(rates f_i for i < rot / 2, the factor on cosines and sines).  Plain:
     f_i = base^(-2i / rot) and 1.  With ``scaling`` = {factor, original, fast,

@@ -52,6 +52,7 @@ def _register_builtin() -> None:
     from .models.sulepel import sulepel_spec
     from .models.zepilix import zepilix_spec
     from .models.ribozen import ribozen_spec
+    from .models.zuzenex import zuzenex_spec
 
     register_architecture("LlamaForCausalLM", llama_spec)
     register_architecture("llama", llama_spec)
@@ -59,6 +60,7 @@ def _register_builtin() -> None:
     register_architecture("Kaditar", kaditar_spec)
     register_architecture("Zepilix", zepilix_spec)
     register_architecture("Ribozen", ribozen_spec)
+    register_architecture("Zuzenex", zuzenex_spec)
 
 
 _register_builtin()
