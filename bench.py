@@ -1925,6 +1925,335 @@ def run_ribozen(args):
     return 0
 
 
+# ---------------------------------------------------------------------------------------------- Zuzenex
+ZUZENEX_EXPERTS, ZUZENEX_IDENTITY, ZUZENEX_TOP = 8, 2, 2
+
+
+def zuzenex_config(llama: dict) -> dict:
+    """A Zuzenex model with the width, heads, head size, vocabulary and number of layers of the given Llama shapes:
+    three layers of lightning attention (heads of 128 x 128, their values as wide as the model), then one of attention,
+    and so on; every layer has eight routed experts and two identity experts (two per token) and a shared expert.  An
+    expert has two matrices where a gated one has three, so each is three eighths of the Llama feed-forward's size, as
+    many weights as the gated experts of a quarter that the other routed designs are measured with."""
+    nh, nkv, hd, W = llama["num_attention_heads"], llama["num_key_value_heads"], llama["head_dim"], llama["hidden_size"]
+    ff = llama["intermediate_size"] * 3 // 8
+    mlp = {"kind": "moe", "expert": {"ff": ff}, "shared": {"ff": ff},
+           "router": {"experts": ZUZENEX_EXPERTS, "identity": ZUZENEX_IDENTITY, "top": ZUZENEX_TOP}}
+    H = W // 128
+    memory = {"type": "lightning", "mlp": mlp,
+              "mixer": {"heads": H, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-1.0 - 9.0 * h / max(H - 1, 1)) for h in range(H)]}}
+    attn = {"type": "attention", "mlp": mlp,
+            "mixer": {"heads": nh, "kv_heads": nkv, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "q_temp": {"coef": 0.1, "every": 2048}}}
+    return {"architecture": "Zuzenex", "vocab": llama["vocab_size"], "width": W, "norm": {"eps": 1e-5},
+            "layers": [attn if i % 4 == 3 else memory for i in range(llama["num_hidden_layers"])]}
+
+
+def zuzenex_decode_bytes(cfg, batch, context):
+    """Bytes one decode step of a Zuzenex model must move: the bfloat16 weights it touches (of the routed experts
+    those that batch * top tokens can reach), each live request's states read and written (32-bit), and its keys and
+    values."""
+    W, V = cfg["width"], cfg["vocab"]
+    total = 2 * V * W + 4 * W
+    for layer in cfg["layers"]:
+        m, f = layer["mixer"], layer["mlp"]
+        F, r, S = f["expert"]["ff"], f["router"], f["shared"]["ff"]
+        total += 2 * 2 * W * (F * min(r["experts"], batch * r["top"]) + S) + 4 * (r["experts"] + r["identity"]) * W + 4 * W
+        H, d, e = m["heads"], m["dim"], m["vdim"]
+        if layer["type"] == "lightning":
+            total += 2 * ((2 * H * d + 2 * H * e) * W + W * H * e) + batch * 2 * 4 * H * d * e
+        else:
+            G = m["kv_heads"]
+            total += 2 * ((H * d + G * d + G * e) * W + W * H * e) + 2 * batch * context * G * (d + e)
+    return total
+
+
+def zuzenex_prefill_flops(cfg, tokens):
+    """Flops of the matrix products and the attentions, and of the recurrence as four per entry of the state and
+    token.  Of a token's choices all are counted as experts with a product."""
+    W, V = cfg["width"], cfg["vocab"]
+    flops = 2 * V * W
+    for layer in cfg["layers"]:
+        m, f = layer["mixer"], layer["mlp"]
+        F, r, S = f["expert"]["ff"], f["router"], f["shared"]["ff"]
+        flops += 2 * tokens * (2 * W * (r["top"] * F + S) + (r["experts"] + r["identity"]) * W)
+        H, d, e = m["heads"], m["dim"], m["vdim"]
+        if layer["type"] == "lightning":
+            flops += 2 * tokens * ((2 * H * d + 2 * H * e) * W + W * H * e) + 4 * tokens * H * d * e
+        else:
+            G = m["kv_heads"]
+            flops += 2 * tokens * ((H * d + G * d + G * e) * W + W * H * e) + H * (d + e) * tokens * (tokens + 1)
+    return flops
+
+
+def zuzenex_kernel_rows(pk, llama):
+    """Each kernel the design adds, alone, beside the like kernel of the closest existing path at like sizes:
+    microseconds per launch inside a captured graph over rotating tensors, the share of the measured copy bandwidth
+    that the bytes it must move make, and for products their share of the measured bfloat16 peak."""
+    import torch
+
+    from lyapunov_engine_b200 import ops
+    from lyapunov_engine_b200.engine.runtime import Workspace
+
+    dev = "cuda:0"
+    cfg = zuzenex_config(llama)
+    W, nh, nkv, hd = llama["hidden_size"], llama["num_attention_heads"], llama["num_key_value_heads"], llama["head_dim"]
+    page = BLOCK_SIZE
+    ws = Workspace(dev)
+    rows = []
+
+    def row(kernel, like, tokens, nbytes, launch, sets, flops=0):
+        us = graph_median_us(launch, sets)
+        entry = {"kernel": kernel, "like": like, "tokens": tokens, "us": round(us, 2), "gbs": round(nbytes / us / 1e3, 1),
+                 "hbm_frac": round(nbytes / us / 1e3 / pk["hbm_gbs"], 3)}
+        if flops:
+            entry["bf16_frac"] = round(flops / us / 1e6 / pk["bf16_tflops"], 3)
+        rows.append(entry)
+
+    bf = torch.bfloat16
+    status = ops.new_status(dev)
+    lm = cfg["layers"][0]["mixer"]
+    H, d, e = lm["heads"], lm["dim"], lm["vdim"]
+    parts, powers = ops.lightning_tables(lm["decay"], dev)
+    seg = ops.lightning_segment()
+    f = cfg["layers"][0]["mlp"]
+    F, E, I, top = f["expert"]["ff"], f["router"]["experts"], f["router"]["identity"], f["router"]["top"]
+    for T in (8, 64, 2048, 8192):
+        reqs = T if T <= 64 else 1
+        cu = torch.arange(reqs + 1, dtype=torch.int32, device=dev) if T <= 64 else torch.tensor([0, T], dtype=torch.int32, device=dev)
+        slots = torch.arange(reqs, dtype=torch.int32, device=dev)
+        sets = 4 if T <= 64 else 2
+        # the recurrence
+        width = 2 * H * d + 2 * H * e
+        proj = [torch.randn(T, width, device=dev).to(bf) for _ in range(2)]
+        o = torch.empty(T, H * e, device=dev)
+        states = [torch.zeros(reqs + 1, H, e, d, device=dev) for _ in range(sets)]
+        nbytes = reqs * 2 * 4 * H * d * e + T * ((2 * H * d + H * e) * 2 + H * e * 4)
+        like = f"matrix memory, {W // 256} heads of 128 x 256"
+        if T <= 64:
+            row(f"lightning, {H} heads of {d} x {e}, token by token, {reqs} requests", like, T, nbytes,
+                lambda i: ops.lightning_scan(o, proj[i % 2], 0, H * d, 2 * H * d, parts, states[i], slots, cu, reqs, H, d, e, single=True), sets)
+        else:
+            n = T // seg
+            tr, tq = torch.zeros(n, dtype=torch.int32, device=dev), torch.arange(0, T, seg, dtype=torch.int32, device=dev)
+            scratch = torch.empty(n, H, e, d, device=dev)
+            row(f"lightning, {H} heads of {d} x {e}, over chunks (sums, starts, outputs)", like, T, nbytes,
+                lambda i: ops.lightning_chunks(o, proj[i], 0, H * d, 2 * H * d, powers, states[i], scratch, slots, cu, tr, tq, n, H, d, e),
+                sets, flops=4 * T * H * d * e)
+        Hm, em = W // 256, 256
+        wm = (2 * Hm * 128 + 2 * Hm * em + 2 * Hm + 7) // 8 * 8
+        rows_m = torch.randn(T, wm, device=dev).to(bf)
+        om = torch.empty(T, Hm * em, device=dev)
+        states = [torch.zeros(reqs + 1, *ops.mlstm_state_shape(Hm, 128, em), device=dev) for _ in range(sets)]
+        zeros_m = torch.zeros(Hm, device=dev)
+        row(f"matrix memory, {Hm} heads of 128 x {em}, {reqs} request(s)", "", T, reqs * 2 * states[0][0].numel() * 4 + T * (wm * 2 + Hm * em * 4),
+            lambda i: ops.mlstm_scan(om, rows_m, 0, Hm * 128, 2 * Hm * 128, 2 * Hm * 128 + 2 * Hm * em, 2 * Hm * 128 + 2 * Hm * em + Hm,
+                                     zeros_m, zeros_m, states[i], slots, cu, reqs, Hm, 128, em, 15.0, 128 ** -0.5), sets)
+        del states
+        # the norm over all heads and the gate
+        gated = torch.empty(T, H * e, device=dev, dtype=bf)
+        wn = torch.ones(H * e, device=dev)
+        g_at = slice(2 * H * d + H * e, 2 * H * d + 2 * H * e)
+        row("norm over all heads times sigmoid gate", "norm per head times sigmoid gate", T, T * H * e * 8,
+            lambda i: ops.head_norm_gate(gated, o, proj[i][:, g_at], wn, 1e-5, 1, H * e, sigmoid=True), 2)
+        row("norm per head times sigmoid gate", "", T, T * H * e * 8,
+            lambda i: ops.head_norm_gate(gated, o, proj[i][:, g_at], wn, 1e-5, H, e, sigmoid=True), 2)
+        del proj, o
+        # norm per head, temperature, cache write
+        pages = (T + page - 1) // page + 1
+        btab = torch.arange(pages, dtype=torch.int32, device=dev).view(1, -1).contiguous()
+        req0 = torch.zeros(T, dtype=torch.int32, device=dev)
+        pos = torch.arange(T, dtype=torch.int32, device=dev)
+        qkv = torch.randn(T, (nh + 2 * nkv) * hd, device=dev).to(bf)
+        kc = torch.zeros(pages + 1, nkv, page, hd, device=dev, dtype=bf)
+        vc = torch.zeros_like(kc)
+        w_head = torch.ones(hd, device=dev)
+        row("norm per head + query temperature + cache write", "bias + norm over all of q and of k + turn + cache write", T,
+            T * 4 * (nh + 2 * nkv) * hd,
+            lambda i: ops.rope_norm_store(qkv, kc, vc, None, pos, req0, btab, nh, nkv, hd, 0, 0, 1e-5, hd, page, True, False, status,
+                                          w_q=w_head, w_k=w_head, temperature=(0.1, 2048), store_values=True), 1)
+        bias = torch.zeros((nh + 2 * nkv) * hd, device=dev)
+        wq, wk = torch.ones(nh * hd, device=dev), torch.ones(nkv * hd, device=dev)
+        rates = torch.rand(hd // 2, device=dev, dtype=torch.float64)
+        row("bias + norm over all of q and of k + turn + cache write", "", T, T * 4 * (nh + 2 * nkv) * hd,
+            lambda i: ops.rope_qknorm_store(qkv, bias, wq, wk, 1e-5, nh * hd, nkv * hd, rates, hd, 1.0, kc, vc, pos, req0, btab, nh, nkv, hd,
+                                            page, True, status), 1)
+        del kc, vc, qkv
+        # both outputs into the stream, in the norm's kernel
+        resid = [torch.randn(T, W, device=dev) for _ in range(4)]
+        a, b = torch.randn(T, W, device=dev).to(bf), torch.randn(T, W, device=dev).to(bf)
+        normed = torch.empty(T, W, device=dev, dtype=bf)
+        w1 = torch.ones(W, device=dev)
+        row("rmsnorm + two outputs added to the stream", "rmsnorm + residual", T, T * W * 14 + 4 * W,
+            lambda i: ops.rmsnorm_pair(normed, None, resid[i], w1, None, 1e-5, addend=a, addend2=b), 4)
+        row("rmsnorm + residual", "", T, T * W * 12 + 4 * W, lambda i: ops.rmsnorm(normed, resid[i], a, w1, 1e-5), 4)
+        del resid, a, b
+        # the four projections of lightning attention
+        x = [torch.randn(T, W, device=dev).to(bf) for _ in range(4)]
+        w_in = torch.randn(width, W, device=dev).to(bf) * 0.02
+        p_out = torch.empty(T, width, device=dev, dtype=bf)
+        row("projections, silu on q, k and v in the epilogue", "the library's product (or the weight-streaming one)", T,
+            2 * (width * W + T * W + T * width),
+            lambda i: ops.activated_linear(p_out, x[i], w_in, ops.ACT_SILU_COLUMNS, status, columns=2 * H * d + H * e), 4, flops=2 * T * width * W)
+        row("projections alone", "", T, 2 * (width * W + T * W + T * width), lambda i: ops.linear(p_out, x[i], w_in, status), 4,
+            flops=2 * T * width * W)
+        del p_out, w_in
+        # the shared expert's first product
+        wu = [torch.randn(F, W, device=dev).to(bf) * 0.02 for _ in range(4)]
+        act = torch.empty(T, F, device=dev, dtype=bf)
+        row("product with relu squared in its epilogue", "gate/up product, silu", T, 2 * (F * W + T * W + T * F),
+            lambda i: ops.activated_linear(act, x[i], wu[i], ops.ACT_RELU_SQUARED, status), 4, flops=2 * T * F * W)
+        Fg = F * 2 // 3
+        wg = [torch.randn(2 * Fg, W, device=dev).to(bf) * 0.02 for _ in range(4)]
+        act_g = torch.empty(T, Fg, device=dev, dtype=bf)
+        row("gate/up product, silu", "", T, 2 * (2 * Fg * W + T * W + T * Fg),
+            lambda i: ops.gated_linear(act_g, x[i], wg[i], ws, status), 4, flops=4 * T * Fg * W)
+        # router and experts
+        ids, share = torch.zeros(T, top, dtype=torch.int32, device=dev), torch.zeros(T, top, device=dev)
+        zbuf = torch.zeros(T * (E + I + 1), device=dev)
+        wr, cor = torch.randn(E + I, W, device=dev) * 0.05, torch.zeros(E + I, device=dev)
+        row("router: logits, softmax over all, corrected choice", "router: logits, sigmoid of the chosen", T, T * W * 2 + 4 * (E + I) * W,
+            lambda i: ops.moe_route(ids, share, None, x[i], wr, None, None, top, scratch=zbuf, scoring=ops.MOE_SOFTMAX_ALL, correction=cor), 4)
+        ids_l, share_l = torch.zeros_like(ids), torch.zeros_like(share)
+        row("router: logits, sigmoid of the chosen", "", T, T * W * 2 + 4 * (E + I) * W,
+            lambda i: ops.moe_route(ids_l, share_l, None, x[i], wr, None, None, top, scratch=zbuf, scoring=ops.MOE_SIGMOID), 4)
+        pairs = T * top
+        wide = ops.moe_wide_tiles(pairs, E, bf, W, F)
+        max_tiles = ops.moe_max_tiles(pairs, E, wide)
+        tiles, meta = torch.zeros(3, max_tiles, dtype=torch.int32, device=dev), torch.zeros(4, dtype=torch.int32, device=dev)
+        real = int((ids < E).sum())
+        used = len(set(ids[ids < E].tolist()))
+        we, wd = torch.randn(E, F, W, device=dev).to(bf) * 0.02, torch.randn(E, W, F, device=dev).to(bf) * 0.02
+        weg = torch.randn(E, 2 * Fg, W, device=dev).to(bf) * 0.02
+        shared_out, o2 = torch.randn(T, W, device=dev).to(bf), torch.empty(T, W, device=dev, dtype=bf)
+        relu2 = (ops.ACT_RELU_SQUARED, 1.0, 0.0)
+        if wide:
+            cap = max_tiles * ops.moe_tile_rows(True)
+            slots_p, pair_slot = torch.zeros(cap, dtype=torch.int32, device=dev), torch.zeros(pairs, dtype=torch.int32, device=dev)
+            xs = torch.zeros(cap, W, device=dev, dtype=bf)
+            ops.moe_group(ids, E, slots_p, tiles, meta, True, padded=True, pair_slot=pair_slot)
+            ops.moe_gather(xs, x[0], slots_p, meta, top)
+            act, act_g = torch.empty(cap, F, device=dev, dtype=bf), torch.empty(cap, Fg, device=dev, dtype=bf)
+            y = torch.zeros(cap, W, device=dev, dtype=bf)
+            row("experts' product, relu squared (tcgen05, grouped)", "experts' gate/up product, silu", T, 2 * (used * F * W + real * W + real * F),
+                lambda i: ops.gemm_tc_grouped(act, xs, we, tiles[0], meta, status=status, activation=relu2), 1, flops=2 * real * F * W)
+            row("experts' gate/up product, silu (tcgen05, grouped)", "", T, 2 * (used * 2 * Fg * W + real * W + real * Fg),
+                lambda i: ops.gemm_tc_grouped(act_g, xs, weg, tiles[0], meta, gated=True, status=status), 1, flops=4 * real * Fg * W)
+            row("experts' outputs and identity experts weighted and summed", "without identity experts", T, pairs * W * 2 + T * W * 4,
+                lambda i: ops.moe_combine_sorted(o2, y, pair_slot, share, top, shared_out, identity=(ids, x[i], E)), 4)
+            ids0 = ids % E
+            ops.moe_group(ids0, E, slots_p, tiles, meta, True, padded=True, pair_slot=pair_slot)
+            row("experts' outputs weighted and summed", "", T, pairs * W * 2 + T * W * 4,
+                lambda i: ops.moe_combine_sorted(o2, y, pair_slot, share, top, shared_out), 2)
+        else:
+            slots_p = torch.zeros(pairs, dtype=torch.int32, device=dev)
+            ops.moe_group(ids, E, slots_p, tiles, meta, wide)
+            act, act_g = torch.empty(pairs, F, device=dev, dtype=bf), torch.empty(pairs, Fg, device=dev, dtype=bf)
+            y = torch.zeros(pairs, W, device=dev)
+            row("experts' product, relu squared (mma.sync)", "experts' gate/up product, silu", T, 2 * (used * F * W + T * W + real * F),
+                lambda i: ops.moe_grouped(act, x[i], we, slots_p, tiles, meta, max_tiles, src_div=top, scatter=False, wide=wide, activation=relu2),
+                4, flops=2 * real * F * W)
+            row("experts' gate/up product, silu (mma.sync)", "", T, 2 * (used * 2 * Fg * W + T * W + real * Fg),
+                lambda i: ops.moe_grouped(act_g, x[i], weg, slots_p, tiles, meta, max_tiles, src_div=top, scatter=False, gated=True, wide=wide),
+                4, flops=4 * real * Fg * W)
+            row("experts' outputs and identity experts summed", "without identity experts", T, pairs * W * 4 + T * W * 4,
+                lambda i: ops.moe_combine(o2, y, top, shared_out, identity=(ids, x[i], E), share=share), 4)
+            row("experts' outputs summed", "", T, pairs * W * 4 + T * W * 4, lambda i: ops.moe_combine(o2, y, top, shared_out), 2)
+        del we, wd, weg, wu, wg, x
+    # attention with a sink, beside the same without
+    sink = torch.zeros(nh, device=dev)
+    for label, q_lens, ctx in (("decode, 8 requests at 4,096", [1] * 8, [4095] * 8), ("prompt of 2,048", [2048], [0])):
+        T, B = sum(q_lens), len(q_lens)
+        total = [c + n for c, n in zip(ctx, q_lens)]
+        per = (max(total) + page - 1) // page
+        btab = torch.arange(B * per, dtype=torch.int32, device=dev).view(B, per).contiguous()
+        kc = torch.randn(B * per + 1, nkv, page, hd, device=dev).to(bf)
+        vc = torch.randn(B * per + 1, nkv, page, hd, device=dev).to(bf)
+        q = torch.randn(T, nh * hd, device=dev).to(bf)
+        out = torch.empty(T, nh * hd, device=dev, dtype=bf)
+        cu = torch.tensor([0] + list(torch.tensor(q_lens).cumsum(0)), dtype=torch.int32, device=dev)
+        before = torch.tensor(ctx, dtype=torch.int32, device=dev)
+        nbytes = sum(total) * nkv * hd * 4 + T * nh * hd * 4
+        flops = 0 if T == B else 2 * nh * hd * T * (T + 1)
+        if T == B:
+            splits = 4
+            scratch = torch.zeros(max(ops.attention_decode_scratch_floats(hd, B, nh, splits), 1), device=dev)
+            forms = [("split keys", lambda i, s: ops.attention_decode_bf16(
+                out, scratch, q, q.stride(0), kc, vc, btab, cu, before, None, B, nh, nkv, hd, page, 0, hd ** -0.5, splits, status, sink=s))]
+        else:
+            req = torch.zeros(T // 128, dtype=torch.int32, device=dev)
+            q0 = torch.arange(0, T, 128, dtype=torch.int32, device=dev)
+            forms = [("mma.sync", lambda i, s: ops.attention_prefill_bf16(
+                out, q, q.stride(0), kc, vc, btab, cu, before, req, q0, T // 128, nh, nkv, hd, page, 0, hd ** -0.5, status, sink=s))]
+            if ops.attention_tc_available(hd, page):
+                forms.append(("tcgen05", lambda i, s: ops.attention_prefill_tc_bf16(
+                    out, q, q.stride(0), kc, vc, btab, cu, before, req, q0, T // 128, nh, nkv, hd, page, 0, hd ** -0.5, status, sink=s)))
+        for form, launch in forms:
+            row(f"attention ({form}) with a sink; {label}", "without", T, nbytes, lambda i: launch(i, sink), 1, flops=flops)
+            row(f"attention ({form}) without; {label}", "", T, nbytes, lambda i: launch(i, None), 1, flops=flops)
+    ops.check_status(status)
+    return rows
+
+
+def run_zuzenex(args):
+    """--only zuzenex: decode (1 and 8 requests at --context) and prefill (2,048 tokens) of a Zuzenex model beside the
+    Ribozen model (the closest existing design: a matrix of state per head, one attention layer in four, routed experts
+    with a shared one) and the Llama model of the same width, heads, layers and vocabulary (random weights, bfloat16),
+    and the design's own kernels alone beside their likes."""
+    global BLOCK_SIZE
+    import torch
+
+    BLOCK_SIZE = args.page
+    pk = peaks()
+    context = args.context or CONTEXT
+    if args.profile_step:
+        llama = dict(SHAPES[args.shapes])
+        llama["num_hidden_layers"] = args.layers or 4
+        rig = make_rig(zuzenex_config(llama), context, 8, args.page)
+        rig.runner.use_cuda_graphs = False
+        if args.profile_step == "decode":
+            ms, _, _ = rig.timed_decode(args.batch, 2, 2, context)
+        else:
+            ms = rig.timed_prefill(args.tokens or PREFILL_TOKENS, 1, 2)
+        print(json.dumps({"only": "zuzenex", "profile_step": args.profile_step, "layers": llama["num_hidden_layers"], "ms": round(ms, 3)}))
+        return 0
+    out = {"only": "zuzenex", "peaks": pk["source"], "context": context, "sizes": {}}
+    for name in ([args.shapes] if args.shapes != "1b" or args.layers else ["1b", "3b"]):
+        llama = dict(SHAPES[name])
+        if args.layers:
+            llama["num_hidden_layers"] = args.layers
+        res = {}
+        for label, cfg in (("zuzenex", zuzenex_config(llama)), ("ribozen", ribozen_config(llama)), ("llama", llama)):
+            rig = make_rig(cfg, context, 8, args.page)
+            for b in (1, 8):
+                rig.timed_decode(b, 3, 2, context - 200)
+                ms, graph_steps, _ = rig.timed_decode(b, 24, 6, context)
+                nbytes = {"zuzenex": zuzenex_decode_bytes, "ribozen": ribozen_decode_bytes, "llama": decode_bytes}[label](cfg, b, context - 12)
+                res[f"{label}_decode_b{b}_ms"] = round(ms, 4)
+                res[f"{label}_decode_b{b}_tokens_per_s"] = round(b * 1000.0 / ms, 1)
+                res[f"{label}_decode_b{b}_hbm_frac"] = round(nbytes / (ms * 1e-3) / 1e9 / pk["hbm_gbs"], 4)
+                res[f"{label}_decode_b{b}_graph_steps"] = graph_steps
+            ms = rig.timed_prefill(PREFILL_TOKENS, 3, 2)
+            if label == "zuzenex":
+                flops = zuzenex_prefill_flops(cfg, PREFILL_TOKENS)
+            else:
+                flops = ribozen_prefill_flops(cfg, PREFILL_TOKENS)[0] if label == "ribozen" else prefill_flops(cfg, PREFILL_TOKENS)
+            res[f"{label}_prefill_{PREFILL_TOKENS}_ms"] = round(ms, 3)
+            res[f"{label}_prefill_{PREFILL_TOKENS}_tokens_per_s"] = round(PREFILL_TOKENS * 1000.0 / ms, 1)
+            res[f"{label}_prefill_{PREFILL_TOKENS}_bf16_frac"] = round(flops / (ms * 1e-3) / 1e12 / pk["bf16_tflops"], 4)
+            rig.close()
+            del rig
+            torch.cuda.empty_cache()
+        out["sizes"][name] = res
+        for k, v in res.items():
+            print(f"{name}  {k} = {v}", file=sys.stderr)
+    rows = zuzenex_kernel_rows(pk, dict(SHAPES["1b"]))
+    for r in rows:
+        print("  ".join(f"{k}={v}" for k, v in r.items() if v != ""), file=sys.stderr)
+    out["kernels"] = rows
+    print(json.dumps(out))
+    return 0
+
+
 def main():
     p = argparse.ArgumentParser()
     p.add_argument("--gpus", type=int, default=1)
@@ -1932,14 +2261,15 @@ def main():
     p.add_argument("--warmup", type=int, default=16)
     p.add_argument("--impl", default="ours", choices=["ours", "reference"])
     p.add_argument("--layers", type=int, default=0, help="fewer layers than the model has (named in config)")
-    p.add_argument("--only", choices=["decode", "prefill", "mixed", "serving", "kernels", "sulepel", "kaditar", "zepilix", "ribozen"], default=None,
+    p.add_argument("--only", choices=["decode", "prefill", "mixed", "serving", "kernels", "sulepel", "kaditar", "zepilix", "ribozen", "zuzenex"], default=None,
                    help="run one kind of step and exit (for profilers and for further sizes); mixed = --batch decoding "
                         "requests beside one --tokens portion of a prompt in every step; serving = the reference's "
                         "serving benchmark (small model, prompts of 128 tokens, 32 generated: TTFT, ITL, tokens/s); "
                         "kernels = its kernel benchmark (RMSNorm and prefill attention over a grid of sizes); "
                         "sulepel = the Sulepel design beside Llama at equal sizes (decode, prefill, its kernels alone); "
                         "kaditar = the same for the Kaditar design; zepilix = the Zepilix design beside Sulepel and Llama; "
-                        "ribozen = the Ribozen design beside Zepilix and Llama")
+                        "ribozen = the Ribozen design beside Zepilix and Llama; "
+                        "zuzenex = the Zuzenex design beside Ribozen and Llama")
     p.add_argument("--batch-sizes", nargs="+", type=int, default=[1, 4, 8, 16], help="with --only serving")
     p.add_argument("--shapes", choices=sorted(SHAPES), default="1b", help="with --only: layer sizes of Llama-3.2-1B, 3.2-3B or 3.1-8B")
     p.add_argument("--batch", type=int, default=8, help="batch of --only decode")
@@ -1953,7 +2283,7 @@ def main():
     p.add_argument("--without", choices=["norms", "qkv", "attention", "o", "gate_up", "down", "head"], default=None,
                    help="with --only decode (batches up to 16): time the step with this kind of kernel left out")
     p.add_argument("--profile-step", choices=["decode", "prefill"], default=None,
-                   help="with --only sulepel, kaditar, zepilix or ribozen: run a few steps of that kind launch by launch (no captured graph) on a model of "
+                   help="with --only sulepel, kaditar, zepilix, ribozen or zuzenex: run a few steps of that kind launch by launch (no captured graph) on a model of "
                         "--layers layers (4 by default) and exit; for profilers")
     p.add_argument("--points", choices=["all", "1b"], default="all",
                    help="all: also decode, prefill and the mixed step at the 3B and 8B shapes (context 8192) in `points`")
@@ -1975,6 +2305,8 @@ def main():
         return run_zepilix(args)
     if args.only == "ribozen" and args.impl == "ours":
         return run_ribozen(args)
+    if args.only == "zuzenex" and args.impl == "ours":
+        return run_zuzenex(args)
     if args.impl == "reference":
         return run_reference(args)
     return run_ours(args)

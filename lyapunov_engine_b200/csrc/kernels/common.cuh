@@ -232,12 +232,18 @@ struct GatedActivation {
   int inter = 0;
 };
 // An activation of a product that has no gate beside it, applied by the ungated forms of the product kernels to their
-// 32-bit sums.  kind 3: max(v, 0)^2; every other kind leaves the product as it is.
-constexpr int ACT_RELU_SQUARED = 3;
-__device__ __forceinline__ float ungated_activation(float v, const GatedActivation &a) {
+// 32-bit sums, in column n.  kind 3: max(v, 0)^2; kind 4: silu(v) in the first `inter` columns, the others as they are
+// (a projection whose parts stand side by side); every other kind leaves the product as it is.
+constexpr int ACT_RELU_SQUARED = 3, ACT_SILU_COLUMNS = 4;
+template <bool FAST_EXP = false>
+__device__ __forceinline__ float ungated_activation(float v, int n, const GatedActivation &a) {
   if (a.kind == ACT_RELU_SQUARED) {
     const float r = fmaxf(v, 0.0f);
     return r * r;
+  }
+  if (a.kind == ACT_SILU_COLUMNS && n < a.inter) {
+    if constexpr (FAST_EXP) return __fdividef(v, 1.0f + __expf(-v));
+    return v / (1.0f + expf(-v));
   }
   return v;
 }

@@ -314,7 +314,7 @@ gemm_skinny_kernel(TO *__restrict__ out, const bf16 *__restrict__ x, const bf16 
           le::gated_bias(x, u, n, act);
           x = le::gated_activation(x, u, act);
         } else {
-          x = le::ungated_activation(x, act);
+          x = le::ungated_activation(x, n, act);
         }
         dst[row * ldo + n] = le::from_f32<TO>(x);
       }
@@ -440,7 +440,7 @@ int dispatch_m(void *out, const void *x, const void *w, int M, int N, int K, int
 // out is float32 [splits, M, N] (split s at out + s * split_stride elements).
 // gated = 1: W is [N = 2 I, K], out is bfloat16 [M, I] = act(x Wg^T, x Wu^T) with the activation
 // (act_kind, act_slope, act_limit) of le::GatedActivation (0: silu(g) * u); splits must be 1.  With gated = 0 and one
-// split act_kind le::ACT_RELU_SQUARED puts that activation on the product.
+// split act_kind le::ACT_RELU_SQUARED or le::ACT_SILU_COLUMNS (act_limit: how many columns) puts that activation on it.
 // Needs M <= 64, K a multiple of 8, 16-byte aligned rows of x and W.
 LE_API int le_gemm_skinny_bias_bf16(void *out, int out_dtype, const void *x, const void *w, int M, int N, int K, int64_t ldx,
                                     int64_t ldw, int64_t ldo, int splits, int64_t split_stride, int gated, int act_kind,
@@ -467,8 +467,9 @@ LE_API int le_gemm_skinny_bias_bf16(void *out, int out_dtype, const void *x, con
     return dispatch_m<true, bf16>(out, x, w, M, N, K, ldx, ldw, ldo, 1, 0, stream,
                                   le::GatedActivation{act_kind, act_slope, act_limit, bias, N / 2});
   }
-  const le::GatedActivation act{act_kind, act_slope, act_limit};
-  if (splits > 1 && act_kind == le::ACT_RELU_SQUARED) return le::invalid("le_gemm_skinny_bf16: partial sums of a split K take no activation");
+  const le::GatedActivation act{act_kind, act_slope, act_limit, nullptr,
+                                act_kind == le::ACT_SILU_COLUMNS ? static_cast<int>(act_limit) : 0};
+  if (splits > 1 && act_kind >= le::ACT_RELU_SQUARED) return le::invalid("le_gemm_skinny_bf16: partial sums of a split K take no activation");
   if (splits > 1 && out_dtype != LE_F32) return le::invalid("le_gemm_skinny_bf16: partial sums of a split K are float32");
   if (out_dtype == LE_F32) return dispatch_m<false, float>(out, x, w, M, N, K, ldx, ldw, ldo, splits, split_stride, stream, act);
   if (out_dtype == LE_BF16) return dispatch_m<false, bf16>(out, x, w, M, N, K, ldx, ldw, ldo, splits, split_stride, stream, act);

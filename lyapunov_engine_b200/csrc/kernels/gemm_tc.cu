@@ -285,7 +285,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                 if (col + i < n_limit) le::gated_bias(f[i], up, col + i, act);
                 f[i] = le::gated_activation<true>(f[i], up, act);
               } else {
-                f[i] = le::ungated_activation(f[i], act);
+                f[i] = le::ungated_activation<true>(f[i], col + i, act);
               }
             }
             if (col + 8 <= n_limit && (reinterpret_cast<uintptr_t>(dst + col) & 15) == 0) {
@@ -413,7 +413,8 @@ int launch(void *out, const void *x, const void *w, int M, int N, int K, int64_t
 // [N = 2 I, K] (gate rows, then up rows), out is bfloat16 [M, I] =
 // act(x Wg^T, x Wu^T) with the activation (act_kind, act_slope, act_limit) of
 // le::GatedActivation (0: silu(g) * u).  With gated = 0 act_kind
-// le::ACT_RELU_SQUARED puts that activation on the product.  Needs K and the leading dimensions of x and W to
+// le::ACT_RELU_SQUARED or le::ACT_SILU_COLUMNS (act_limit: how many
+// columns) puts that activation on the product.  Needs K and the leading dimensions of x and W to
 // be multiples of 8 and their base addresses 16-byte aligned (TMA).
 LE_API int le_gemm_tc_bias_bf16(void *out, int out_dtype, const void *x, const void *w, int M, int N, int K, int64_t ldx,
                                 int64_t ldw, int64_t ldo, int gated, int act_kind, float act_slope, float act_limit,
@@ -431,8 +432,9 @@ LE_API int le_gemm_tc_bias_bf16(void *out, int out_dtype, const void *x, const v
                                 int64_t ldw, int64_t ldo, int gated, int act_kind, float act_slope, float act_limit,
                                 const float *bias, int *status, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
-  if (act_kind < 0 || act_kind > (gated ? 2 : le::ACT_RELU_SQUARED)) return le::invalid("le_gemm_tc_bf16: unknown activation %d", act_kind);
-  const le::GatedActivation act{act_kind, act_slope, act_limit, gated ? bias : nullptr, N / 2};
+  if (act_kind < 0 || act_kind > (gated ? 2 : le::ACT_SILU_COLUMNS)) return le::invalid("le_gemm_tc_bf16: unknown activation %d", act_kind);
+  const le::GatedActivation act{act_kind, act_slope, act_limit, gated ? bias : nullptr,
+                                act_kind == le::ACT_SILU_COLUMNS ? static_cast<int>(act_limit) : N / 2};
   if (K <= 0 || K % 8 || ldx % 8 || ldw % 8) return le::invalid("le_gemm_tc_bf16: K (%d) and the leading dimensions must be multiples of 8", K);
   if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15) return le::invalid("le_gemm_tc_bf16: x and W must be 16-byte aligned");
   // pairs of SMs on 256 x 256 tiles where those give at least half of the pairs a tile and the second block of a

@@ -9,8 +9,7 @@
 // scan: token by token, any type and size.  A block takes one request, one
 // head and ROWS of the vdim columns of S; a column has LANES threads, each with
 // every LANES-th group of four entries in registers.  Tokens pass in tiles
-// through shared memory.  q, k and v come as projected (silu is applied here and
-// rounded to the activations' type) or activated already.  The decay comes in
+// through shared memory.  The decay comes in
 // two floats whose sum is the 64-bit number: its rounding to one float would lean
 // the same way at every token, and a memory of a thousand tokens would be off
 // by a thousand times that.  This is the kernel of decoded tokens, which is
@@ -44,8 +43,6 @@ constexpr int LS_THREADS = 256;
 constexpr int LS_TILE = 16;
 constexpr int LS_QUADS = 4;       // groups of four entries a thread holds at most
 
-__device__ __forceinline__ float silu_f32(float v) { return v / (1.0f + expf(-v)); }
-
 struct ScanArgs {
   float *out; int64_t out_stride;
   const void *rows; int64_t row_stride; int q_col, k_col, v_col;
@@ -53,7 +50,7 @@ struct ScanArgs {
   float *state; int num_state_rows;
   const int32_t *state_slots, *cu_q;
   const int32_t *requests;        // the requests this launch takes, or null: all in order
-  int heads, dim, vdim, rows_per_block, activated, tile;
+  int heads, dim, vdim, rows_per_block, tile;
 };
 
 template <typename T, int LANES>
@@ -98,7 +95,6 @@ lightning_scan_kernel(ScanArgs p) {
     }
   }
   const T *rows = static_cast<const T *>(p.rows);
-  auto enter = [&](T x) { return p.activated ? le::to_f32(x) : le::to_f32(le::from_f32<T>(silu_f32(le::to_f32(x)))); };
 
   for (int t0 = 0; t0 < q_len; t0 += p.tile) {
     const int tile = min(p.tile, q_len - t0);
@@ -106,12 +102,12 @@ lightning_scan_kernel(ScanArgs p) {
     for (int i = threadIdx.x; i < tile * DQ; i += threads) {
       const int t = i / DQ, d = i - t * DQ;
       const T *row = rows + static_cast<int64_t>(first + t0 + t) * p.row_stride + static_cast<int64_t>(head) * D + d;
-      s_q[i] = d < D ? enter(row[p.q_col]) : 0.0f;
-      s_k[i] = d < D ? enter(row[p.k_col]) : 0.0f;
+      s_q[i] = d < D ? le::to_f32(row[p.q_col]) : 0.0f;
+      s_k[i] = d < D ? le::to_f32(row[p.k_col]) : 0.0f;
     }
     for (int i = threadIdx.x; i < tile * ROWS; i += threads) {
       const int t = i / ROWS, c = i - t * ROWS;
-      s_v[i] = c < cols ? enter(rows[static_cast<int64_t>(first + t0 + t) * p.row_stride + p.v_col +
+      s_v[i] = c < cols ? le::to_f32(rows[static_cast<int64_t>(first + t0 + t) * p.row_stride + p.v_col +
                                      static_cast<int64_t>(head) * p.vdim + e0 + c]) : 0.0f;
     }
     __syncthreads();
@@ -209,17 +205,17 @@ __device__ __forceinline__ float high_of(uint32_t v) { return __uint_as_float(v 
 struct ChunkArgs {
   float *out; int64_t out_stride;
   const bf16 *rows; int64_t row_stride; int q_col, k_col, v_col;
-  const float *powers;            // [heads, CHUNK + 1]: decay^n
-  const double *decay;            // [heads]
+  const float *powers;            // [heads, SEGMENT + 1]: decay^n
   float *state; int num_state_rows;
   float *scratch;                 // [segments, heads, vdim, dim], or null: every request is one segment
   const int32_t *state_slots, *cu_q, *tile_request, *tile_q0;
   int heads, dim, vdim, vector;   // vector: 16-byte pieces are whole and aligned
 };
 
-template <int DP>
+template <int DP, bool SUMS>
 constexpr size_t chunk_smem() {
-  return sizeof(bf16) * (2 * CHUNK * (DP + 8) + CHUNK * LC_LDV + 2 * DP * LC_LDV) + sizeof(float) * (CHUNK + 4);
+  return sizeof(bf16) * ((SUMS ? 2 : 3) * CHUNK * (DP + 8) + 2 * CHUNK * LC_LDV + (SUMS ? 0 : 2 * DP * LC_LDV)) +
+         sizeof(float) * (CHUNK + 4);
 }
 
 // DP: the heads' entries, padded to a multiple of 32 (zeros behind the real ones).  SUMS: only the segment's own sum
@@ -234,11 +230,11 @@ lightning_chunk_kernel(ChunkArgs p) {
   constexpr int TILES = DP / 16 * NT / 8;          // tiles of S a warp holds
   constexpr int KSTEPS = DP / 16;
   bf16 *s_q = reinterpret_cast<bf16 *>(lc_smem);   // [CHUNK][LD]
-  bf16 *s_k = s_q + CHUNK * LD;                    // [CHUNK][LD]
-  bf16 *s_v = s_k + CHUNK * LD;                    // [CHUNK][LC_LDV]
-  bf16 *s_sh = s_v + CHUNK * LC_LDV;               // [DP][LC_LDV]: S, high parts
+  bf16 *s_k = s_q + (SUMS ? 0 : CHUNK * LD);       // [2][CHUNK][LD]
+  bf16 *s_v = s_k + 2 * CHUNK * LD;                // [2][CHUNK][LC_LDV]
+  bf16 *s_sh = s_v + 2 * CHUNK * LC_LDV;           // [DP][LC_LDV]: S, high parts
   bf16 *s_sl = s_sh + DP * LC_LDV;                 // low parts
-  float *s_pow = reinterpret_cast<float *>(s_sl + DP * LC_LDV);      // [CHUNK + 1]
+  float *s_pow = reinterpret_cast<float *>(SUMS ? s_sh : s_sl + DP * LC_LDV);      // [CHUNK + 1]
   le::let_successor_start();
   const int slices = (p.vdim + LC_COLS - 1) / LC_COLS;
   const int head = blockIdx.x / slices, e0 = (blockIdx.x % slices) * LC_COLS;
@@ -246,7 +242,7 @@ lightning_chunk_kernel(ChunkArgs p) {
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int g = lane >> 2, t4 = lane & 3, j8 = lane >> 3, r8 = lane & 7;
   const int D = p.dim, cols = min(LC_COLS, p.vdim - e0);
-  for (int i = tid; i <= CHUNK; i += LC_THREADS) s_pow[i] = p.powers[head * (CHUNK + 1) + i];
+  for (int i = tid; i <= CHUNK; i += LC_THREADS) s_pow[i] = p.powers[head * (SEGMENT + 1) + i];
   le::wait_for_predecessor();
   const int b = p.tile_request[seg], q0 = p.tile_q0[seg];
   const int tokens = min(SEGMENT, p.cu_q[b + 1] - p.cu_q[b] - q0);
@@ -271,51 +267,34 @@ lightning_chunk_kernel(ChunkArgs p) {
       acc_s[i][e] = from != nullptr && d < D && c < cols ? from[static_cast<int64_t>(e0 + c) * D + d] : 0.0f;
     }
 
-  // a chunk's raw pieces: asked for one chunk ahead, kept in registers while the one before is worked on
-  constexpr int QK_PIECES = CHUNK * DP / 8 / LC_THREADS;        // of q and of k, per thread
-  constexpr int V_PIECES = CHUNK * LC_COLS / 8 / LC_THREADS;
-  uint4 raw_q[SUMS ? 1 : QK_PIECES], raw_k[QK_PIECES], raw_v[V_PIECES];
-  auto piece = [&](int col, int64_t token, bool live, int at, int limit) {      // 8 values from column `at` of a head
-    uint4 r = make_uint4(0, 0, 0, 0);
-    if (!live || at >= limit) return r;
-    const bf16 *src = p.rows + token * p.row_stride + col + at;
-    if (p.vector) return *reinterpret_cast<const uint4 *>(src);
-    bf16 *e = reinterpret_cast<bf16 *>(&r);
+  // A chunk's rows, copied straight into shared memory while the chunk before is worked on: k and v have two buffers,
+  // q one (it is free once the fragments are in registers).  Rows beyond the tokens and entries beyond the sizes: zeros.
+  auto copy_rows = [&](bf16 *dst, int ld, int pieces, int col, int limit, int c0) {
+    for (int id = tid; id < CHUNK * pieces; id += LC_THREADS) {
+      const int t = id / pieces, at = (id - t * pieces) * 8;
+      const bool live = c0 + t < tokens && at < limit;
+      const bf16 *src = live ? p.rows + (first + c0 + t) * p.row_stride + col + at : p.rows;
+      bf16 *to = dst + t * ld + at;
+      if (p.vector) {
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(smem_addr(to)), "l"(src), "r"(live ? 16 : 0) : "memory");
+      } else {
 #pragma unroll
-    for (int u = 0; u < 8; ++u)
-      if (at + u < limit) e[u] = src[u];
-    return r;
+        for (int u = 0; u < 8; ++u) to[u] = live && at + u < limit ? src[u] : __float2bfloat16_rn(0.0f);
+      }
+    }
   };
   auto fetch = [&](int c0) {
-#pragma unroll
-    for (int i = 0; i < QK_PIECES; ++i) {
-      const int id = tid + i * LC_THREADS, t = id / (DP / 8), d = (id % (DP / 8)) * 8;
-      const bool live = c0 + t < tokens;
-      if constexpr (!SUMS) raw_q[i] = piece(p.q_col + head * D, first + c0 + t, live, d, D);
-      raw_k[i] = piece(p.k_col + head * D, first + c0 + t, live, d, D);
-    }
-#pragma unroll
-    for (int i = 0; i < V_PIECES; ++i) {
-      const int id = tid + i * LC_THREADS, t = id / (LC_COLS / 8), c = (id % (LC_COLS / 8)) * 8;
-      raw_v[i] = piece(p.v_col + head * p.vdim + e0, first + c0 + t, c0 + t < tokens, c, cols);
-    }
+    const int buffer = (c0 / CHUNK) & 1;
+    if constexpr (!SUMS) copy_rows(s_q, LD, DP / 8, p.q_col + head * D, D, c0);
+    copy_rows(s_k + buffer * CHUNK * LD, LD, DP / 8, p.k_col + head * D, D, c0);
+    copy_rows(s_v + buffer * CHUNK * LC_LDV, LC_LDV, LC_COLS / 8, p.v_col + head * p.vdim + e0, cols, c0);
+    asm volatile("cp.async.commit_group;\n" ::: "memory");
   };
   fetch(0);
 
   for (int c0 = 0; c0 < tokens; c0 += CHUNK) {
     const int L = min(CHUNK, tokens - c0);
-    __syncthreads();                             // everyone is done with the chunk before
-#pragma unroll
-    for (int i = 0; i < QK_PIECES; ++i) {
-      const int id = tid + i * LC_THREADS, t = id / (DP / 8), d = (id % (DP / 8)) * 8;
-      if constexpr (!SUMS) *reinterpret_cast<uint4 *>(s_q + t * LD + d) = raw_q[i];
-      *reinterpret_cast<uint4 *>(s_k + t * LD + d) = raw_k[i];
-    }
-#pragma unroll
-    for (int i = 0; i < V_PIECES; ++i) {
-      const int id = tid + i * LC_THREADS, t = id / (LC_COLS / 8), c = (id % (LC_COLS / 8)) * 8;
-      *reinterpret_cast<uint4 *>(s_v + t * LC_LDV + c) = raw_v[i];
-    }
+    const bf16 *k_at = s_k + ((c0 / CHUNK) & 1) * CHUNK * LD, *v_at = s_v + ((c0 / CHUNK) & 1) * CHUNK * LC_LDV;
     if constexpr (!SUMS) {
 #pragma unroll
       for (int i = 0; i < TILES; ++i)
@@ -328,16 +307,24 @@ lightning_chunk_kernel(ChunkArgs p) {
           *reinterpret_cast<uint32_t *>(s_sl + at) = low;
         }
     }
-    __syncthreads();
+    asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+    __syncthreads();                             // the chunk and the state before it are there
+    // this warp's tokens and columns (the later tokens see more keys: the warps of a scheduler share them out)
+    const int r0 = 16 * (warp < 4 ? warp : 7 - warp), n0 = 32 * (warp >> 2);
+    const bool outputs = !SUMS && r0 < L && n0 < cols;
+    uint32_t qf[KSTEPS][4];
+    if constexpr (!SUMS) {
+      if (outputs) {
+#pragma unroll
+        for (int ks = 0; ks < KSTEPS; ++ks) ldsm4(qf[ks], s_q + (r0 + (j8 & 1) * 8 + r8) * LD + ks * 16 + (j8 >> 1) * 8);
+      }
+      __syncthreads();                           // q is in registers
+    }
     if (c0 + CHUNK < tokens) fetch(c0 + CHUNK);
 
     if constexpr (!SUMS) {
-      const int r0 = 16 * (warp & 3), n0 = 32 * (warp >> 2);      // this warp's tokens and columns
-      if (r0 < L && n0 < cols) {
+      if (outputs) {
         const int row[2] = {r0 + g, r0 + g + 8};
-        uint32_t qf[KSTEPS][4];
-#pragma unroll
-        for (int ks = 0; ks < KSTEPS; ++ks) ldsm4(qf[ks], s_q + (r0 + (j8 & 1) * 8 + r8) * LD + ks * 16 + (j8 >> 1) * 8);
         // what the state before the chunk gives
         float o[4][4];
 #pragma unroll
@@ -367,7 +354,7 @@ lightning_chunk_kernel(ChunkArgs p) {
 #pragma unroll
           for (int ks = 0; ks < KSTEPS; ++ks) {
             uint32_t kf[4];
-            ldsm4(kf, s_k + (kb + (j8 >> 1) * 8 + r8) * LD + ks * 16 + (j8 & 1) * 8);
+            ldsm4(kf, k_at + (kb + (j8 >> 1) * 8 + r8) * LD + ks * 16 + (j8 & 1) * 8);
             mma(s[0], qf[ks], kf[0], kf[1]);
             mma(s[1], qf[ks], kf[2], kf[3]);
           }
@@ -384,7 +371,7 @@ lightning_chunk_kernel(ChunkArgs p) {
 #pragma unroll
           for (int np = 0; np < 2; ++np) {
             uint32_t vf[4];
-            ldsm4_trans(vf, s_v + (kb + (j8 & 1) * 8 + r8) * LC_LDV + n0 + np * 16 + (j8 >> 1) * 8);
+            ldsm4_trans(vf, v_at + (kb + (j8 & 1) * 8 + r8) * LC_LDV + n0 + np * 16 + (j8 >> 1) * 8);
             mma(o[2 * np], pl, vf[0], vf[1]);
             mma(o[2 * np + 1], pl, vf[2], vf[3]);
             mma(o[2 * np], ph, vf[0], vf[1]);
@@ -432,13 +419,13 @@ lightning_chunk_kernel(ChunkArgs p) {
           if (tile_row(i) != have) {
             have = tile_row(i);
             uint32_t kf[4];
-            ldsm4_trans(kf, s_k + (kb + (j8 >> 1) * 8 + r8) * LD + have + (j8 & 1) * 8);
+            ldsm4_trans(kf, k_at + (kb + (j8 >> 1) * 8 + r8) * LD + have + (j8 & 1) * 8);
 #pragma unroll
             for (int u = 0; u < 4; ++u)
               split_pair(low_of(kf[u]) * f[(u >> 1) * 2], high_of(kf[u]) * f[(u >> 1) * 2 + 1], ah[u], al[u]);
           }
           uint32_t vf[4];
-          ldsm4_trans(vf, s_v + (kb + (j8 & 1) * 8 + r8) * LC_LDV + tile_col(i) + (j8 >> 1) * 8);
+          ldsm4_trans(vf, v_at + (kb + (j8 & 1) * 8 + r8) * LC_LDV + tile_col(i) + (j8 >> 1) * 8);
           mma(acc_s[i], al, vf[0], vf[1]);
           if (pair) mma(acc_s[i + 1], al, vf[2], vf[3]);
           mma(acc_s[i], ah, vf[0], vf[1]);
@@ -446,6 +433,7 @@ lightning_chunk_kernel(ChunkArgs p) {
         }
       }
     }
+    __syncthreads();                             // everyone is done with this chunk's keys and values and with S
   }
 
   float *to = nullptr;
@@ -462,44 +450,70 @@ lightning_chunk_kernel(ChunkArgs p) {
 }
 
 // From every segment's own sum: the state each segment starts from (in place of the sums) and the request's new state
-// row.  A request's segments are neighbours in the list; the blocks of its first one do its work.
+// row.  A request's segments stand in the list in their order, other requests' between them; the blocks of its first one
+// do its work, a thread for four entries of S (V = 4; 1 where they are no whole pieces), with the sums of eight segments
+// asked for at a time.
+constexpr int LC_AHEAD = 8;
+template <int V>
 __global__ void __launch_bounds__(256)
 lightning_starts_kernel(ChunkArgs p, int num_segments) {
   le::let_successor_start();
   const int seg = blockIdx.z, head = blockIdx.y;
   const int n = p.vdim * p.dim;
-  __shared__ float s_keep, s_last;
-  le::wait_for_predecessor();
-  if (p.tile_q0[seg] != 0) return;
+  const int i = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+  if (p.tile_q0[seg] != 0 || i >= n) return;      // (the step's integers are older than the kernel before this one)
   const int b = p.tile_request[seg];
   const int q_len = p.cu_q[b + 1] - p.cu_q[b];
-  const int segments = min((q_len + SEGMENT - 1) / SEGMENT, num_segments - seg);
-  if (threadIdx.x == 0) {
-    s_keep = static_cast<float>(pow(p.decay[head], static_cast<double>(SEGMENT)));
-    s_last = static_cast<float>(pow(p.decay[head], static_cast<double>(q_len - (segments - 1) * SEGMENT)));
-  }
-  __syncthreads();
+  const int segments = (q_len + SEGMENT - 1) / SEGMENT;
+  const float keep = p.powers[head * (SEGMENT + 1) + SEGMENT];
+  const float last = p.powers[head * (SEGMENT + 1) + min(SEGMENT, q_len - (segments - 1) * SEGMENT)];
   const int slot = p.state_slots[b];
   const bool has_state = slot >= 0 && slot < p.num_state_rows;
-  const int i = blockIdx.x * blockDim.x + threadIdx.x;
-  if (i >= n) return;
   float *row = has_state ? p.state + (static_cast<int64_t>(slot) * p.heads + head) * n + i : nullptr;
-  float *part = p.scratch + (static_cast<int64_t>(seg) * p.heads + head) * n + i;
+  float *part = p.scratch + static_cast<int64_t>(head) * n + i;       // of segment s of the list: + s * step
   const int64_t step = static_cast<int64_t>(p.heads) * n;
-  float S = row != nullptr ? *row : 0.0f;
-  float next = part[0];
-  for (int s = 0; s < segments; ++s) {
-    const float sum = next;
-    if (s + 1 < segments) next = part[(s + 1) * step];
-    part[s * step] = S;
-    S = fmaf(s + 1 < segments ? s_keep : s_last, S, sum);
+  auto load = [](float (&v)[V], const float *at) {
+    if constexpr (V == 4) {
+      const float4 r = *reinterpret_cast<const float4 *>(at);
+      v[0] = r.x, v[1] = r.y, v[2] = r.z, v[3] = r.w;
+    } else {
+      v[0] = *at;
+    }
+  };
+  auto store = [](float *at, const float (&v)[V]) {
+    if constexpr (V == 4) *reinterpret_cast<float4 *>(at) = make_float4(v[0], v[1], v[2], v[3]);
+    else *at = v[0];
+  };
+  le::wait_for_predecessor();
+  float S[V];
+#pragma unroll
+  for (int v = 0; v < V; ++v) S[v] = 0.0f;
+  if (row != nullptr) load(S, row);
+  int at = seg;                                   // the request's next segment in the list
+  for (int s0 = 0; s0 < segments; s0 += LC_AHEAD) {
+    float sum[LC_AHEAD][V];
+    int where[LC_AHEAD];
+#pragma unroll
+    for (int u = 0; u < LC_AHEAD; ++u) {
+      while (at < num_segments && p.tile_request[at] != b) ++at;
+      where[u] = s0 + u < segments && at < num_segments ? at++ : -1;
+      if (where[u] >= 0) load(sum[u], part + where[u] * step);
+    }
+#pragma unroll
+    for (int u = 0; u < LC_AHEAD; ++u) {
+      if (where[u] < 0) break;
+      store(part + where[u] * step, S);
+      const float f = s0 + u + 1 < segments ? keep : last;
+#pragma unroll
+      for (int v = 0; v < V; ++v) S[v] = fmaf(f, S[v], sum[u][v]);
+    }
   }
-  if (row != nullptr) *row = S;
+  if (row != nullptr) store(row, S);
 }
 
 template <int DP, bool SUMS>
 int launch_chunks(const ChunkArgs &p, int segments, cudaStream_t stream) {
-  constexpr size_t smem = chunk_smem<DP>();
+  constexpr size_t smem = chunk_smem<DP, SUMS>();
   auto kernel = lightning_chunk_kernel<DP, SUMS>;
   if (smem > 48 * 1024) {
     static bool raised = false;                  // once per form and process
@@ -518,8 +532,11 @@ int run_chunks(const ChunkArgs &p, int segments, cudaStream_t stream) {
   if (p.scratch != nullptr) {
     int rc = launch_chunks<DP, true>(p, segments, stream);
     if (rc != 0) return rc;
-    const dim3 grid((p.vdim * p.dim + 255) / 256, p.heads, segments);
-    rc = le::launch_chained(lightning_starts_kernel, grid, dim3(256), 0, stream, p, segments);
+    const int n = p.vdim * p.dim;
+    const bool quads = n % 4 == 0 && (reinterpret_cast<uintptr_t>(p.scratch) | reinterpret_cast<uintptr_t>(p.state)) % 16 == 0;
+    const dim3 grid((n / (quads ? 4 : 1) + 255) / 256, p.heads, segments);
+    rc = quads ? le::launch_chained(lightning_starts_kernel<4>, grid, dim3(256), 0, stream, p, segments)
+               : le::launch_chained(lightning_starts_kernel<1>, grid, dim3(256), 0, stream, p, segments);
     if (rc != 0) return rc;
   }
   return launch_chunks<DP, false>(p, segments, stream);
@@ -528,11 +545,11 @@ int run_chunks(const ChunkArgs &p, int segments, cudaStream_t stream) {
 }  // namespace
 
 // out: float32 [T, heads * vdim].  rows (`dtype`): per token q [heads, dim] at q_col, k at k_col, v [heads, vdim] at
-// v_col, as projected, or after silu with `activated`.  decay: float32 [2, heads], the decays' high and low parts.
+// v_col, after their activation.  decay: float32 [2, heads], the decays' high and low parts.
 // state: float32 [num_state_rows, heads, vdim, dim].  requests: the indices of the num_requests requests to run, or
 // null: requests 0 .. num_requests - 1.  single: every one of them brings one token (it only chooses the launch's shape).
 LE_API int le_lightning_scan(float *out, int64_t out_stride, const void *rows, int64_t row_stride, int q_col, int k_col, int v_col,
-                             int dtype, int activated, const float *decay, float *state, int num_state_rows,
+                             int dtype, const float *decay, float *state, int num_state_rows,
                              const int32_t *state_slots, const int32_t *cu_q, const int32_t *requests, int num_requests,
                              int heads, int dim, int vdim, int single, cudaStream_t stream) {
   if (num_requests <= 0) return 0;
@@ -544,7 +561,7 @@ LE_API int le_lightning_scan(float *out, int64_t out_stride, const void *rows, i
   ScanArgs p;
   p.out = out, p.out_stride = out_stride, p.rows = rows, p.row_stride = row_stride, p.q_col = q_col, p.k_col = k_col, p.v_col = v_col;
   p.decay = decay, p.state = state, p.num_state_rows = num_state_rows, p.state_slots = state_slots, p.cu_q = cu_q;
-  p.requests = requests, p.heads = heads, p.dim = dim, p.vdim = vdim, p.activated = activated;
+  p.requests = requests, p.heads = heads, p.dim = dim, p.vdim = vdim;
   p.tile = single ? 1 : LS_TILE;
   const int most = LS_THREADS / lanes;
   p.rows_per_block = vdim < most ? vdim : most;
@@ -566,15 +583,14 @@ LE_API int le_lightning_scan(float *out, int64_t out_stride, const void *rows, i
 }
 
 LE_API int le_lightning_segment() { return SEGMENT; }
-LE_API int le_lightning_chunk() { return CHUNK; }
 
-// The same over chunks, for bfloat16 rows that went through their activation and heads of up to 128 entries.
+// The same over chunks, for bfloat16 rows and heads of up to 128 entries.
 // tile_request / tile_q0 list num_segments segments of le_lightning_segment() tokens: their requests and their first
-// tokens within them, a request's segments one after the other.  powers: float32 [heads, le_lightning_chunk() + 1],
-// decay^n; decay: float64 [heads].  scratch: float32 [num_segments, heads, vdim, dim] where a request has several
+// tokens within them, a request's segments in their order (other requests' may stand between them).  powers: float32 [heads, le_lightning_segment() + 1],
+// decay^n.  scratch: float32 [num_segments, heads, vdim, dim] where a request has several
 // segments, else null.
 LE_API int le_lightning_chunks(float *out, int64_t out_stride, const void *rows, int64_t row_stride, int q_col, int k_col,
-                               int v_col, const float *powers, const double *decay, float *state, int num_state_rows,
+                               int v_col, const float *powers, float *state, int num_state_rows,
                                float *scratch, const int32_t *state_slots, const int32_t *cu_q, const int32_t *tile_request,
                                const int32_t *tile_q0, int num_segments, int heads, int dim, int vdim, cudaStream_t stream) {
   if (num_segments <= 0) return 0;
@@ -582,7 +598,7 @@ LE_API int le_lightning_chunks(float *out, int64_t out_stride, const void *rows,
     return le::invalid("le_lightning_chunks: %d heads of %d x %d in %d segments", heads, dim, vdim, num_segments);
   ChunkArgs p;
   p.out = out, p.out_stride = out_stride, p.rows = static_cast<const bf16 *>(rows), p.row_stride = row_stride;
-  p.q_col = q_col, p.k_col = k_col, p.v_col = v_col, p.powers = powers, p.decay = decay, p.state = state;
+  p.q_col = q_col, p.k_col = k_col, p.v_col = v_col, p.powers = powers, p.state = state;
   p.num_state_rows = num_state_rows, p.scratch = scratch, p.state_slots = state_slots, p.cu_q = cu_q;
   p.tile_request = tile_request, p.tile_q0 = tile_q0, p.heads = heads, p.dim = dim, p.vdim = vdim;
   p.vector = dim % 8 == 0 && vdim % 8 == 0 && q_col % 8 == 0 && k_col % 8 == 0 && v_col % 8 == 0 && row_stride % 8 == 0 &&

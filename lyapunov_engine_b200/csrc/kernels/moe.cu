@@ -286,27 +286,96 @@ __global__ void moe_gather_kernel(T *__restrict__ out, const T *__restrict__ x, 
   for (int i = threadIdx.x; i < width / PIECE; i += blockDim.x) dst[i] = src != nullptr ? src[i] : make_uint4(0, 0, 0, 0);
 }
 
-// out[t] = sum_j share[t, j] * y[pair_slot[t * top + j]] (+ gate[t] * shared[t]): the weighted sum over rows that
-// lie in slot order.  ids (or nullptr): pairs of an identity expert (id >= experts) add share * h[t] instead.
-template <typename T, typename TY>
-__global__ void moe_combine_sorted_kernel(T *__restrict__ out, const TY *__restrict__ y, const int32_t *__restrict__ pair_slot,
-                                          const float *__restrict__ share, const T *__restrict__ shared_out,
-                                          const float *__restrict__ gate, const int32_t *__restrict__ ids,
-                                          const T *__restrict__ h, int64_t h_stride, int experts, int64_t n, int width, int top) {
+// VEC values at p as floats and back: pieces of up to 16 bytes where VEC > 1 (aligned to them).
+template <typename T, int VEC>
+__device__ __forceinline__ void load_values(float (&v)[VEC], const T *p) {
+  if constexpr (VEC * sizeof(T) >= 16) {
+    constexpr int PIECE = le::Piece16<T>::COUNT;
+#pragma unroll
+    for (int i = 0; i < VEC; i += PIECE) {
+      float part[PIECE];
+      le::load_piece16<T>(part, p + i);
+#pragma unroll
+      for (int e = 0; e < PIECE; ++e) v[i + e] = part[e];
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] = le::to_f32(p[i]);
+  }
+}
+template <typename T, int VEC>
+__device__ __forceinline__ void store_values(T *p, const float (&v)[VEC]) {
+  if constexpr (VEC * sizeof(T) == 16) {
+    uint4 raw;
+    T *e = reinterpret_cast<T *>(&raw);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) e[i] = le::from_f32<T>(v[i]);
+    *reinterpret_cast<uint4 *>(p) = raw;
+  } else {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) p[i] = le::from_f32<T>(v[i]);
+  }
+}
+
+// The last step: a token's experts' outputs and the shared expert's, VEC values a thread (16 bytes of T, or one).
+//   SORTED:  out[t] = sum_j share[t, j] * y[pair_slot[t * top + j]]      (rows of y in slot order; share null: 1)
+//   else:    out[t] = sum_j y[t * top + j]                               (rows of y by pair, weighted already)
+// (+ gate[t] * shared[t]; gate null: 1).  ids (or null): a pair of an identity expert (id >= experts) adds share * h[t]
+// instead of a row of y.
+template <typename T, typename TY, bool SORTED, int VEC>
+__global__ void __launch_bounds__(256)
+moe_combine_kernel(T *__restrict__ out, const TY *__restrict__ y, const int32_t *__restrict__ pair_slot,
+                   const float *__restrict__ share, const T *__restrict__ shared_out, const float *__restrict__ gate,
+                   const int32_t *__restrict__ ids, const T *__restrict__ h, int64_t h_stride, int experts, int64_t n, int width,
+                   int top) {
   le::let_successor_start();
   le::wait_for_predecessor();
   const int64_t i = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x;
-  if (i >= n) return;
-  const int64_t t = i / width, c = i - t * width;
-  float acc = 0.0f;
+  if (i >= n) return;                       // n: groups of VEC values
+  const int per_row = width / VEC;
+  const int64_t t = i / per_row, c = (i - t * per_row) * VEC;
+  float acc[VEC], v[VEC];
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) acc[e] = 0.0f;
   for (int j = 0; j < top; ++j) {
-    const bool identity = ids != nullptr && ids[t * top + j] >= experts;
-    const float v = identity ? le::to_f32(h[t * h_stride + c])
-                             : le::to_f32(y[static_cast<int64_t>(pair_slot[t * top + j]) * width + c]);
-    acc = fmaf(share != nullptr ? share[t * top + j] : 1.0f, v, acc);
+    const int64_t p = t * top + j;
+    const bool identity = ids != nullptr && ids[p] >= experts;
+    if (identity) load_values<T, VEC>(v, h + t * h_stride + c);
+    else load_values<TY, VEC>(v, y + static_cast<int64_t>(SORTED ? pair_slot[p] : p) * width + c);
+    if (SORTED || identity) {
+      const float f = share != nullptr ? share[p] : 1.0f;
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) acc[e] = fmaf(f, v[e], acc[e]);
+    } else {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) acc[e] += v[e];
+    }
   }
-  if (shared_out != nullptr) acc = fmaf(gate != nullptr ? gate[t] : 1.0f, le::to_f32(shared_out[i]), acc);
-  out[i] = le::from_f32<T>(acc);
+  if (shared_out != nullptr) {
+    const float f = gate != nullptr ? gate[t] : 1.0f;
+    load_values<T, VEC>(v, shared_out + t * width + c);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) acc[e] = fmaf(f, v[e], acc[e]);
+  }
+  store_values<T, VEC>(out + t * width + c, acc);
+}
+
+template <typename T, typename TY, bool SORTED>
+int launch_combine(void *out, const void *y, const int32_t *pair_slot, const float *share, const void *shared_out, const float *gate,
+                   const int32_t *ids, const void *h, int64_t h_stride, int experts, int tokens, int width, int top,
+                   cudaStream_t stream) {
+  constexpr int VEC = le::Piece16<T>::COUNT;
+  const auto on16 = [](const void *p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+  const bool wide = width % VEC == 0 && h_stride % VEC == 0 && on16(out) && on16(y) && on16(shared_out) && on16(h);
+  const int64_t n = static_cast<int64_t>(tokens) * width / (wide ? VEC : 1);
+  const dim3 grid(static_cast<unsigned>((n + 255) / 256)), block(256);
+#define LE_GO(V)                                                                                                            \
+  return le::launch_chained(moe_combine_kernel<T, TY, SORTED, V>, grid, block, 0, stream, static_cast<T *>(out),            \
+                            static_cast<const TY *>(y), pair_slot, share, static_cast<const T *>(shared_out), gate, ids,    \
+                            static_cast<const T *>(h), h_stride, experts, n, width, top)
+  if (wide) LE_GO(VEC);
+  LE_GO(1);
+#undef LE_GO
 }
 
 template <typename T, typename TOut, bool GATED>
@@ -388,7 +457,7 @@ __global__ void moe_grouped_kernel(TOut *__restrict__ out, int64_t out_stride, c
         v = le::gated_activation(v * row_factor[m], acc_up[i][j] * row_factor[m], act);
         o[n] = le::from_f32<TOut>(v);
       } else {
-        o[n] = le::from_f32<TOut>(le::ungated_activation(v, act) * row_factor[m]);
+        o[n] = le::from_f32<TOut>(le::ungated_activation(v, n, act) * row_factor[m]);
       }
     }
   }
@@ -552,7 +621,7 @@ moe_grouped_mma_kernel(TOut *__restrict__ out, int64_t out_stride, const __nv_bf
             v = le::gated_activation(v * f, acc[1][mt][nt][half * 2 + j] * f, act);
             o[n] = le::from_f32<TOut>(v);
           } else {
-            o[n] = le::from_f32<TOut>(le::ungated_activation(v, act) * f);
+            o[n] = le::from_f32<TOut>(le::ungated_activation(v, n, act) * f);
           }
         }
     }
@@ -572,26 +641,6 @@ int launch_grouped_mma(int N, int max_tiles, cudaStream_t stream, Args... args) 
   }
   const dim3 grid((N + MmaShape<TM>::TN - 1) / MmaShape<TM>::TN, max_tiles);
   return le::launch_chained(kernel, grid, dim3(MmaShape<TM>::THREADS), smem, stream, args...);
-}
-
-template <typename T>
-__global__ void moe_combine_kernel(T *__restrict__ out, const float *__restrict__ y, const T *__restrict__ shared_out,
-                                   const float *__restrict__ gate, const int32_t *__restrict__ ids,
-                                   const float *__restrict__ share, const T *__restrict__ h, int64_t h_stride, int experts,
-                                   int64_t n, int width, int top) {
-  le::let_successor_start();
-  le::wait_for_predecessor();
-  const int64_t i = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x;
-  if (i >= n) return;
-  const int64_t t = i / width, c = i - t * width;
-  float acc = 0.0f;
-  for (int j = 0; j < top; ++j) {
-    const int64_t p = t * top + j;
-    if (ids != nullptr && ids[p] >= experts) acc = fmaf(share != nullptr ? share[p] : 1.0f, le::to_f32(h[t * h_stride + c]), acc);
-    else acc += y[p * width + c];
-  }
-  if (shared_out != nullptr) acc = fmaf(gate != nullptr ? gate[t] : 1.0f, le::to_f32(shared_out[i]), acc);
-  out[i] = le::from_f32<T>(acc);
 }
 
 }  // namespace
@@ -667,23 +716,13 @@ LE_API int le_moe_combine_sorted(void *out, int dtype, const void *y, int y_dtyp
                                  const float *share, const void *shared_out, const float *gate, const int32_t *ids,
                                  const void *h, int64_t h_stride, int experts, int tokens, int width, int top,
                                  cudaStream_t stream) {
-  const int64_t n = static_cast<int64_t>(tokens) * width;
-  if (n <= 0) return 0;
-  const dim3 grid(static_cast<unsigned>((n + 255) / 256)), block(256);
-  if (dtype == LE_BF16 && y_dtype == LE_F32)
-    return le::launch_chained(moe_combine_sorted_kernel<__nv_bfloat16, float>, grid, block, 0, stream,
-                              static_cast<__nv_bfloat16 *>(out), static_cast<const float *>(y), pair_slot, share,
-                              static_cast<const __nv_bfloat16 *>(shared_out), gate, ids, static_cast<const __nv_bfloat16 *>(h),
-                              h_stride, experts, n, width, top);
-  if (dtype == LE_BF16 && y_dtype == LE_BF16)
-    return le::launch_chained(moe_combine_sorted_kernel<__nv_bfloat16, __nv_bfloat16>, grid, block, 0, stream,
-                              static_cast<__nv_bfloat16 *>(out), static_cast<const __nv_bfloat16 *>(y), pair_slot, share,
-                              static_cast<const __nv_bfloat16 *>(shared_out), gate, ids, static_cast<const __nv_bfloat16 *>(h),
-                              h_stride, experts, n, width, top);
-  if (dtype == LE_F32 && y_dtype == LE_F32)
-    return le::launch_chained(moe_combine_sorted_kernel<float, float>, grid, block, 0, stream, static_cast<float *>(out),
-                              static_cast<const float *>(y), pair_slot, share, static_cast<const float *>(shared_out), gate,
-                              ids, static_cast<const float *>(h), h_stride, experts, n, width, top);
+  if (tokens <= 0 || width <= 0) return 0;
+#define LE_GO(T, TY) \
+  return launch_combine<T, TY, true>(out, y, pair_slot, share, shared_out, gate, ids, h, h_stride, experts, tokens, width, top, stream)
+  if (dtype == LE_BF16 && y_dtype == LE_F32) LE_GO(__nv_bfloat16, float);
+  if (dtype == LE_BF16 && y_dtype == LE_BF16) LE_GO(__nv_bfloat16, __nv_bfloat16);
+  if (dtype == LE_F32 && y_dtype == LE_F32) LE_GO(float, float);
+#undef LE_GO
   return le::invalid("le_moe_combine_sorted: no form for output type %d and rows of type %d", dtype, y_dtype);
 }
 
@@ -746,14 +785,8 @@ LE_API int le_moe_grouped(void *out, int out_dtype, int64_t out_stride, const vo
 LE_API int le_moe_combine(void *out, int dtype, const float *y, const void *shared_out, const float *gate, const int32_t *ids,
                           const float *share, const void *h, int64_t h_stride, int experts, int tokens, int width, int top,
                           cudaStream_t stream) {
-  const int64_t n = static_cast<int64_t>(tokens) * width;
-  if (n <= 0) return 0;
-  const dim3 grid(static_cast<unsigned>((n + 255) / 256)), block(256);
-  if (dtype == LE_BF16)
-    return le::launch_chained(moe_combine_kernel<__nv_bfloat16>, grid, block, 0, stream, static_cast<__nv_bfloat16 *>(out), y,
-                              static_cast<const __nv_bfloat16 *>(shared_out), gate, ids, share,
-                              static_cast<const __nv_bfloat16 *>(h), h_stride, experts, n, width, top);
-  return le::launch_chained(moe_combine_kernel<float>, grid, block, 0, stream, static_cast<float *>(out), y,
-                            static_cast<const float *>(shared_out), gate, ids, share, static_cast<const float *>(h), h_stride,
-                            experts, n, width, top);
+  if (tokens <= 0 || width <= 0) return 0;
+  LE_DISPATCH_DTYPE(dtype, T,
+                    return launch_combine<T, float, false>(out, y, nullptr, share, shared_out, gate, ids, h, h_stride, experts,
+                                                           tokens, width, top, stream));
 }

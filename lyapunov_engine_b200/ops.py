@@ -109,10 +109,9 @@ _CORE_SIGNATURES = {
                     c_int, c_int, c_int, c_float, c_void_p],
     "le_activate": [c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_void_p],
     "le_lightning_segment": [],
-    "le_lightning_chunk": [],
-    "le_lightning_scan": [c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
+    "le_lightning_scan": [c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
                           c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
-    "le_lightning_chunks": [c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int,
+    "le_lightning_chunks": [c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_void_p, c_int,
                             c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "le_mlstm_rows": [c_int, c_int],
     "le_mlstm_scan": [c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
@@ -326,8 +325,9 @@ def swiglu(out: torch.Tensor, gate_up: torch.Tensor) -> None:
 
 
 GLU_SILU, GLU_CLAMPED, GLU_RELU = 0, 1, 2
-# activations of a product without a gate (as the second-to-last numbers of the products' ``activation``): max(v, 0)^2
-ACT_SILU, ACT_RELU_SQUARED = 0, 3
+# activations of a product without a gate (the kind in a product's ``activation``): max(v, 0)^2; silu in the first
+# ``limit`` columns
+ACT_SILU, ACT_RELU_SQUARED, ACT_SILU_COLUMNS = 0, 3, 4
 
 
 def glu(out: torch.Tensor, gate_up: torch.Tensor, kind: int = GLU_SILU, alpha: float = 1.0, limit: float = 0.0,
@@ -612,8 +612,8 @@ def gemm_skinny(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, splits: int
     ``gated``: ``w`` is [2 I, K] (gate rows, then up rows), out = act(gate, up)
     with ``activation`` = (kind, slope, limit) as glu() takes them (silu(gate) * up by default), and
     ``bias`` (float32 [2 I] or None) added to the product's columns before it.
-    Without a gate and with one split, the kind ACT_RELU_SQUARED puts that
-    activation on the product."""
+    Without a gate and with one split, the kinds ACT_RELU_SQUARED and
+    ACT_SILU_COLUMNS put that activation on the product."""
     _need_cuda(out, a, w, bias)
     M, K = a.shape
     N = w.shape[0]
@@ -671,8 +671,8 @@ def gemm_tc(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, gated: bool = F
     out = a @ w^T (bfloat16 or float32), or with ``gated`` out = act(a Wg^T,
     a Wu^T) for w = [Wg; Wu], ``activation`` = (kind, slope, limit) as glu()
     takes them (silu(g) * u by default), and ``bias`` (float32 [2 I] or None)
-    added to the product's columns before it.  Without a gate the kind
-    ACT_RELU_SQUARED puts that activation on the product."""
+    added to the product's columns before it.  Without a gate the kinds
+    ACT_RELU_SQUARED and ACT_SILU_COLUMNS put that activation on the product."""
     _need_cuda(out, a, w, bias)
     M, K = a.shape
     N = w.shape[0]
@@ -761,19 +761,24 @@ def gated_linear(out: torch.Tensor, a: torch.Tensor, w_gate_up: torch.Tensor, wo
     glu(out, gu, *activation)
 
 
-def activated_linear(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, kind: int, status=None) -> None:
-    """out = act(a @ w^T) for an activation without a gate (``kind``:
-    ACT_RELU_SQUARED).  bfloat16: one kernel of the package (weight-streaming
-    for few rows, tcgen05 for many) with the activation in its epilogue, on
-    the 32-bit sums; else the product, then the activation's kernel."""
+def activated_linear(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, kind: int, status=None, columns: int = 0) -> None:
+    """out = act(a @ w^T) for an activation without a gate: ACT_RELU_SQUARED,
+    or ACT_SILU_COLUMNS with silu in the first ``columns`` columns and the
+    product itself in the others.  bfloat16: one kernel of the package
+    (weight-streaming for few rows, tcgen05 for many) with the activation in
+    its epilogue, on the 32-bit sums; else the product, then the activation's
+    kernel."""
     if skinny_applies(a, w):
-        gemm_skinny(out, a, w, activation=(kind, 1.0, 0.0))
+        gemm_skinny(out, a, w, activation=(kind, 1.0, float(columns)))
         return
     if tc_applies(a, w):
-        gemm_tc(out, a, w, status=status, activation=(kind, 1.0, 0.0))
+        gemm_tc(out, a, w, status=status, activation=(kind, 1.0, float(columns)))
         return
     linear(out, a, w, status)
-    activate(out, out, kind)
+    if kind == ACT_SILU_COLUMNS:
+        activate(out[:, :columns], out[:, :columns], ACT_SILU)
+    else:
+        activate(out, out, kind)
 
 
 FUSE_GATED_BIAS = os.environ.get("LYAPUNOV_FUSE_GATED_BIAS", "1") not in ("0", "")
@@ -1559,20 +1564,18 @@ def lightning_segment() -> int:
     """Tokens per segment of lightning_chunks()."""
     if "segment" not in _lightning_sizes:
         _lightning_sizes["segment"] = int(core().le_lightning_segment())
-        _lightning_sizes["chunk"] = int(core().le_lightning_chunk())
     return _lightning_sizes["segment"]
 
 
 def lightning_tables(decay, device):
     """What the two forms of lightning attention need of the decays (one
     64-bit number per head): (their high and low float32 parts [2, heads],
-    their powers 0 .. chunk as float32 [heads, chunk + 1], the decays as float64)."""
-    lightning_segment()
+    their powers 0 .. segment as float32 [heads, segment + 1])."""
     d = torch.as_tensor([float(x) for x in decay], dtype=torch.float64)
     high = d.to(torch.float32)
     parts = torch.stack([high, (d - high.to(torch.float64)).to(torch.float32)])
-    powers = d[:, None] ** torch.arange(_lightning_sizes["chunk"] + 1, dtype=torch.float64)[None, :]
-    return (parts.to(device).contiguous(), powers.to(torch.float32).to(device).contiguous(), d.to(device).contiguous())
+    powers = d[:, None] ** torch.arange(lightning_segment() + 1, dtype=torch.float64)[None, :]
+    return parts.to(device).contiguous(), powers.to(torch.float32).to(device).contiguous()
 
 
 def _lightning_checks(out, rows, state, heads, dim, vdim):
@@ -1583,41 +1586,37 @@ def _lightning_checks(out, rows, state, heads, dim, vdim):
 
 
 def lightning_scan(out, rows, q_col: int, k_col: int, v_col: int, decay_parts, state, state_slots, cu_q, num_requests: int,
-                   heads: int, dim: int, vdim: int, activated: bool = False, requests=None, single: bool = False) -> None:
+                   heads: int, dim: int, vdim: int, requests=None, single: bool = False) -> None:
     """Lightning attention token by token, from each request's state row
     (``state`` float32 [rows, heads, vdim, dim]) and back into it: S <- decay S
     + k v^T, ``out`` (float32 [T, heads * vdim]) = S^T q.  ``rows``: q [heads,
-    dim] at column ``q_col``, k at ``k_col``, v [heads, vdim] at ``v_col``, each
-    before its silu (``activated``: after it).  ``requests``: indices of the
-    ``num_requests`` requests to run (None: all, in order); ``single``: each
-    brings one token."""
+    dim] at column ``q_col``, k at ``k_col``, v [heads, vdim] at ``v_col``, after
+    their activation.  ``requests``: indices of the ``num_requests`` requests
+    to run (None: all, in order); ``single``: each brings one token."""
     _need_cuda(out, rows, decay_parts, state, state_slots, cu_q, requests)
     _lightning_checks(out, rows, state, heads, dim, vdim)
     assert decay_parts.dtype == torch.float32 and tuple(decay_parts.shape) == (2, heads) and decay_parts.is_contiguous()
     _check(core().le_lightning_scan(_ptr(out), out.stride(0), _ptr(rows), rows.stride(0), q_col, k_col, v_col,
-                                    dtype_code(rows.dtype), 1 if activated else 0, _ptr(decay_parts), _ptr(state),
+                                    dtype_code(rows.dtype), _ptr(decay_parts), _ptr(state),
                                     state.shape[0], _ptr(state_slots), _ptr(cu_q), _ptr(requests), num_requests, heads, dim,
                                     vdim, 1 if single else 0, _stream()), "le_lightning_scan")
 
 
-def lightning_chunks(out, rows, q_col: int, k_col: int, v_col: int, powers, decay, state, scratch, state_slots, cu_q,
+def lightning_chunks(out, rows, q_col: int, k_col: int, v_col: int, powers, state, scratch, state_slots, cu_q,
                      tile_request, tile_q0, num_segments: int, heads: int, dim: int, vdim: int) -> None:
     """The same over chunks on the tensor cores, for the requests whose
-    segments (lightning_segment() tokens each, a request's one after the
-    other) the first ``num_segments`` entries of the tile lists name.  ``rows``
-    bfloat16, after silu.  ``powers``, ``decay``: see lightning_tables().
-    ``scratch``: float32 [num_segments, heads, vdim, dim] where a request has
+    segments (lightning_segment() tokens each, a request's in their order,
+    others' between them or not) the first ``num_segments`` entries of the tile lists name.  ``rows``
+    bfloat16.  ``powers``: see lightning_tables().  ``scratch``: float32 [num_segments, heads, vdim, dim] where a request has
     several segments, else None."""
-    _need_cuda(out, rows, powers, decay, state, scratch, state_slots, cu_q, tile_request, tile_q0)
+    _need_cuda(out, rows, powers, state, scratch, state_slots, cu_q, tile_request, tile_q0)
     _lightning_checks(out, rows, state, heads, dim, vdim)
-    lightning_segment()
     assert rows.dtype == torch.bfloat16 and dim <= LIGHTNING_CHUNK_MAX_DIM
-    assert powers.dtype == torch.float32 and tuple(powers.shape) == (heads, _lightning_sizes["chunk"] + 1)
-    assert powers.is_contiguous() and decay.dtype == torch.float64 and decay.numel() == heads
+    assert powers.dtype == torch.float32 and tuple(powers.shape) == (heads, lightning_segment() + 1) and powers.is_contiguous()
     assert scratch is None or (scratch.dtype == torch.float32 and scratch.is_contiguous()
                                and scratch.numel() >= num_segments * heads * vdim * dim)
     _check(core().le_lightning_chunks(_ptr(out), out.stride(0), _ptr(rows), rows.stride(0), q_col, k_col, v_col, _ptr(powers),
-                                      _ptr(decay), _ptr(state), state.shape[0], _ptr(scratch), _ptr(state_slots), _ptr(cu_q),
+                                      _ptr(state), state.shape[0], _ptr(scratch), _ptr(state_slots), _ptr(cu_q),
                                       _ptr(tile_request), _ptr(tile_q0), num_segments, heads, dim, vdim, _stream()),
            "le_lightning_chunks", launches=1 if scratch is None else 3)
 

@@ -7,12 +7,11 @@ With x the mixer's input, H heads, d the query/key size and e the value size:
     y = Wo ( o / sqrt(mean(o^2) + eps) * w * sigmoid(Wg x) )                   over all heads together
 
 S is carried from token to token in 32 bits, per request and head
-(``state_need``).  One product makes all four projections.  Decoded tokens (and
-whatever the tensor-core form does not take: 32-bit runs, heads of more than
-128 entries) run token by token (ops.lightning_scan, with the silu inside);
-requests that bring several tokens in bfloat16 run over chunks on the tensor
-cores (ops.lightning_chunks), after one pass that puts the silu on q, k and v in
-place.  The norm and the gate are one kernel (ops.head_norm_gate, the heads
+(``state_need``).  One product makes all four projections, with the silu of q, k
+and v in its epilogue.  Decoded tokens (and whatever the tensor-core form does
+not take: 32-bit runs, heads of more than 128 entries) run token by token
+(ops.lightning_scan); requests that bring several tokens in bfloat16 run over
+chunks on the tensor cores (ops.lightning_chunks).  The norm and the gate are one kernel (ops.head_norm_gate, the heads
 taken as one).
 """
 from __future__ import annotations
@@ -70,7 +69,7 @@ class LightningMixer(Mixer):
         self.w_in = torch.cat(rows, dim=0).contiguous()
         self.norm_weight = get(self.norm_name).contiguous()
         self.w_o = get(self.o_name)
-        self.decay_parts, self.powers, self.decay64 = ops.lightning_tables(self.decay, runtime.device)
+        self.decay_parts, self.powers = ops.lightning_tables(self.decay, runtime.device)
         if ops.lightning_segment() != SEGMENT:
             raise RuntimeError(f"the kernels' segments have {ops.lightning_segment()} tokens, the mixer lists {SEGMENT}")
         self.runtime = runtime
@@ -91,21 +90,20 @@ class LightningMixer(Mixer):
         H, d, e = self.num_heads, self.head_dim, self.value_dim
         T = x.shape[0]
         proj = ws.get("lightning_proj", (T, self.width), rt.dtype)
-        ops.linear(proj, x, self.w_in, ctx.status)
+        ops.activated_linear(proj, x, self.w_in, ops.ACT_SILU_COLUMNS, ctx.status, columns=self.gate_col)
         o = ws.get("lightning_out", (T, H * e), torch.float32)
         request, q0, _, segments = ctx.tiles[SEGMENT]
         columns = (self.q_col, self.k_col, self.v_col)
         if segments and self._in_chunks():
-            ops.activate(proj[:, :self.gate_col], proj[:, :self.gate_col], ops.ACT_SILU)
             # (a step in which no request has a second segment goes from state row to state row)
             scratch = None
             if segments > ctx.num_requests - ctx.num_decode:
                 scratch = ws.get("lightning_scratch", (segments, H, e, d), torch.float32)
-            ops.lightning_chunks(o, proj, *columns, self.powers, self.decay64, cache.state, scratch, ctx.state_slots, ctx.cu_q,
-                                 request, q0, segments, H, d, e)
+            ops.lightning_chunks(o, proj, *columns, self.powers, cache.state, scratch, ctx.state_slots, ctx.cu_q, request, q0,
+                                 segments, H, d, e)
             if ctx.num_decode:
                 ops.lightning_scan(o, proj, *columns, self.decay_parts, cache.state, ctx.state_slots, ctx.cu_q, ctx.num_decode,
-                                   H, d, e, activated=True, requests=ctx.decode_requests, single=True)
+                                   H, d, e, requests=ctx.decode_requests, single=True)
         else:
             ops.lightning_scan(o, proj, *columns, self.decay_parts, cache.state, ctx.state_slots, ctx.cu_q, ctx.num_requests,
                                H, d, e, single=ctx.max_q_len == 1)

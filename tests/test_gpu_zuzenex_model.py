@@ -79,8 +79,15 @@ CONFIGS = {
     "d": (config(130, 100, [attention(3, 1, 21, 10, 0.4, (0.3, 5), moe(36, 3, 1, 2, 20)),
                             lightning(11, 7, (0.9, 0.99, 0.6), moe(42, 2, 2, 1, 0))], loop=(0, 2, 2)), 8),
 }
-LENGTHS = {"a": (23, 47, 75, 141), "b": (9, 70, 35, 101), "c": (40, 130, 601, 215), "d": (12, 66, 31, 90)}
-PROMPTS = {"a": (3, 30, 41, 100), "b": (1, 64, 2, 67), "c": (8, 128, 560, 101), "d": (2, 40, 30, 51)}
+CONFIGS["e"] = (
+    # no router, so that no rounding can flip a choice and every place is held to the tight bounds in bfloat16 too;
+    # sizes that are padded (lightning heads of 80 and 48, attention heads of 56 beside values of 64), several segments
+    config(256, 160, [lightning(80, 96, (0.97, 0.9993), dense(224)),
+                      attention(4, 2, 56, 64, 0.15, (0.3, 100), dense(320)),
+                      lightning(48, 64, (0.6, 0.99, 0.998), None),
+                      attention(3, 3, 32, 48, 0.25, None, dense(96))], loop=(1, 3, 2)), 16)
+LENGTHS = {"a": (23, 47, 75, 141), "b": (9, 70, 35, 101), "c": (40, 130, 601, 215), "d": (12, 66, 31, 90), "e": (70, 150, 580, 310)}
+PROMPTS = {"a": (3, 30, 41, 100), "b": (1, 64, 2, 67), "c": (8, 128, 560, 101), "d": (2, 40, 30, 51), "e": (50, 129, 540, 290)}
 
 
 def write_folder(folder, cfg, weights, dtype):
@@ -113,7 +120,7 @@ def models(tmp_path_factory):
                              LENGTHS[name], PROMPTS[name]) for name, (cfg, page) in CONFIGS.items()}
 
 
-CLOSE_CALL = 0.002      # choice scores nearer than this: rounding to bfloat16 may choose either expert
+CLOSE_CALL = 0.01      # choice scores nearer than this: rounding to bfloat16 may choose either expert
 
 
 def close_calls(cfg, weights, ids):
@@ -138,13 +145,14 @@ def check(m, trace, dtype, out_dir, pool=None, what="", extra=()):
     is as far off, and the place is measured from that run instead; places
     at or behind a router's close call are left out of this bound: no
     comparison rests on which way such a call falls), and no more loud places
-    than twice what the plain implementation's own rounded run has."""
+    than twice what the plain implementation's own rounded run has (the same
+    places left out; of all places a tenth at most)."""
     pool = pool or sum((len(v) + 63) // 64 * 64 for v in m["requests"].values())
     got = ru.run_trace(trace, m["folders"][dtype], dtype, str(out_dir), pool, m["page"], extra=extra)
     assert len(got) == sum(len(w) for w in trace.wanted)
     if dtype == "float32":
         return ru.compare(got, {r: v.float() for r, v in m["exact"].items()}, atol=3e-4, rtol=3e-4, what=what)
-    units, own, near = [], [], []
+    units, own, near, clear = [], [], [], []
     close = m.setdefault("close", {})
     for (rid, p), row in sorted(got.items()):
         assert np.all(np.isfinite(row))
@@ -153,12 +161,14 @@ def check(m, trace, dtype, out_dir, pool=None, what="", extra=()):
         d = row.astype(np.float64) - m["exact"][rid][p].numpy()
         units.append(float(np.sqrt(np.mean(d * d))) / m["noise"])
         own.append(float((m["rounded"][rid][p] - m["exact"][rid][p]).pow(2).mean().sqrt()) / m["noise"])
+        clear.append(not close[rid][p])
         d = row.astype(np.float64) - m["rounded"][rid][p].numpy()
         near.append(0.0 if close[rid][p] else min(units[-1], float(np.sqrt(np.mean(d * d))) / m["noise"]))
     worst = int(np.argmax(near))
     assert near[worst] <= 30.0, f"{what}: place {sorted(got)[worst]}: {near[worst]:.1f} units of rounding noise"
     assert float(np.median(units)) <= 1.5, f"{what}: the median place lies {np.median(units):.2f} units of rounding noise off"
-    loud, loud_own = sum(u > 4.0 for u in units), sum(u > 4.0 for u in own)
+    assert sum(u > 4.0 for u in units) <= 2 * sum(u > 4.0 for u in own) + max(2, len(units) // 10), what
+    loud, loud_own = (sum(u > 4.0 and c for u, c in zip(us, clear)) for us in (units, own))
     assert loud <= 2 * loud_own + max(2, len(units) // 50), \
         f"{what}: {loud} of {len(units)} places above 4 units of rounding noise (the plain rounded run: {loud_own})"
     return float(np.median(units))
@@ -242,10 +252,12 @@ def test_mixed_batches_on_a_pool_that_is_used_again(models, name, dtype, tmp_pat
     assert pages["allocations"] > pages["pool_pages"] and pages["reuses"] > 0, pages
 
 
-def test_a_batch_of_unequal_requests_against_each_alone(models, tmp_path):
+@pytest.mark.parametrize("name", ["c", "e"])
+def test_a_batch_of_unequal_requests_against_each_alone(models, name, tmp_path):
     """Four requests whose portions have 1 to 300 tokens in one step (segments
-    of one request beside single tokens of others): the logits of each alone."""
-    m = models["c"]
+    of one request beside single tokens of others, and the list of segments goes from one request to
+    another and back): the logits of each alone."""
+    m = models[name]
     requests = m["requests"]
     trace, at = ru.Trace(), {r: 0 for r in requests}
     for sizes in ((300, 2, 40, 1), (1, 128, 1, 257), (258, 1, 100, 5), (42, 84, 3, 3)):
@@ -257,7 +269,7 @@ def test_a_batch_of_unequal_requests_against_each_alone(models, tmp_path):
                 at[r] += n
         trace.step(entries)
     for dtype in ("float32", "bfloat16"):
-        check(m, trace, dtype, tmp_path / dtype, what=f"unequal {dtype}")
+        check(m, trace, dtype, tmp_path / dtype, what=f"{name} unequal {dtype}")
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])

@@ -44,7 +44,7 @@ def run_in_cuts(seqs, cuts, state_rows, H, d, e, decay, dtype, chunks, poison=7.
     requests of a step as one batch; requests take the lowest free state row
     and give it back when they end.  Returns their outputs and the last states."""
     from lyapunov_engine_b200 import ops
-    parts, powers, decay64 = ops.lightning_tables(decay, DEV)
+    parts, powers = ops.lightning_tables(decay, DEV)
     state = torch.full((state_rows + 1, H, e, d), poison, device=DEV)     # (the last row belongs to nobody)
     q_col, k_col, v_col = 0, H * d, 2 * H * d
     free, slot_of, at = list(range(state_rows)), {}, [0] * len(seqs)
@@ -59,17 +59,19 @@ def run_in_cuts(seqs, cuts, state_rows, H, d, e, decay, dtype, chunks, poison=7.
                 state[slot_of[r]].zero_()
         q_lens = [cuts[r][step] for r in live]
         rows = torch.cat([seqs[r][at[r]:at[r] + n] for r, n in zip(live, q_lens)]).to(dtype).to(DEV)
+        ops.activate(rows[:, :v_col + H * e], rows[:, :v_col + H * e], ops.ACT_SILU)
         out = torch.full((rows.shape[0], H * e), -5.0, device=DEV)
         cu, slots = i32([0] + torch.tensor(q_lens).cumsum(0).tolist()), i32(slot_of[r] for r in live)
         multi = [b for b, n in enumerate(q_lens) if n > 1]
         single = [b for b, n in enumerate(q_lens) if n == 1]
         if chunks and multi:
-            ops.activate(rows[:, :v_col + H * e], rows[:, :v_col + H * e], ops.ACT_SILU)
-            tr, tq, n = tiles(q_lens, seg, only=multi)
+            # the order of a step's list: by the keys a tile of attention sees, the requests' segments between one another
+            listed = sorted(((b, s) for b in multi for s in range(0, q_lens[b], seg)), key=lambda x: at[live[x[0]]] + x[1])
+            tr, tq, n = i32(b for b, _ in listed), i32(s for _, s in listed), len(listed)
             scratch = torch.full((n, H, e, d), 3.0, device=DEV) if n > len(multi) else None
-            ops.lightning_chunks(out, rows, q_col, k_col, v_col, powers, decay64, state, scratch, slots, cu, tr, tq, n, H, d, e)
+            ops.lightning_chunks(out, rows, q_col, k_col, v_col, powers, state, scratch, slots, cu, tr, tq, n, H, d, e)
             if single:
-                ops.lightning_scan(out, rows, q_col, k_col, v_col, parts, state, slots, cu, len(single), H, d, e, activated=True,
+                ops.lightning_scan(out, rows, q_col, k_col, v_col, parts, state, slots, cu, len(single), H, d, e,
                                    requests=i32(single), single=True)
         else:
             ops.lightning_scan(out, rows, q_col, k_col, v_col, parts, state, slots, cu, len(live), H, d, e,
@@ -111,11 +113,11 @@ SHAPES = [
     (2, 13, 9, [0.8, 0.99]),                   # no 16-byte pieces
     (1, 64, 200, [0.98]),
 ]
-LENS = (700, 70, 1, 131)
-CUTS = [((700,), (70,), (1,), (131,)),
-        ((1, 2, 61, 64, 65, 257, 250), (2,) * 35, (1,), (128, 1, 2)),
-        ((256, 256, 188), (1,) * 70, (1,), (63, 1, 1, 66)),
-        ((513, 1, 1, 185), (64, 1, 5), (1,), (3, 128))]
+LENS = (700, 70, 1, 531)
+CUTS = [((700,), (70,), (1,), (531,)),
+        ((1, 2, 61, 64, 65, 257, 250), (2,) * 35, (1,), (128, 1, 2, 400)),
+        ((256, 256, 188), (1,) * 70, (1,), (463, 1, 1, 66)),
+        ((513, 1, 1, 185), (64, 1, 5), (1,), (3, 528))]
 
 
 @pytest.mark.parametrize("cut", range(len(CUTS)))
@@ -176,7 +178,7 @@ def test_requests_without_a_state_row_leave_everything_alone():
     """Slot -1 (padding of a fixed-shape step): zeros out, no state touched."""
     from lyapunov_engine_b200 import ops
     H, d, e = 2, 16, 24
-    parts, powers, decay64 = ops.lightning_tables([0.9, 0.5], DEV)
+    parts, _ = ops.lightning_tables([0.9, 0.5], DEV)
     state = torch.full((3, H, e, d), 4.0, device=DEV)
     rows = torch.randn(4, 2 * H * d + H * e, device=DEV).to(torch.bfloat16)
     out = torch.full((4, H * e), 9.0, device=DEV)
@@ -376,6 +378,22 @@ def test_relu_squared_in_the_products_epilogue(rows, width, inner, dtype):
     want = pz.relu_squared(x.double() @ w.double().T)
     torch.testing.assert_close(out.double().cpu(), want, **tol_of(dtype, tight=5e-5))
     assert float((out == 0).float().mean()) > 0.3                      # (about half of the products are negative)
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("rows,width,inner,columns", [(1, 64, 48, 32), (12, 128, 96, 96), (20, 256, 200, 1), (300, 192, 520, 390),
+                                                      (5, 50, 33, 20), (600, 512, 1024, 700)])
+def test_silu_on_the_first_columns_of_a_product(rows, width, inner, columns, dtype):
+    from lyapunov_engine_b200 import ops
+    g = torch.Generator().manual_seed(rows)
+    x, w = torch.randn(rows, width, generator=g).to(dtype), (torch.randn(inner, width, generator=g) / math.sqrt(width)).to(dtype)
+    out = torch.zeros(rows, inner, dtype=dtype, device=DEV)
+    status = ops.new_status(DEV)
+    ops.activated_linear(out, x.to(DEV), w.to(DEV), ops.ACT_SILU_COLUMNS, status, columns=columns)
+    ops.check_status(status)
+    z = x.double() @ w.double().T
+    want = torch.cat([pz.silu(z[:, :columns]), z[:, columns:]], dim=1)
+    torch.testing.assert_close(out.double().cpu(), want, **tol_of(dtype, tight=5e-5))
 
 
 # ------------------------------------------------------------------ router, experts, identity experts
