@@ -2091,7 +2091,7 @@ def zuzenex_kernel_rows(pk, llama):
         x = [torch.randn(T, W, device=dev).to(bf) for _ in range(4)]
         w_in = torch.randn(width, W, device=dev).to(bf) * 0.02
         p_out = torch.empty(T, width, device=dev, dtype=bf)
-        row("projections, silu on q, k and v in the epilogue", "the library's product (or the weight-streaming one)", T,
+        row("projections with silu on q, k and v", "the product alone", T,
             2 * (width * W + T * W + T * width),
             lambda i: ops.activated_linear(p_out, x[i], w_in, ops.ACT_SILU_COLUMNS, status, columns=2 * H * d + H * e), 4, flops=2 * T * width * W)
         row("projections alone", "", T, 2 * (width * W + T * W + T * width), lambda i: ops.linear(p_out, x[i], w_in, status), 4,
@@ -2100,7 +2100,7 @@ def zuzenex_kernel_rows(pk, llama):
         # the shared expert's first product
         wu = [torch.randn(F, W, device=dev).to(bf) * 0.02 for _ in range(4)]
         act = torch.empty(T, F, device=dev, dtype=bf)
-        row("product with relu squared in its epilogue", "gate/up product, silu", T, 2 * (F * W + T * W + T * F),
+        row("product with relu squared", "gate/up product, silu", T, 2 * (F * W + T * W + T * F),
             lambda i: ops.activated_linear(act, x[i], wu[i], ops.ACT_RELU_SQUARED, status), 4, flops=2 * T * F * W)
         Fg = F * 2 // 3
         wg = [torch.randn(2 * Fg, W, device=dev).to(bf) * 0.02 for _ in range(4)]

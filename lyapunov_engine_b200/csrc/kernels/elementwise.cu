@@ -134,6 +134,8 @@ __device__ __forceinline__ T activated(T x, int kind) {
     const float r = fmaxf(v, 0.0f);
     return le::from_f32<T>(r * r);
   }
+  // (bfloat16: a few units of error in 32 bits do not show behind the rounding, and the pass is bound by its arithmetic)
+  if constexpr (sizeof(T) == 2) return le::from_f32<T>(__fdividef(v, 1.0f + __expf(-v)));
   return le::from_f32<T>(v / (1.0f + expf(-v)));
 }
 template <typename T, int VEC>

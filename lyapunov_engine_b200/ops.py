@@ -764,14 +764,16 @@ def gated_linear(out: torch.Tensor, a: torch.Tensor, w_gate_up: torch.Tensor, wo
 def activated_linear(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, kind: int, status=None, columns: int = 0) -> None:
     """out = act(a @ w^T) for an activation without a gate: ACT_RELU_SQUARED,
     or ACT_SILU_COLUMNS with silu in the first ``columns`` columns and the
-    product itself in the others.  bfloat16: one kernel of the package
-    (weight-streaming for few rows, tcgen05 for many) with the activation in
-    its epilogue, on the 32-bit sums; else the product, then the activation's
-    kernel."""
-    if skinny_applies(a, w):
+    product itself in the others.  bfloat16 with few rows: the
+    weight-streaming kernel with the activation in its epilogue, on the 32-bit
+    sums.  Else the product (linear()), then the activation's kernel in place:
+    with more rows the library's product and that pass together take less time
+    than the package's tcgen05 product with the activation in its epilogue
+    (LYAPUNOV_TC_PLAIN=1 takes that one)."""
+    if skinny_applies(a, w, SKINNY_NARROW_ROWS):
         gemm_skinny(out, a, w, activation=(kind, 1.0, float(columns)))
         return
-    if tc_applies(a, w):
+    if TC_PLAIN_PRODUCTS and tc_applies(a, w):
         gemm_tc(out, a, w, status=status, activation=(kind, 1.0, float(columns)))
         return
     linear(out, a, w, status)

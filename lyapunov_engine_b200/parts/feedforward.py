@@ -91,7 +91,7 @@ class GatedFeedForward(FeedForward):
 @register_feed_forward("relu_squared")
 class PlainFeedForward(FeedForward):
     """down(act(up x)) without a gate and without biases; the activation is
-    taken in 32 bits in the first product's epilogue and rounded once."""
+    taken in 32 bits (see ops.activated_linear)."""
     activation = ops.ACT_RELU_SQUARED
 
     def __init__(self, hidden_size: int, intermediate_size: int, up_name: str, down_name: str):

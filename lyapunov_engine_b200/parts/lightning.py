@@ -7,8 +7,8 @@ With x the mixer's input, H heads, d the query/key size and e the value size:
     y = Wo ( o / sqrt(mean(o^2) + eps) * w * sigmoid(Wg x) )                   over all heads together
 
 S is carried from token to token in 32 bits, per request and head
-(``state_need``).  One product makes all four projections, with the silu of q, k
-and v in its epilogue.  Decoded tokens (and whatever the tensor-core form does
+(``state_need``).  One product makes all four projections, and silu on q, k and
+v comes with it (ops.activated_linear).  Decoded tokens (and whatever the tensor-core form does
 not take: 32-bit runs, heads of more than 128 entries) run token by token
 (ops.lightning_scan); requests that bring several tokens in bfloat16 run over
 chunks on the tensor cores (ops.lightning_chunks).  The norm and the gate are one kernel (ops.head_norm_gate, the heads

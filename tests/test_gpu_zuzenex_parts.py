@@ -5,8 +5,8 @@ chunks under every cut of a sequence into steps, with state rows used again and
 a far token that decides; sinks on all attention kernels with scores made so
 that the sink matters; the norm per head with the query temperature and the
 cache write; two outputs that enter the stream beside one another in the norm's
-kernel; the norm over all heads at once; products with relu squared in their
-epilogue; the router's corrected choice; experts without a gate and identity
+kernel; the norm over all heads at once; products with relu squared
+or silu on some of their columns; the router's corrected choice; experts without a gate and identity
 experts."""
 import math
 
@@ -377,6 +377,10 @@ def test_relu_squared_in_the_products_epilogue(rows, width, inner, dtype):
     ops.check_status(status)
     want = pz.relu_squared(x.double() @ w.double().T)
     torch.testing.assert_close(out.double().cpu(), want, **tol_of(dtype, tight=5e-5))
+    if dtype == torch.bfloat16 and ops.tc_applies(x.to(DEV), w.to(DEV)):        # the activation in the tcgen05 product's epilogue
+        ops.gemm_tc(out, x.to(DEV), w.to(DEV), status=status, activation=(ops.ACT_RELU_SQUARED, 1.0, 0.0))
+        ops.check_status(status)
+        torch.testing.assert_close(out.double().cpu(), want, **tol_of(dtype))
     assert float((out == 0).float().mean()) > 0.3                      # (about half of the products are negative)
 
 
@@ -394,6 +398,10 @@ def test_silu_on_the_first_columns_of_a_product(rows, width, inner, columns, dty
     z = x.double() @ w.double().T
     want = torch.cat([pz.silu(z[:, :columns]), z[:, columns:]], dim=1)
     torch.testing.assert_close(out.double().cpu(), want, **tol_of(dtype, tight=5e-5))
+    if dtype == torch.bfloat16 and ops.tc_applies(x.to(DEV), w.to(DEV)):
+        ops.gemm_tc(out, x.to(DEV), w.to(DEV), status=status, activation=(ops.ACT_SILU_COLUMNS, 1.0, float(columns)))
+        ops.check_status(status)
+        torch.testing.assert_close(out.double().cpu(), want, **tol_of(dtype))
 
 
 # ------------------------------------------------------------------ router, experts, identity experts
