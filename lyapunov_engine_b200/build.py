@@ -48,7 +48,7 @@ CORE_KERNEL_SOURCES = ["kernels/elementwise.cu", "kernels/norm.cu", "kernels/rop
                        "kernels/short_conv.cu", "kernels/kv_store.cu", "kernels/gemm_heads.cu", "kernels/streams.cu",
                        "kernels/rope_pairs.cu", "kernels/moe.cu", "kernels/delta_rule.cu", "kernels/rope_norm.cu",
                        "kernels/residual.cu", "kernels/state_space.cu", "kernels/mlstm.cu", "kernels/rope_qknorm.cu",
-                       "kernels/lightning.cu"]
+                       "kernels/lightning.cu", "kernels/conv_turn.cu", "kernels/addend_norm.cu"]
 ATTENTION_SOURCES = ["kernels/attention_generic.cu", "kernels/attention_mma.cu", "kernels/attention_tc.cu"]
 
 _lock = threading.Lock()

@@ -10,11 +10,17 @@ constexpr int GR_ROWS = 8;      // rows of a a block takes (blockIdx.z walks the
 constexpr int GR_COLS = 4;      // output columns per warp
 constexpr int GR_WARPS = 4;
 
+// Where the heads lie in a row and what gates them.
+struct Heads {
+  int64_t a_head, out_head;     // elements between two heads of a row of a / of out (at least K / N)
+  int gate_entries;             // the gate has a number per head (0) or per entry: head h's at columns h * N ..
+};
+
 // The work of one block of the few-rows form (blockIdx.x: 16 output columns, blockIdx.y: the head, blockIdx.z: 8 rows).
 template <typename T>
 __device__ __forceinline__ void gemm_heads_rows_block(T *__restrict__ out, int64_t out_stride, const T *__restrict__ a,
                                                       int64_t a_stride, const T *__restrict__ w, const T *__restrict__ gate,
-                                                      int64_t gate_stride, int M, int N, int K) {
+                                                      int64_t gate_stride, int M, int N, int K, const Heads &at) {
   constexpr int VEC = 16 / sizeof(T);
   const int head = blockIdx.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -48,7 +54,7 @@ __device__ __forceinline__ void gemm_heads_rows_block(T *__restrict__ out, int64
 #pragma unroll
     for (int r = 0; r < GR_ROWS; ++r) {
       if (r < rows) {
-        const uint4 raw = *reinterpret_cast<const uint4 *>(a + (m0 + r) * a_stride + static_cast<int64_t>(head) * K + k);
+        const uint4 raw = *reinterpret_cast<const uint4 *>(a + (m0 + r) * a_stride + head * at.a_head + k);
         const T *e = reinterpret_cast<const T *>(&raw);
 #pragma unroll
         for (int v = 0; v < VEC; ++v) {
@@ -66,11 +72,14 @@ __device__ __forceinline__ void gemm_heads_rows_block(T *__restrict__ out, int64
   if (lane < GR_COLS && n0 + lane < N) {
     for (int r = 0; r < rows; ++r) {
       float g = 1.0f;
-      if (gate) g = 1.0f / (1.0f + expf(-le::to_f32(gate[(m0 + r) * gate_stride + head])));
+      if (gate) {
+        const int64_t i = (m0 + r) * gate_stride + (at.gate_entries ? static_cast<int64_t>(head) * N + n0 + lane : head);
+        g = 1.0f / (1.0f + expf(-le::to_f32(gate[i])));
+      }
       float v = acc[r][0];
 #pragma unroll
       for (int c = 1; c < GR_COLS; ++c) v = lane == c ? acc[r][c] : v;
-      out[(m0 + r) * out_stride + static_cast<int64_t>(head) * N + n0 + lane] = le::from_f32<T>(v * g);
+      out[(m0 + r) * out_stride + head * at.out_head + n0 + lane] = le::from_f32<T>(v * g);
     }
   }
 }

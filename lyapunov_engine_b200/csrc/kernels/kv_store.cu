@@ -11,13 +11,15 @@
 // [pages, 1, page, padded_rank]; columns from `rank` on are written as zeros.
 // That pool serves as keys and as values of an attention over the latents.
 //
-// latent_prepare (few rows, a decode step): latent_norm_store and the
+// latent_prepare (few rows, a decode step): the latent's norm and store, the
+// turns of rotated parts of keys and queries where there are any, and the
 // per-head products that carry each head's query into the latent space, in one
-// launch: both read the projection's rows and neither reads the other's
+// launch: all read the projection's rows and none reads another's
 // result.  Blocks whose blockIdx.y is below `heads` do the products, those at
-// blockIdx.y == heads walk the tokens.
-#include "common.cuh"
+// blockIdx.y == heads walk the tokens' latents, those behind them the queries'
+// turns.
 #include "gemm_heads_rows.cuh"
+#include "latent_token.cuh"
 
 namespace {
 
@@ -47,67 +49,43 @@ __global__ void kv_store_kernel(const T *__restrict__ src, int64_t src_stride, i
   }
 }
 
-// One token's latent: norm and store (the whole block works on it).
 template <typename T>
-__device__ __forceinline__ void latent_norm_store_token(int t, float *scratch, const T *__restrict__ src, int64_t src_stride,
-                                                        int col, int rank, int padded_rank, const float *__restrict__ weight,
-                                                        float eps, T *__restrict__ cache, const int32_t *__restrict__ positions,
-                                                        const int32_t *__restrict__ request_of_token,
-                                                        const int32_t *__restrict__ block_table, int max_blocks, int page_size,
-                                                        int num_pages, int *__restrict__ status) {
-  const int pos = positions[t];
-  const int b = request_of_token[t];
-  const int page = pos >= 0 ? block_table[static_cast<int64_t>(b) * max_blocks + pos / page_size] : -1;
-  const bool bad = page < 0 || page >= num_pages;
-  if (bad && threadIdx.x == 0) atomicOr(status, LE_STATUS_BAD_PAGE);
-  const T *x = src + static_cast<int64_t>(t) * src_stride + col;
-  float ss = 0.0f;
-  for (int i = threadIdx.x; i < rank; i += blockDim.x) {
-    const float v = le::to_f32(x[i]);
-    ss += v * v;
-  }
-  ss = le::block_sum(ss, scratch);
-  if (bad) return;
-  const float inv = rsqrtf(ss / static_cast<float>(rank) + eps);
-  T *dst = cache + (static_cast<int64_t>(page) * page_size + pos % page_size) * padded_rank;
-  for (int i = threadIdx.x; i < padded_rank; i += blockDim.x)
-    dst[i] = i < rank ? le::from_f32<T>(le::to_f32(x[i]) * inv * weight[i]) : le::from_f32<T>(0.0f);
-}
-
-template <typename T>
-__global__ void latent_norm_store_kernel(const T *__restrict__ src, int64_t src_stride, int col, int rank, int padded_rank,
-                                         const float *__restrict__ weight, float eps, T *__restrict__ cache,
-                                         const int32_t *__restrict__ positions,
-                                         const int32_t *__restrict__ request_of_token,
-                                         const int32_t *__restrict__ block_table, int max_blocks, int page_size,
-                                         int num_pages, int *__restrict__ status) {
+__global__ void latent_norm_store_kernel(const le_latent::Args<T> a) {
   __shared__ float scratch[33];
   le::let_successor_start();
   le::wait_for_predecessor();
-  latent_norm_store_token<T>(blockIdx.x, scratch, src, src_stride, col, rank, padded_rank, weight, eps, cache, positions,
-                             request_of_token, block_table, max_blocks, page_size, num_pages, status);
+  le_latent::store_latent(a, blockIdx.x, nullptr, scratch);
 }
 
 template <typename T>
 __global__ void __launch_bounds__(le_heads::GR_WARPS * 32)
-latent_prepare_kernel(const T *__restrict__ src, int64_t src_stride, int num_tokens, int heads, int head_dim,
-                      const T *__restrict__ w_into, T *__restrict__ q_latent, int64_t q_latent_stride, int col, int rank,
-                      int padded_rank, const float *__restrict__ weight, float eps, T *__restrict__ cache,
-                      const int32_t *__restrict__ positions, const int32_t *__restrict__ request_of_token,
-                      const int32_t *__restrict__ block_table, int max_blocks, int page_size, int num_pages,
-                      int *__restrict__ status) {
+latent_prepare_kernel(const le_latent::Args<T> a, int num_tokens, int head_dim, const T *__restrict__ w_into) {
   __shared__ float scratch[33];
+  __shared__ float2 turn[le_latent::MAX_PAIRS];
   le::let_successor_start();
-  if (static_cast<int>(blockIdx.y) < heads) {
-    le_heads::gemm_heads_rows_block<T>(q_latent, q_latent_stride, src, src_stride, w_into, static_cast<const T *>(nullptr), 0,
-                                       num_tokens, padded_rank, head_dim);
+  const int part = static_cast<int>(blockIdx.y) - a.heads;
+  if (part < 0) {
+    // (with a rotated part the product ends at the latent's own columns; without one w_into has rows for the padding too)
+    const int N = a.rot > 0 ? a.rank : a.padded;
+    le_heads::gemm_heads_rows_block<T>(a.q_out, a.q_stride, a.src, a.src_stride, w_into, static_cast<const T *>(nullptr), 0,
+                                       num_tokens, N, head_dim, le_heads::Heads{head_dim + a.rot, a.padded, 0});
     return;
   }
-  le::wait_for_predecessor();
-  if (cache == nullptr) return;
-  for (int t = blockIdx.z * gridDim.x + blockIdx.x; t < num_tokens; t += gridDim.x * gridDim.z)
-    latent_norm_store_token<T>(t, scratch, src, src_stride, col, rank, padded_rank, weight, eps, cache, positions,
-                               request_of_token, block_table, max_blocks, page_size, num_pages, status);
+  const bool waits = a.rot == 0;
+  if (waits) le::wait_for_predecessor();
+  if (part == 0 && a.cache == nullptr) return;
+  bool waited = waits;
+  for (int t = blockIdx.z * gridDim.x + blockIdx.x; t < num_tokens; t += gridDim.x * gridDim.z) {
+    if (a.rot > 0) {
+      __syncthreads();             // (the last token's turns are done with)
+      le_latent::make_turns(turn, a, t);
+      if (!waited) le::wait_for_predecessor();
+      waited = true;
+      __syncthreads();
+    }
+    if (part == 0) le_latent::store_latent(a, t, turn, scratch);
+    else le_latent::turn_queries(a, t, turn);
+  }
 }
 
 }  // namespace
@@ -129,27 +107,32 @@ LE_API int le_kv_store(const void *src, int64_t src_stride, int k_col, int v_col
 }
 
 // For at most 32 rows.  src: the projection's rows (stride src_stride, 16-byte aligned): head h's query at columns
-// h * head_dim .., the latent at columns col .. col + rank.  q_latent[t, h, :] = w_into[h] @ query (w_into:
-// [heads, padded_rank, head_dim]); the latent is normed and stored as le_latent_norm_store does (cache null: not stored).
+// h * (head_dim + rot) .., head_dim plain entries and rot turned ones; the latent at columns col .. col + rank and its
+// rotated part behind it.  q_latent[t, h, :] = w_into[h] @ plain part (w_into: [heads, padded_rank, head_dim], or [heads,
+// rank, head_dim] where rot > 0) with the turned part behind the rank columns; the latent is normed and stored as
+// le_latent_norm_store (rot 0) or le_latent_rope_store does (cache null: not stored).
 LE_API int le_latent_prepare(const void *src, int64_t src_stride, int num_tokens, int heads, int head_dim, const void *w_into,
-                             void *q_latent, int64_t q_latent_stride, int col, int rank, int padded_rank, const float *weight,
-                             float eps, void *cache, int dtype, const int32_t *positions, const int32_t *request_of_token,
-                             const int32_t *block_table, int max_blocks, int page_size, int num_pages, int *status,
-                             cudaStream_t stream) {
+                             void *q_latent, int64_t q_latent_stride, int col, int rank, int rot, int padded_rank,
+                             const float *weight, float eps, const double *rates, float magnitude, void *cache, int dtype,
+                             const int32_t *positions, const int32_t *request_of_token, const int32_t *block_table,
+                             int max_blocks, int page_size, int num_pages, int *status, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
   const int vec = dtype == LE_BF16 ? 8 : 4;
-  if (num_tokens > 32 || head_dim % vec || src_stride % vec || heads < 1 || heads >= 65535 ||
+  if (num_tokens > 32 || head_dim % vec || rot % vec || src_stride % vec || heads < 1 || heads >= 65530 ||
       ((reinterpret_cast<uintptr_t>(src) | reinterpret_cast<uintptr_t>(w_into)) & 15))
     return le::invalid("le_latent_prepare: at most 32 rows, 16-byte aligned rows and head sizes");
-  if (rank < 1 || padded_rank < rank) return le::invalid("le_latent_prepare: rank %d, padded rank %d", rank, padded_rank);
-  const dim3 grid((padded_rank + le_heads::GR_WARPS * le_heads::GR_COLS - 1) / (le_heads::GR_WARPS * le_heads::GR_COLS), heads + 1,
-                  (num_tokens + le_heads::GR_ROWS - 1) / le_heads::GR_ROWS);
-  LE_DISPATCH_DTYPE(dtype, T,
-                    return le::launch_chained(latent_prepare_kernel<T>, grid, dim3(le_heads::GR_WARPS * 32), 0, stream,
-                                              static_cast<const T *>(src), src_stride, num_tokens, heads, head_dim,
-                                              static_cast<const T *>(w_into), static_cast<T *>(q_latent), q_latent_stride, col,
-                                              rank, padded_rank, weight, eps, static_cast<T *>(cache), positions,
-                                              request_of_token, block_table, max_blocks, page_size, num_pages, status));
+  if (rank < 1 || rot < 0 || rot > 2 * le_latent::MAX_PAIRS || padded_rank < rank + rot)
+    return le::invalid("le_latent_prepare: rank %d, %d turned entries, padded %d", rank, rot, padded_rank);
+  const dim3 grid((padded_rank + le_heads::GR_WARPS * le_heads::GR_COLS - 1) / (le_heads::GR_WARPS * le_heads::GR_COLS),
+                  heads + (rot > 0 ? 2 : 1), (num_tokens + le_heads::GR_ROWS - 1) / le_heads::GR_ROWS);
+  LE_DISPATCH_DTYPE(dtype, T, {
+    le_latent::Args<T> a{static_cast<const T *>(src), src_stride, col, rank, rot, padded_rank, weight, eps, rates, magnitude,
+                         static_cast<T *>(cache), positions, request_of_token, block_table, max_blocks, page_size, num_pages,
+                         status, head_dim, head_dim + rot, heads, static_cast<T *>(q_latent), q_latent_stride, 0};
+    a.q_pairs = le_latent::pairs_together(a);
+    return le::launch_chained(latent_prepare_kernel<T>, grid, dim3(le_heads::GR_WARPS * 32), 0, stream, a, num_tokens, head_dim,
+                              static_cast<const T *>(w_into));
+  });
 }
 
 // src: rows of stride src_stride with the latent at columns col .. col + rank; cache: [pages, 1, page, padded_rank].
@@ -160,9 +143,10 @@ LE_API int le_latent_norm_store(const void *src, int64_t src_stride, int col, in
   if (num_tokens <= 0) return 0;
   if (rank < 1 || padded_rank < rank) return le::invalid("le_latent_norm_store: rank %d, padded rank %d", rank, padded_rank);
   const int threads = rank >= 512 ? 256 : 128;
-  LE_DISPATCH_DTYPE(dtype, T,
-                    return le::launch_chained(latent_norm_store_kernel<T>, dim3(num_tokens), dim3(threads), 0, stream,
-                                              static_cast<const T *>(src), src_stride, col, rank, padded_rank, weight, eps,
-                                              static_cast<T *>(cache), positions, request_of_token, block_table,
-                                              max_blocks, page_size, num_pages, status));
+  LE_DISPATCH_DTYPE(dtype, T, {
+    const le_latent::Args<T> a{static_cast<const T *>(src), src_stride, col, rank, 0, padded_rank, weight, eps, nullptr, 1.0f,
+                               static_cast<T *>(cache), positions, request_of_token, block_table, max_blocks, page_size,
+                               num_pages, status, 0, 0, 0, nullptr, 0, 0};
+    return le::launch_chained(latent_norm_store_kernel<T>, dim3(num_tokens), dim3(threads), 0, stream, a);
+  });
 }

@@ -17,17 +17,21 @@
 // receives the keys as projected (before turn and norm) when
 // `values_are_keys`, the value heads [kv_heads][head_dim] behind the keys as
 // they are when `store_values`, else nothing.  A warp takes a head, a lane up to eight
-// pairs of it; a token's sines and cosines are made once per block.  Angle,
-// sine, cosine, turn and norm are 32-bit; the result is rounded once.
+// pairs of it; a token's sines and cosines are made once per block, the angle
+// (position times a 64-bit rate) in 64 bits, the rest in 32; the result is
+// rounded once.
 //
 // latent_rope_store_kernel.  Columns [col, col + rank) of a token's row are a
 // latent: normed with a weight over `rank`; the `rot` columns behind it are one
-// rotated key part shared by all heads: turned as above, not normed.  Both go
+// rotated key part shared by all heads: turned as above (cosine and sine times
+// a factor), not normed.  Both go
 // to the one pool of the layer, [pages, 1, page, padded] with the latent at
 // columns [0, rank), the rotated part at [rank, rank + rot) and zeros behind.
 // Optionally a second latent at columns [col2, col2 + rank2) (the queries'
-// own) is normed with its weight into `out2`.
-#include "common.cuh"
+// own) is normed with its weight into `out2`, and the rotated parts of the
+// row's queries are turned into the rows of another buffer, behind the columns
+// that the queries' plain parts will take in the latent space.
+#include "latent_token.cuh"
 
 namespace {
 
@@ -39,6 +43,7 @@ struct HeadExtras {
   float temp_coef;             // temp_every 0: no query temperature
   int temp_every;
   int store_values;            // the rows' value heads go to the value pool
+  float magnitude;             // on cosines and sines
 };
 __device__ __forceinline__ float query_temperature(int pos, const HeadExtras &x) {
   return x.temp_every > 0 ? fmaf(x.temp_coef, logf(static_cast<float>((pos + 1) / x.temp_every + 1)), 1.0f) : 1.0f;
@@ -77,7 +82,7 @@ __device__ __forceinline__ void store_pair(T *p, bool together, float u, float v
 template <typename T>
 __global__ void __launch_bounds__(128)
 rope_norm_store_kernel(T *__restrict__ rows, int64_t row_stride, T *__restrict__ k_cache, T *__restrict__ v_cache,
-                       const float *__restrict__ rates, const int32_t *__restrict__ positions,
+                       const double *__restrict__ rates, const int32_t *__restrict__ positions,
                        const int32_t *__restrict__ request_of_token, const int32_t *__restrict__ block_table,
                        int max_blocks, int heads, int kv_heads, int head_dim, int rot_col, int rot, int unit, float eps,
                        int norm_dim, int page_size, int num_pages, int write_kv, int values_are_keys, int heads_per_block,
@@ -87,8 +92,10 @@ rope_norm_store_kernel(T *__restrict__ rows, int64_t row_stride, T *__restrict__
   le::wait_for_predecessor();
   const int t = blockIdx.x;
   const int pos = positions[t];
-  const float fpos = static_cast<float>(pos);
-  for (int i = threadIdx.x; i < (rot >> 1); i += blockDim.x) sincosf(fpos * rates[i], &turn[2 * i], &turn[2 * i + 1]);
+  for (int i = threadIdx.x; i < (rot >> 1); i += blockDim.x) {
+    const float2 cs = le::turn_of(pos, rates[i], extras.magnitude);
+    turn[2 * i] = cs.y, turn[2 * i + 1] = cs.x;
+  }
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
   T *row = rows + static_cast<int64_t>(t) * row_stride;
   int page = 0;
@@ -188,7 +195,7 @@ struct Piece<float> {
 template <typename T>
 __global__ void __launch_bounds__(128)
 rope_norm_store_pieces_kernel(T *__restrict__ rows, int64_t row_stride, T *__restrict__ k_cache, T *__restrict__ v_cache,
-                              const float *__restrict__ rates, const int32_t *__restrict__ positions,
+                              const double *__restrict__ rates, const int32_t *__restrict__ positions,
                               const int32_t *__restrict__ request_of_token, const int32_t *__restrict__ block_table,
                               int max_blocks, int heads, int kv_heads, int head_dim, int rot_col, int rot, int unit, float eps,
                               int norm_dim, int page_size, int num_pages, int write_kv, int values_are_keys,
@@ -200,8 +207,10 @@ rope_norm_store_pieces_kernel(T *__restrict__ rows, int64_t row_stride, T *__res
   le::wait_for_predecessor();
   const int t = blockIdx.x;
   const int pos = positions[t];
-  const float fpos = static_cast<float>(pos);
-  for (int i = threadIdx.x; i < (rot >> 1); i += blockDim.x) sincosf(fpos * rates[i], &turn[2 * i], &turn[2 * i + 1]);
+  for (int i = threadIdx.x; i < (rot >> 1); i += blockDim.x) {
+    const float2 cs = le::turn_of(pos, rates[i], extras.magnitude);
+    turn[2 * i] = cs.y, turn[2 * i + 1] = cs.x;
+  }
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
   T *row = rows + static_cast<int64_t>(t) * row_stride;
   int page = 0;
@@ -276,84 +285,44 @@ rope_norm_store_pieces_kernel(T *__restrict__ rows, int64_t row_stride, T *__res
 
 template <typename T>
 __global__ void __launch_bounds__(128)
-latent_rope_store_kernel(const T *__restrict__ src, int64_t src_stride, int col, int rank, int rot, int padded,
-                         const float *__restrict__ weight, float eps, const float *__restrict__ rates, T *__restrict__ cache,
-                         int col2, int rank2, const float *__restrict__ weight2, T *__restrict__ out2, int64_t out2_stride,
-                         const int32_t *__restrict__ positions, const int32_t *__restrict__ request_of_token,
-                         const int32_t *__restrict__ block_table, int max_blocks, int page_size, int num_pages,
-                         int *__restrict__ status) {
+latent_rope_store_kernel(const le_latent::Args<T> a, int col2, int rank2, const float *__restrict__ weight2,
+                         T *__restrict__ out2, int64_t out2_stride) {
   __shared__ float scratch[33];
+  __shared__ float2 turn[le_latent::MAX_PAIRS];
   le::let_successor_start();
-  le::wait_for_predecessor();
   const int t = blockIdx.x;
-  const T *row = src + static_cast<int64_t>(t) * src_stride;
-  // Everything is asked for before anything is waited for: the page, both latents' sums of squares.
-  int pos = 0, page = -1;
-  if (cache != nullptr) {
-    pos = positions[t];
-    const int b = request_of_token[t];
-    page = pos >= 0 ? block_table[static_cast<int64_t>(b) * max_blocks + pos / page_size] : -1;
-  }
-  const T *x = row + col;
-  float ss2 = 0.0f, ss = 0.0f;
+  le_latent::make_turns(turn, a, t);
+  le::wait_for_predecessor();
+  __syncthreads();
   if (out2 != nullptr) {
+    const T *x = a.src + static_cast<int64_t>(t) * a.src_stride + col2;
+    float ss = 0.0f;
     for (int i = threadIdx.x; i < rank2; i += blockDim.x) {
-      const float v = le::to_f32(row[col2 + i]);
-      ss2 = fmaf(v, v, ss2);
-    }
-  }
-  if (cache != nullptr) {
-    for (int i = threadIdx.x; i < rank; i += blockDim.x) {
       const float v = le::to_f32(x[i]);
       ss = fmaf(v, v, ss);
     }
-  }
-  if (out2 != nullptr) {
-    ss2 = le::block_sum(ss2, scratch);
-    const float inv = rsqrtf(ss2 / static_cast<float>(rank2) + eps);
+    const float inv = rsqrtf(le::block_sum(ss, scratch) / static_cast<float>(rank2) + a.eps);
     T *dst = out2 + static_cast<int64_t>(t) * out2_stride;
-    for (int i = threadIdx.x; i < rank2; i += blockDim.x) dst[i] = le::from_f32<T>(le::to_f32(row[col2 + i]) * inv * weight2[i]);
+    for (int i = threadIdx.x; i < rank2; i += blockDim.x) dst[i] = le::from_f32<T>(le::to_f32(x[i]) * inv * weight2[i]);
   }
-  if (cache == nullptr) return;
-  const bool bad = page < 0 || page >= num_pages;
-  if (bad && threadIdx.x == 0) atomicOr(status, LE_STATUS_BAD_PAGE);
-  ss = le::block_sum(ss, scratch);
-  if (bad) return;
-  const float inv = rsqrtf(ss / static_cast<float>(rank) + eps);
-  const float fpos = static_cast<float>(pos);
-  T *dst = cache + (static_cast<int64_t>(page) * page_size + pos % page_size) * padded;
-  for (int i = threadIdx.x; i < padded; i += blockDim.x) {
-    float v = 0.0f;
-    if (i < rank) {
-      v = le::to_f32(x[i]) * inv * weight[i];
-    } else if (i < rank + rot) {
-      const int j = i - rank;
-      v = le::to_f32(x[i]);
-      if ((j | 1) < rot) {
-        const float other = le::to_f32(x[rank + (j ^ 1)]);
-        float s, c;
-        sincosf(fpos * rates[j >> 1], &s, &c);
-        v = (j & 1) ? v * c + other * s : v * c - other * s;
-      }
-    }
-    dst[i] = le::from_f32<T>(v);
-  }
+  if (a.q_out != nullptr) le_latent::turn_queries(a, t, turn);
+  if (a.cache != nullptr) le_latent::store_latent(a, t, turn, scratch);
 }
 
 }  // namespace
 
 // rows: [tokens] rows of row_stride elements, queries then keys, heads of head_dim entries (even, at most 512).
 // k_cache / v_cache: [pages, kv_heads, page, head_dim].  write_kv 0: queries only (the keys' columns are not read).
-// w_q / w_k: float32 [head_dim] or null; temp_every 0: no query temperature; store_values: value heads lie behind the keys.
-LE_API int le_rope_norm_store(void *rows, int64_t row_stride, int dtype, void *k_cache, void *v_cache, const float *rates,
+// rates: float64.  w_q / w_k: float32 [head_dim] or null; temp_every 0: no query temperature; store_values: value heads lie behind the keys.
+LE_API int le_rope_norm_store(void *rows, int64_t row_stride, int dtype, void *k_cache, void *v_cache, const double *rates,
                               const int32_t *positions, const int32_t *request_of_token, const int32_t *block_table,
                               int max_blocks, int num_tokens, int heads, int kv_heads, int head_dim, int rot_col, int rot,
                               int unit, float eps, int norm_dim, int page_size, int num_pages, int write_kv,
                               int values_are_keys, const float *w_q, const float *w_k, float temp_coef, int temp_every,
-                              int store_values, int *status, cudaStream_t stream) {
+                              int store_values, float magnitude, int *status, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
   if (temp_every < 0 || (values_are_keys && store_values)) return le::invalid("le_rope_norm_store: bad options");
-  const HeadExtras extras{w_q, w_k, temp_coef, temp_every, store_values};
+  const HeadExtras extras{w_q, w_k, temp_coef, temp_every, store_values, magnitude};
   if (head_dim < 2 || head_dim % 2 || head_dim > 64 * RN_MAX_PAIRS)
     return le::invalid("le_rope_norm_store: heads of %d entries (even, at most %d)", head_dim, 64 * RN_MAX_PAIRS);
   if (rot < 0 || rot % 2 || rot_col < 0 || rot_col % 2 || rot_col + rot > head_dim)
@@ -386,19 +355,23 @@ LE_API int le_rope_norm_store(void *rows, int64_t row_stride, int dtype, void *k
                                               page_size, num_pages, write_kv, values_are_keys, per_block, together, extras, status));
 }
 
-// cache: [pages, 1, page, padded] or null (nothing is stored); out2 null: no second latent.
+// cache: [pages, 1, page, padded] or null (nothing is stored); out2 null: no second latent; q_out null: no queries are
+// turned (else rows of q_stride elements, heads * padded wide: see latent_token.cuh); rates: float64.
 LE_API int le_latent_rope_store(const void *src, int64_t src_stride, int dtype, int col, int rank, int rot, int padded,
-                                const float *weight, float eps, const float *rates, void *cache, int col2, int rank2,
-                                const float *weight2, void *out2, int64_t out2_stride, const int32_t *positions,
+                                const float *weight, float eps, const double *rates, float magnitude, void *cache, int col2,
+                                int rank2, const float *weight2, void *out2, int64_t out2_stride, int q_col, int q_head,
+                                int heads, void *q_out, int64_t q_stride, const int32_t *positions,
                                 const int32_t *request_of_token, const int32_t *block_table, int max_blocks, int num_tokens,
                                 int page_size, int num_pages, int *status, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
-  if (rank < 1 || rot < 0 || rot % 2 || padded < rank + rot)
+  if (rank < 1 || rot < 0 || rot % 2 || rot > 2 * le_latent::MAX_PAIRS || padded < rank + rot)
     return le::invalid("le_latent_rope_store: rank %d, %d turned entries, padded %d", rank, rot, padded);
-  LE_DISPATCH_DTYPE(dtype, T,
-                    return le::launch_chained(latent_rope_store_kernel<T>, dim3(num_tokens), dim3(128), 0, stream,
-                                              static_cast<const T *>(src), src_stride, col, rank, rot, padded, weight, eps,
-                                              rates, static_cast<T *>(cache), col2, rank2, weight2, static_cast<T *>(out2),
-                                              out2_stride, positions, request_of_token, block_table, max_blocks, page_size,
-                                              num_pages, status));
+  LE_DISPATCH_DTYPE(dtype, T, {
+    le_latent::Args<T> a{static_cast<const T *>(src), src_stride, col, rank, rot, padded, weight, eps, rates, magnitude,
+                         static_cast<T *>(cache), positions, request_of_token, block_table, max_blocks, page_size, num_pages,
+                         status, q_col, q_head, heads, static_cast<T *>(q_out), q_stride, 0};
+    a.q_pairs = le_latent::pairs_together(a);
+    return le::launch_chained(latent_rope_store_kernel<T>, dim3(num_tokens), dim3(128), 0, stream, a, col2, rank2, weight2,
+                              static_cast<T *>(out2), out2_stride);
+  });
 }

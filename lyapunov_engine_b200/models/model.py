@@ -82,6 +82,8 @@ class Model:
                     group = self.groups.index(plan)
                     stream = self.streams_per_group[group]
                     self.streams_per_group[group] += 1
+                if mixer.reads_only and writes:
+                    raise ValueError(f"run order entry {index} has no keys of its own and names no entry whose cache it reads")
             elif run.reads_cache_of is not None:
                 raise ValueError(f"run order entry {index} reads a cache but its mixer keeps no pages")
             state_index = None

@@ -92,10 +92,16 @@ _CORE_SIGNATURES = {
                           c_int, c_int, c_int, c_float, c_void_p],
     "le_rope_norm_store": [c_void_p, c_int64, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                            c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_int, c_int,
-                           c_void_p, c_void_p, c_float, c_int, c_int, c_void_p, c_void_p],
-    "le_latent_rope_store": [c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_void_p,
-                             c_int, c_int, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                             c_int, c_void_p, c_void_p],
+                           c_void_p, c_void_p, c_float, c_int, c_int, c_float, c_void_p, c_void_p],
+    "le_latent_rope_store": [c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_float,
+                             c_void_p, c_int, c_int, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_int64,
+                             c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
+    "le_conv_turn_store": [c_void_p, c_int64, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
+                           c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_float, c_int, c_float, c_int, c_void_p, c_int64,
+                           c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
+                           c_void_p],
+    "le_addend_norm": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int64, c_void_p, c_void_p, c_void_p, c_float, c_int,
+                       c_void_p, c_void_p, c_float, c_int, c_void_p, c_int, c_int, c_void_p],
     "le_rmsnorm_pair": [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int64, c_void_p, c_int, c_int, c_int64,
                         c_void_p, c_float, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_void_p],
     "le_residual_add": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int64, c_void_p, c_int, c_int, c_int64,
@@ -123,10 +129,11 @@ _CORE_SIGNATURES = {
                     c_int, c_int, c_int, c_int, c_void_p, c_void_p],
     "le_latent_norm_store": [c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p,
                              c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
-    "le_latent_prepare": [c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_void_p,
-                          c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p],
+    "le_latent_prepare": [c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int,
+                          c_void_p, c_float, c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                          c_int, c_void_p, c_void_p],
     "le_gemm_heads": [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int,
-                      c_void_p],
+                      c_int, c_int64, c_int64, c_void_p],
     "le_gemm_tc_bf16": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int64, c_int64, c_int64, c_int,
                         c_int, c_float, c_float, c_void_p, c_void_p],
     "le_gemm_skinny_bf16": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int64, c_int64, c_int64, c_int,
@@ -434,48 +441,66 @@ def latent_norm_store(src, col, rank, weight, eps, cache, positions, request_of_
 LATENT_PREPARE_ROWS = 32
 
 
-def latent_prepare_applies(src: torch.Tensor, head_dim: int) -> bool:
+def latent_prepare_applies(src: torch.Tensor, head_dim: int, rot: int = 0) -> bool:
     """Whether latent_prepare() takes these rows (few of them, 16-byte pieces)."""
     vec = 16 // src.element_size()
-    return (src.shape[0] <= LATENT_PREPARE_ROWS and head_dim % vec == 0 and src.stride(0) % vec == 0
+    return (src.shape[0] <= LATENT_PREPARE_ROWS and head_dim % vec == 0 and rot % vec == 0 and src.stride(0) % vec == 0
             and src.data_ptr() % 16 == 0 and src.stride(1) == 1)
 
 
 def latent_prepare(q_latent, src, w_into, col, rank, weight, eps, cache, positions, request_of_token, block_table,
-                   page_size, status) -> None:
+                   page_size, status, rot: int = 0, rates=None, magnitude: float = 1.0) -> None:
     """For a step of few rows, in one launch: gemm_heads(q_latent, src[:, :heads
     * head_dim], w_into) and latent_norm_store(src, col, rank, ...) (``cache``
-    None: the latent is not stored)."""
-    _need_cuda(q_latent, src, w_into, weight, cache, positions, block_table)
-    heads, padded, head_dim = w_into.shape
+    None: the latent is not stored).  With ``rot`` > 0 a head's query has
+    ``rot`` turned entries behind its head_dim plain ones, ``w_into`` is [heads,
+    rank, head_dim], and latent_rope_store() with its queries takes the place
+    of latent_norm_store()."""
+    _need_cuda(q_latent, src, w_into, weight, cache, positions, block_table, rates)
+    heads, out_rows, head_dim = w_into.shape
     T = src.shape[0]
-    assert latent_prepare_applies(src, head_dim) and w_into.is_contiguous() and w_into.dtype == src.dtype == q_latent.dtype
-    assert q_latent.shape == (T, heads * padded) and q_latent.stride(1) == 1 and padded >= rank
+    padded = q_latent.shape[1] // heads
+    assert latent_prepare_applies(src, head_dim, rot) and w_into.is_contiguous() and w_into.dtype == src.dtype == q_latent.dtype
+    assert q_latent.shape == (T, heads * padded) and q_latent.stride(1) == 1 and padded >= rank + rot
+    assert out_rows == (rank if rot else padded)
     assert weight.dtype == torch.float32 and weight.numel() == rank and block_table.is_contiguous()
+    _check_rates(rates, rot)
     pages = 0
     if cache is not None:
         assert cache.dtype == src.dtype and cache.is_contiguous() and tuple(cache.shape[1:]) == (1, page_size, padded)
         pages = cache.shape[0]
     _check(core().le_latent_prepare(_ptr(src), src.stride(0), T, heads, head_dim, _ptr(w_into), _ptr(q_latent),
-                                    q_latent.stride(0), col, rank, padded, _ptr(weight), float(eps), _ptr(cache),
-                                    dtype_code(src.dtype), _ptr(positions), _ptr(request_of_token), _ptr(block_table),
-                                    block_table.shape[1], page_size, pages, _ptr(status), _stream()), "le_latent_prepare")
+                                    q_latent.stride(0), col, rank, int(rot), padded, _ptr(weight), float(eps), _ptr(rates),
+                                    float(magnitude), _ptr(cache), dtype_code(src.dtype), _ptr(positions),
+                                    _ptr(request_of_token), _ptr(block_table), block_table.shape[1], page_size, pages,
+                                    _ptr(status), _stream()), "le_latent_prepare")
 
 
-def gemm_heads(out, a, w, gate=None) -> None:
+def _check_rates(rates, rot: int) -> None:
+    assert rot == 0 or (rates is not None and rates.dtype == torch.float64 and rates.is_contiguous() and rates.numel() >= rot // 2)
+
+
+def gemm_heads(out, a, w, gate=None, a_head: int | None = None, out_head: int | None = None) -> None:
     """One product per head: out[t, h, :] = w[h] @ a[t, h, :] (w: [heads, N,
-    K]), times sigmoid(gate[t, h]) where ``gate`` is given.  ``a``, ``out`` and
-    ``gate`` may be column ranges of wider buffers (rows of any stride)."""
+    K]), times sigmoid(gate[t, h]), or, for a gate of heads * N columns,
+    sigmoid(gate[t, h, :]), where ``gate`` is given.  ``a``, ``out`` and
+    ``gate`` may be column ranges of wider buffers (rows of any stride);
+    ``a_head`` / ``out_head``: columns from one head of a / out to the next (K /
+    N by default)."""
     _need_cuda(out, a, w, gate)
     heads, N, K = w.shape
     M = a.shape[0]
-    assert a.shape[1] == heads * K and out.shape == (M, heads * N) and a.stride(1) == 1 and out.stride(1) == 1
+    a_head, out_head = int(a_head or K), int(out_head or N)
+    assert a_head >= K and out_head >= N and a.stride(1) == 1 and out.stride(1) == 1 and out.shape[0] == M
+    assert a.shape[1] >= (heads - 1) * a_head + K and out.shape[1] >= (heads - 1) * out_head + N
     assert w.is_contiguous() and a.dtype == w.dtype == out.dtype
+    entries = False
     if gate is not None:
-        assert gate.shape == (M, heads) and gate.stride(1) == 1 and gate.dtype == a.dtype
+        entries = gate.shape[1] != heads or N == 1
+        assert gate.shape == (M, heads * N if entries else heads) and gate.stride(1) == 1 and gate.dtype == a.dtype
     _check(core().le_gemm_heads(_ptr(out), out.stride(0), _ptr(a), a.stride(0), _ptr(w), _ptr(gate),
-                                gate.stride(0) if gate is not None else 0, dtype_code(a.dtype), M, heads, N, K, _stream()),
-           "le_gemm_heads")
+                                gate.stride(0) if gate is not None else 0, 1 if entries else 0, dtype_code(a.dtype), M, heads, N,
+                                K, a_head, out_head, _stream()), "le_gemm_heads")
 
 
 def convert(out: torch.Tensor, src: torch.Tensor) -> None:
@@ -1376,11 +1401,11 @@ def head_norm_gate(out, o, gate, weight, eps, heads, vdim, sigmoid: bool = False
 # -------------------------------------------------------------------------- rotary pairs with a norm per head
 def rope_norm_store(rows, k_cache, v_cache, rates, positions, request_of_token, block_table, heads, kv_heads, head_dim,
                     rot_col, rot, unit_eps, norm_dim, page_size, write_kv, values_are_keys, status, w_q=None, w_k=None,
-                    temperature=None, store_values: bool = False) -> None:
+                    temperature=None, store_values: bool = False, magnitude: float = 1.0) -> None:
     """Rows hold query heads, then key heads, ``head_dim`` entries each.  The
     entries (rot_col + 2i, rot_col + 2i + 1) below rot_col + ``rot`` of every
-    head turn by position * rates[i]; with ``unit_eps`` not None the head is
-    then divided by sqrt(mean over its first ``norm_dim`` entries of x^2 +
+    head turn by position * rates[i] (``rates`` float64: the angle is taken in
+    64 bits; cosine and sine times ``magnitude``); with ``unit_eps`` not None the head is then divided by sqrt(mean over its first ``norm_dim`` entries of x^2 +
     unit_eps).  Queries are rewritten in place, keys go to ``k_cache``, and
     ``v_cache`` receives the keys as they were projected when
     ``values_are_keys``.  ``write_kv`` False: the queries only.  ``w_q`` /
@@ -1392,7 +1417,7 @@ def rope_norm_store(rows, k_cache, v_cache, rates, positions, request_of_token, 
     T = rows.shape[0]
     assert rows.stride(1) == 1
     assert rows.shape[1] >= (heads + (kv_heads * (2 if store_values else 1) if write_kv else 0)) * head_dim
-    assert rot == 0 or (rates.dtype == torch.float32 and rates.is_contiguous() and rates.numel() >= rot // 2)
+    _check_rates(rates, rot)
     for w in (w_q, w_k):
         assert w is None or (w.dtype == torch.float32 and w.is_contiguous() and w.numel() == head_dim)
     coef, every = temperature if temperature is not None else (0.0, 0)
@@ -1409,20 +1434,24 @@ def rope_norm_store(rows, k_cache, v_cache, rates, positions, request_of_token, 
                                      head_dim, rot_col, rot, 0 if unit_eps is None else 1,
                                      0.0 if unit_eps is None else float(unit_eps), norm_dim, page_size, pages,
                                      1 if write_kv else 0, 1 if values_are_keys else 0, _ptr(w_q), _ptr(w_k), float(coef),
-                                     int(every), 1 if store_values else 0, _ptr(status), _stream()), "le_rope_norm_store")
+                                     int(every), 1 if store_values else 0, float(magnitude), _ptr(status), _stream()), "le_rope_norm_store")
 
 
 def latent_rope_store(src, col, rank, rot, padded, weight, eps, rates, cache, positions, request_of_token, block_table,
-                      page_size, status, second=None) -> None:
+                      page_size, status, second=None, magnitude: float = 1.0, queries=None) -> None:
     """The latent at columns [col, col + rank) of ``src`` is normed (weight
     [rank]) and the ``rot`` columns behind it are turned in neighbouring pairs
-    by position * rates[i]; both go to ``cache`` [pages, 1, page, padded]
-    (None: nothing is stored).  ``second`` = (col2, rank2, weight2, out2): a
-    second latent of the row is normed into ``out2``."""
+    by position * rates[i] (``rates`` float64; cosine and sine times
+    ``magnitude``); both go to ``cache`` [pages, 1, page, padded] (None: nothing
+    is stored).  ``second`` = (col2, rank2, weight2, out2): a second latent of
+    the row is normed into ``out2``.  ``queries`` = (q_col, q_head, heads,
+    q_out): the rot columns from q_col + h * q_head of every head h are turned
+    the same way into columns h * padded + rank .. of ``q_out``, with zeros
+    behind them up to (h + 1) * padded."""
     _need_cuda(src, weight, rates, cache, positions, block_table)
     T = src.shape[0]
     assert src.stride(1) == 1 and weight.dtype == torch.float32 and weight.numel() == rank
-    assert rot == 0 or (rates is not None and rates.dtype == torch.float32 and rates.numel() >= rot // 2)
+    _check_rates(rates, rot)
     pages = 0
     if cache is not None:
         assert cache.dtype == src.dtype and cache.is_contiguous() and tuple(cache.shape[1:]) == (1, page_size, padded)
@@ -1430,11 +1459,61 @@ def latent_rope_store(src, col, rank, rot, padded, weight, eps, rates, cache, po
     col2, rank2, weight2, out2 = second if second is not None else (0, 0, None, None)
     if out2 is not None:
         assert out2.dtype == src.dtype and out2.stride(1) == 1 and weight2.dtype == torch.float32 and weight2.numel() == rank2
+    q_col, q_head, heads, q_out = queries if queries is not None else (0, 0, 0, None)
+    if q_out is not None:
+        assert q_out.dtype == src.dtype and q_out.stride(1) == 1 and q_out.shape == (T, heads * padded)
+        assert src.shape[1] >= q_col + (heads - 1) * q_head + rot
     _check(core().le_latent_rope_store(_ptr(src), src.stride(0), dtype_code(src.dtype), col, rank, rot, padded, _ptr(weight),
-                                       float(eps), _ptr(rates), _ptr(cache), col2, rank2, _ptr(weight2), _ptr(out2),
-                                       out2.stride(0) if out2 is not None else 0, _ptr(positions), _ptr(request_of_token),
+                                       float(eps), _ptr(rates), float(magnitude), _ptr(cache), col2, rank2, _ptr(weight2),
+                                       _ptr(out2), out2.stride(0) if out2 is not None else 0, q_col, q_head, heads, _ptr(q_out),
+                                       q_out.stride(0) if q_out is not None else 0, _ptr(positions), _ptr(request_of_token),
                                        _ptr(block_table), block_table.shape[1], T, page_size, pages, _ptr(status), _stream()),
            "le_latent_rope_store")
+
+
+CONV_TURN_MAX_DIM = 512
+
+
+def conv_turn_store(q_out, src, bias, w_taps, state, state_slots, cu_q, tile_request, tile_q0, num_tiles, rates, rot, magnitude,
+                    unit_eps, norm_dim, k_cache, v_cache, positions, block_table, heads, kv_heads, head_dim, page_size,
+                    write_kv, status) -> None:
+    """Rows of ``src`` hold q [heads, head_dim] | k | v [kv_heads, head_dim]
+    (``kv_heads`` 0: queries only).  ``bias`` (float32 [channels] or None) is
+    added; every channel passes through a causal convolution over time,
+    ``w_taps`` float32 [taps, channels], that continues each request from its
+    row of ``state`` (float32 [rows, taps - 1, channels], the projected values
+    before the step; None when taps is 1) and brings the row up to date; the
+    entries (2i, 2i + 1) below ``rot`` of every head of q and k turn by
+    position * rates[i] (float64), cosine and sine times ``magnitude``; with
+    ``unit_eps`` not None the head is divided by sqrt(sum of squares /
+    ``norm_dim`` + unit_eps).  Queries go to ``q_out``, keys and values to the
+    pages.  Tiles as short_conv() takes them."""
+    _need_cuda(q_out, src, bias, w_taps, state, rates, k_cache, v_cache, positions, block_table)
+    T = src.shape[0]
+    channels = (heads + 2 * kv_heads) * head_dim
+    taps = w_taps.shape[0]
+    assert src.stride(1) == 1 and src.shape[1] >= channels and q_out.dtype == src.dtype and q_out.stride(1) == 1
+    assert q_out.shape == (T, heads * head_dim) and w_taps.dtype == torch.float32 and w_taps.is_contiguous()
+    assert w_taps.shape[1] == channels and block_table.dtype == torch.int32 and block_table.is_contiguous()
+    assert bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == channels)
+    _check_rates(rates, rot)
+    rows = pages = 0
+    if taps > 1:
+        assert state is not None and state.dtype == torch.float32 and state.is_contiguous()
+        assert tuple(state.shape[1:]) == (taps - 1, channels)
+        rows = state.shape[0]
+    if write_kv:
+        assert kv_heads > 0 and k_cache.dtype == src.dtype and k_cache.is_contiguous() and v_cache.is_contiguous()
+        assert tuple(k_cache.shape[1:]) == (kv_heads, page_size, head_dim) and v_cache.shape == k_cache.shape
+        pages = k_cache.shape[0]
+    _check(core().le_conv_turn_store(_ptr(src), src.stride(0), dtype_code(src.dtype), _ptr(bias), _ptr(w_taps), taps,
+                                     _ptr(state) if taps > 1 else None, rows, _ptr(state_slots), _ptr(cu_q),
+                                     _ptr(tile_request), _ptr(tile_q0), num_tiles, SHORT_CONV_TILE, T, _ptr(rates), int(rot),
+                                     float(magnitude), 0 if unit_eps is None else 1,
+                                     0.0 if unit_eps is None else float(unit_eps), int(norm_dim), _ptr(q_out), q_out.stride(0),
+                                     _ptr(k_cache) if write_kv else None, _ptr(v_cache) if write_kv else None,
+                                     _ptr(positions), _ptr(block_table), block_table.shape[1], heads, kv_heads, head_dim,
+                                     page_size, pages, 1 if write_kv else 0, _ptr(status), _stream()), "le_conv_turn_store")
 
 
 # -------------------------------------------------------------------------- sub-layers side by side; inputs per token
@@ -1473,6 +1552,29 @@ def rmsnorm_pair(out1, out2, resid, w1, w2, eps, addend=None, addend_weight=None
     _check(core().le_rmsnorm_pair(_ptr(out1), _ptr(out2), out_code, _ptr(resid), ptr, code, parts, stride,
                                   ptr2, code2, parts2, stride2, _ptr(addend_weight), float(addend_eps), _ptr(w1), _ptr(w2), float(eps), _ptr(rows), n, W,
                                   _stream()), "le_rmsnorm_pair")
+
+
+def addend_norm(out, resid, weight, bias, eps, centered: bool, addend=None, addend_bias=None, addend_weight=None,
+                addend_norm_bias=None, addend_eps: float = 0.0, addend_centered: bool = False, rows=None) -> None:
+    """``addend`` (as _addend() takes it) enters the 32-bit stream ``resid``
+    [T, W] through a norm: with y = addend + ``addend_bias``, resid += (y -
+    mean) / sqrt(var + addend_eps) * ``addend_weight`` + ``addend_norm_bias``;
+    then out = (resid - mean) / sqrt(var + eps) * ``weight`` + ``bias``.  A norm
+    that is not ``centered`` takes mean 0 (a root mean square norm); biases may
+    be None; all vectors float32 [W].  With ``rows`` only those rows are
+    normed, into out[0 .. len(out)), and ``resid`` is left as it is."""
+    _need_cuda(out, resid, weight, bias, addend, addend_bias, addend_weight, addend_norm_bias, rows)
+    T, W = resid.shape
+    n = out.shape[0]
+    assert resid.dtype == torch.float32 and resid.is_contiguous() and out.is_contiguous() and out.shape[1] == W
+    for v in (weight, bias, addend_bias, addend_weight, addend_norm_bias):
+        assert v is None or (v.dtype == torch.float32 and v.is_contiguous() and v.numel() == W)
+    assert n == T if rows is None else (rows.dtype == torch.int32 and rows.numel() >= n)
+    ptr, code, parts, stride = _addend(addend, T, W)
+    _check(core().le_addend_norm(_ptr(out), dtype_code(out.dtype), _ptr(resid), ptr, code, parts, stride, _ptr(addend_bias),
+                                 _ptr(addend_weight), _ptr(addend_norm_bias), float(addend_eps), 1 if addend_centered else 0,
+                                 _ptr(weight), _ptr(bias), float(eps), 1 if centered else 0, _ptr(rows), n, W, _stream()),
+           "le_addend_norm")
 
 
 def residual_add(resid, a=None, f=None, bias=None, copy=None) -> None:

@@ -31,6 +31,11 @@ What a description may choose beyond the reference's Llama layer:
 * ``softcap`` c: a score s (after the scale) becomes c * tanh(s / c);
 * ``sink_name``: a tensor [nh]; the softmax's denominator has one more term
   exp(sink_h) (it has no key and no value, and neither scale nor cap);
+* ``o_bias_name``: a bias [H] on the output projection, left to the block that
+  adds the output to the stream (``output_bias``);
+* ``k_name`` and ``v_name`` None: the layer has queries only and reads the keys
+  and values that another run of the model wrote (the run order names it); its
+  mask, scale and queries are its own;
 * ``v_name`` None: there is no value projection, the values are the keys as
   projected (before any position encoding or norm of the keys); the position
   encoding then fills the value pool itself (it is built with
@@ -83,15 +88,19 @@ def signed_scale(scale: float, head_scale: torch.Tensor | None, num_heads: int, 
 @register_mixer("attention")
 class AttentionMixer(Mixer):
     def __init__(self, hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int, position: PartSpec | None,
-                 q_name: str, k_name: str, v_name: str | None, o_name: str, window: int | None = None,
+                 q_name: str, k_name: str | None, v_name: str | None, o_name: str, window: int | None = None,
                  chunk: int | None = None, scale: float | None = None, value_dim: int | None = None,
                  head_scale_name: str | None = None, gate_name: str | None = None, gate_per_entry: bool = False,
-                 keep_first: int = 0, softcap: float | None = None, sink_name: str | None = None):
+                 keep_first: int = 0, softcap: float | None = None, sink_name: str | None = None,
+                 o_bias_name: str | None = None):
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} heads do not divide into {num_kv_heads} groups")
         self.qk_dim = int(head_dim)
         self.value_dim = int(value_dim) if value_dim else self.qk_dim
-        self.values_are_keys = v_name is None
+        self.reads_only = k_name is None        # (keys and values are another run's)
+        if self.reads_only and v_name is not None:
+            raise ValueError("a layer without keys of its own has no values of its own")
+        self.values_are_keys = v_name is None and not self.reads_only
         if self.values_are_keys and (position is None or self.value_dim != self.qk_dim):
             raise ValueError("values that are the keys need a position encoding that stores them, and the keys' size")
         # the one head size of kernels and pages
@@ -123,6 +132,13 @@ class AttentionMixer(Mixer):
         self.scale = float(scale) if scale is not None else 1.0 / (self.qk_dim ** 0.5)
         self.names = (q_name, k_name, v_name, o_name)
         self.head_scale_name, self.gate_name, self.sink_name = head_scale_name, gate_name, sink_name
+        # a position encoding that does not leave the queries in place says where they are (encode_rows)
+        self.encodes_rows = hasattr(self.position, "encode_rows")
+        if self.reads_only and not self.encodes_rows:
+            raise ValueError("a layer that reads another one's keys needs a position encoding for queries alone")
+        if self.encodes_rows and self.reads_only != getattr(self.position, "queries_only", False):
+            raise ValueError("the position encoding and the mixer must agree on whether there are keys")
+        self.o_bias_name, self.output_bias = o_bias_name, None
         self.gate_per_entry = bool(gate_per_entry) and bool(gate_name)
         # rows of the projection stay 16-byte multiples
         self.gate_rows = 0
@@ -135,8 +151,12 @@ class AttentionMixer(Mixer):
     def cache_need(self):
         return KVNeed(self.num_kv_heads, self.head_dim, self.window, self.chunk, keep_first=self.keep_first)
 
+    def extra_state_needs(self):
+        return dict(self.position.extra_state_needs()) if hasattr(self.position, "extra_state_needs") else {}
+
     def tile_sizes(self):
-        return attention_kernels.tile_sizes()
+        own = self.position.tile_sizes() if hasattr(self.position, "tile_sizes") else []
+        return attention_kernels.tile_sizes() + own
 
     def decode_variant(self, fill, num_decode, context_bound):
         if self.runtime is None or self.runtime.dtype != torch.bfloat16:
@@ -147,10 +167,14 @@ class AttentionMixer(Mixer):
     def tensors(self):
         q, k, v, o = self.names
         H, nh, nkv = self.hidden_size, self.num_heads, self.num_kv_heads
-        decls = [TensorDecl(q, (nh * self.qk_dim, H)), TensorDecl(k, (nkv * self.qk_dim, H)),
-                 TensorDecl(o, (H, nh * self.value_dim))]
-        if not self.values_are_keys:
-            decls.insert(2, TensorDecl(v, (nkv * self.value_dim, H)))
+        decls = [TensorDecl(q, (nh * self.qk_dim, H))]
+        if not self.reads_only:
+            decls.append(TensorDecl(k, (nkv * self.qk_dim, H)))
+            if not self.values_are_keys:
+                decls.append(TensorDecl(v, (nkv * self.value_dim, H)))
+        decls.append(TensorDecl(o, (H, nh * self.value_dim)))
+        if self.o_bias_name:
+            decls.append(TensorDecl(self.o_bias_name, (H,), role="vector", init="taps"))
         if self.head_scale_name:
             decls.append(TensorDecl(self.head_scale_name, (nh,), role="vector", init="ones_jitter"))
         if self.sink_name:
@@ -162,8 +186,10 @@ class AttentionMixer(Mixer):
     def bind(self, get, runtime):
         q, k, v, o = self.names
         nh, nkv, hd = self.num_heads, self.num_kv_heads, self.head_dim
-        rows = [pad_head_rows(get(q), nh, self.qk_dim, hd), pad_head_rows(get(k), nkv, self.qk_dim, hd)]
-        if not self.values_are_keys:
+        rows = [pad_head_rows(get(q), nh, self.qk_dim, hd)]
+        if not self.reads_only:
+            rows.append(pad_head_rows(get(k), nkv, self.qk_dim, hd))
+        if not self.values_are_keys and not self.reads_only:
             rows.append(pad_head_rows(get(v), nkv, self.value_dim, hd))
         if self.gate_name and self.gate_per_entry:
             rows.append(pad_head_rows(get(self.gate_name), nh, self.value_dim, hd))
@@ -177,6 +203,7 @@ class AttentionMixer(Mixer):
         head_scale = get(self.head_scale_name).to(torch.float32) if self.head_scale_name else None
         self.kernel_scale, self.head_scale, self.head_scale_positive = signed_scale(self.scale, head_scale, nh, runtime.device)
         self.sink = get(self.sink_name).contiguous() if self.sink_name else None
+        self.output_bias = get(self.o_bias_name).contiguous() if self.o_bias_name else None
         if self.position is not None:
             self.position.bind(get, runtime)
         attention_kernels.prepare(self.head_dim)
@@ -201,19 +228,22 @@ class AttentionMixer(Mixer):
         nh, nkv, hd = self.num_heads, self.num_kv_heads, self.head_dim
         T = x.shape[0]
         ws = ctx.workspace
-        width = (nh + (1 if self.values_are_keys else 2) * nkv) * hd
+        width = (nh + (0 if self.reads_only else 1 if self.values_are_keys else 2) * nkv) * hd
         qkv = ws.get("qkv", (T, width + self.gate_rows), rt.dtype)
         # a position encoding may know how to run the product itself, with its own work in the epilogue
+        queries = qkv
         fused = getattr(self.position, "product_encode_store", None) if not self.gate_rows else None
         if fused is None or not fused(qkv, x, self.w_qkv, (nh, nkv, hd), ctx, cache.kv, cache.write):
             ops.linear(qkv, x, self.w_qkv, ctx.status)
-            if self.position is not None:
+            if self.encodes_rows:
+                queries = self.position.encode_rows(qkv, (nh, nkv, hd), ctx, cache)
+            elif self.position is not None:
                 self.position.encode_and_store(qkv, (nh, nkv, hd), ctx, cache.kv, cache.write)
             elif cache.write:
                 ops.kv_store(qkv, nh * hd, (nh + nkv) * hd, cache.kv.k, cache.kv.v, ctx.positions, ctx.request_of_token,
                              ctx.block_tables[cache.kv.group], nkv, hd, cache.kv.page_size, ctx.status)
         attn = ws.get("attn", (T, nh * hd), rt.dtype)
-        attention_kernels.run(attn, qkv, ctx, cache.kv, nh, nkv, hd, self.reach, self.kernel_scale, self.head_scale,
+        attention_kernels.run(attn, queries, ctx, cache.kv, nh, nkv, hd, self.reach, self.kernel_scale, self.head_scale,
                               self.head_scale_positive, keep_first=self.keep_first, softcap=self.softcap, sink=self.sink)
         if self.gate_per_entry:
             target = out if out is not None else attn

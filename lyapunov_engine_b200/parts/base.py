@@ -182,6 +182,13 @@ class PositionEncoding(Part):
 
 
 class Mixer(Part):
+    # a bias [H] (32-bit) on the output that forward() leaves to the block that adds the output to the stream (named
+    # by ``o_bias_name``; blocks that add none refuse such a mixer)
+    o_bias_name: str | None = None
+    output_bias = None
+    # True: the mixer writes no keys of its own, its runs must read another run's
+    reads_only = False
+
     def cache_need(self) -> KVNeed | None:
         return None
 
@@ -240,12 +247,20 @@ class StreamInput(Part):
 
 class NormedAddend:
     """How a pending output enters the stream when it is normed on the way:
-    resid += pending / sqrt(mean(pending^2) + eps) * weight (weight [W],
-    32-bit).  A norm that reads such a stream applies it in its own kernel."""
-    __slots__ = ("weight", "eps")
+    with y = pending + ``input_bias``,
+        resid += (y - mean) / sqrt(var + eps) * weight + bias
+    where var is the mean of the squared deviations; not ``centered``: mean is
+    0, a root mean square norm.  ``weight`` [W], ``bias`` and ``input_bias`` [W]
+    or None, all 32-bit; a factor on what enters is a factor on weight and
+    bias.  A norm that reads such a stream applies it in its own kernel."""
+    __slots__ = ("weight", "eps", "bias", "centered", "input_bias")
 
-    def __init__(self, weight, eps: float):
-        self.weight, self.eps = weight, float(eps)
+    def __init__(self, weight, eps: float, bias=None, centered: bool = False, input_bias=None):
+        self.weight, self.eps, self.bias, self.centered, self.input_bias = weight, float(eps), bias, bool(centered), input_bias
+
+    def plain(self) -> bool:
+        """Whether it is a root mean square norm with a weight alone."""
+        return self.bias is None and self.input_bias is None and not self.centered
 
 
 class ScaledAddend:

@@ -15,20 +15,34 @@ sub-layer's output enters the stream times its factor, h = h + s1 *
 mixer(norm1(h)); h = h + s2 * feed_forward(norm2(h)); the norm's kernel that
 adds the output multiplies it.
 
+With output norms (``mixer_output_norm``, ``feed_forward_output_norm``:
+norms of the registry; "norm before and after each sub-layer") a sub-layer's
+output enters through a norm of its own and times ``output_scale`` m:
+    h = h + m * norm1b(mixer(norm1(h)));  h = h + m * norm2b(feed_forward(norm2(h)))
+The output's norm (with m in its weight and bias, and the bias of the mixer's
+output product before it), the addition and the next norm are one kernel.
+
 "parallel": both sub-layers read the same stream (see ``ParallelBlock``).
 """
 from __future__ import annotations
 
 from .. import ops
-from .base import (BLOCKS, FEED_FORWARDS, INPUT_FILTERS, MIXERS, NORMS, STREAM_INPUTS, Block, PartSpec, ScaledAddend,
-                   SecondAddend, TensorDecl, register_block)
+from .base import (BLOCKS, FEED_FORWARDS, INPUT_FILTERS, MIXERS, NORMS, STREAM_INPUTS, Block, NormedAddend, PartSpec,
+                   ScaledAddend, SecondAddend, TensorDecl, register_block)
+
+
+def refuse_output_bias(mixer) -> None:
+    if mixer.o_bias_name:
+        raise ValueError(f"{type(mixer).__name__} leaves a bias on its output to the block, and this arrangement adds none")
 
 
 @register_block("prenorm")
 class PreNormBlock(Block):
     def __init__(self, mixer: PartSpec, feed_forward: PartSpec | None, mixer_norm: PartSpec,
                  feed_forward_norm: PartSpec | None, mixer_input: PartSpec | None = None,
-                 mixer_scale_name: str | None = None, feed_forward_scale_name: str | None = None):
+                 mixer_scale_name: str | None = None, feed_forward_scale_name: str | None = None,
+                 mixer_output_norm: PartSpec | None = None, feed_forward_output_norm: PartSpec | None = None,
+                 output_scale: float = 1.0):
         if (feed_forward is None) != (feed_forward_norm is None):
             raise ValueError("a block has a feed-forward and its norm, or neither")
         self.mixer = MIXERS.build(mixer)
@@ -41,10 +55,25 @@ class PreNormBlock(Block):
         self.mixer_scale = self.feed_forward_scale = None
         if (mixer_scale_name or self.feed_forward_scale_name) and mixer_input is not None:
             raise ValueError("layer scales beside an input filter are not supported")
+        self.mixer_output_norm = NORMS.build(mixer_output_norm) if mixer_output_norm is not None else None
+        self.feed_forward_output_norm = NORMS.build(feed_forward_output_norm) if feed_forward_output_norm is not None else None
+        self.output_scale = float(output_scale)
+        self.mixer_addend = self.feed_forward_addend = None
+        if self.mixer_output_norm is None:
+            refuse_output_bias(self.mixer)
+            if self.feed_forward_output_norm is not None or self.output_scale != 1.0:
+                raise ValueError("output norms and a factor on the outputs come with a norm of the mixer's output")
+        else:
+            if (feed_forward is None) != (feed_forward_output_norm is None):
+                raise ValueError("both sub-layers' outputs are normed, or neither's")
+            if any(getattr(n, "groups", 1) != 1 for n in (self.mixer_output_norm, self.feed_forward_output_norm) if n is not None):
+                raise ValueError("an output's norm runs over whole rows")
+            if mixer_scale_name or feed_forward_scale_name or mixer_input is not None:
+                raise ValueError("output norms beside layer scales or an input filter are not supported")
 
     def parts(self):
-        return [p for p in (self.mixer_norm, self.mixer_input, self.mixer, self.feed_forward_norm, self.feed_forward)
-                if p is not None]
+        return [p for p in (self.mixer_norm, self.mixer_input, self.mixer, self.mixer_output_norm, self.feed_forward_norm,
+                            self.feed_forward, self.feed_forward_output_norm) if p is not None]
 
     def extra_state_needs(self):
         needs = dict(self.mixer.extra_state_needs())
@@ -68,11 +97,34 @@ class PreNormBlock(Block):
         self.mixer_scale = get(self.mixer_scale_name).contiguous() if self.mixer_scale_name else None
         self.feed_forward_scale = get(self.feed_forward_scale_name).contiguous() if self.feed_forward_scale_name else None
 
+        if self.mixer_output_norm is not None:
+            self.mixer_addend = self._addend(self.mixer_output_norm, self.mixer.output_bias)
+        if self.feed_forward_output_norm is not None:
+            self.feed_forward_addend = self._addend(self.feed_forward_output_norm,
+                                                    getattr(self.feed_forward, "output_bias", None))
+
+    def _addend(self, norm, input_bias) -> NormedAddend:
+        """How a sub-layer's output enters the stream through ``norm``, times the block's factor."""
+        bias = getattr(norm, "bias", None)
+        return NormedAddend((norm.weight * self.output_scale).contiguous(), norm.eps,
+                            bias=(bias * self.output_scale).contiguous() if bias is not None else None,
+                            centered=bias is not None, input_bias=input_bias)
+
+    def _forward_normed_outputs(self, stream, ctx, cache) -> None:
+        n = self.mixer_norm.apply_stream(stream, workspace=ctx.workspace)
+        stream.pending, stream.update = self.mixer.forward(n, ctx, cache), self.mixer_addend
+        if self.feed_forward is not None:
+            n = self.feed_forward_norm.apply_stream(stream, workspace=ctx.workspace)
+            stream.pending, stream.update = self.feed_forward.forward(n, ctx), self.feed_forward_addend
+
     def _leave(self, stream, output, scale) -> None:
         stream.pending = output
         stream.update = ScaledAddend(scale) if scale is not None else None
 
     def forward(self, stream, ctx, cache) -> None:
+        if self.mixer_output_norm is not None:
+            self._forward_normed_outputs(stream, ctx, cache)
+            return
         if self.mixer_scale is not None or self.feed_forward_scale is not None or isinstance(stream.update, ScaledAddend):
             # (a pending output with a factor per column: the norms' kernels multiply as they add)
             n = self.mixer_norm.apply_stream(stream, workspace=ctx.workspace)
@@ -94,7 +146,7 @@ class PreNormBlock(Block):
                 n = self.mixer_input.forward(self.mixer_norm.apply(stream.resid, stream.pending, workspace=ctx.workspace),
                                              ctx, state)
         else:
-            n = self.mixer_norm.apply(stream.resid, stream.pending, workspace=ctx.workspace)
+            n = self.mixer_norm.apply_stream(stream, workspace=ctx.workspace)
         a = self.mixer.forward(n, ctx, cache)
         if self.feed_forward is None:
             stream.pending = a
@@ -129,6 +181,7 @@ class ParallelBlock(Block):
         self.mixer_norm = NORMS.build(mixer_norm)
         self.feed_forward_norm = NORMS.build(feed_forward_norm) if feed_forward_norm is not None else None
         self.after = STREAM_INPUTS.build(after) if after is not None else None
+        refuse_output_bias(self.mixer)
         if not hasattr(self.mixer_norm, "apply_pair"):
             raise ValueError("the parallel arrangement needs norms that run as a pair (rmsnorm)")
 

@@ -13,6 +13,7 @@ S = 1 is allowed (one copy with a factor on every path).
 from __future__ import annotations
 
 from .base import FEED_FORWARDS, MIXERS, NORMS, Block, Part, PartSpec, TensorDecl, register_block
+from .block import refuse_output_bias
 
 
 class StreamLink(Part):
@@ -44,6 +45,7 @@ class HyperPreNormBlock(Block):
             raise ValueError(f"the residual stream is kept in 1 to 8 copies, got {copies}")
         self.mixer = MIXERS.build(mixer)
         self.feed_forward = FEED_FORWARDS.build(feed_forward) if feed_forward is not None else None
+        refuse_output_bias(self.mixer)
         self.mixer_norm = NORMS.build(mixer_norm)
         self.feed_forward_norm = NORMS.build(feed_forward_norm) if feed_forward_norm is not None else None
         self.mixer_link = StreamLink(self.copies, **mixer_link)

@@ -12,6 +12,22 @@ from .. import ops
 from .base import Norm, NormedAddend, ScaledAddend, SecondAddend, TensorDecl, register_norm
 
 
+def normed_addend_stream(norm, stream, weight, bias, centered, rows, workspace, key):
+    """``norm`` of a stream in one copy whose pending output enters through a
+    norm of its own (``NormedAddend``), both in one kernel."""
+    if stream.copies != 1 or getattr(norm, "groups", 1) != 1:
+        raise ValueError("an output that enters through a norm takes a stream in one copy and a norm over whole rows")
+    update, W = stream.update, norm.hidden_size
+    ws = workspace or norm.runtime.workspace
+    out = ws.get(key, (stream.resid.shape[0] if rows is None else rows.shape[0], W), norm.runtime.dtype)
+    ops.addend_norm(out, stream.resid, weight, bias, norm.eps, centered, addend=stream.pending, addend_bias=update.input_bias,
+                    addend_weight=update.weight, addend_norm_bias=update.bias, addend_eps=update.eps,
+                    addend_centered=update.centered, rows=rows)
+    if rows is None:
+        stream.pending = stream.update = None
+    return out
+
+
 @register_norm("rmsnorm")
 class RMSNorm(Norm):
     """``groups`` > 1: the row is cut into that many equal consecutive parts,
@@ -59,6 +75,8 @@ class RMSNorm(Norm):
             if rows is None:
                 stream.pending = stream.update = None
             return out
+        if isinstance(stream.update, NormedAddend) and not stream.update.plain():
+            return normed_addend_stream(self, stream, self.weight, None, False, rows, workspace, key)
         if not isinstance(stream.update, (NormedAddend, SecondAddend)):
             return super().apply_stream(stream, read, rows, workspace, key)
         return self.apply_pair(stream, None, rows=rows, workspace=workspace, keys=(key, None))[0]
@@ -71,7 +89,7 @@ class RMSNorm(Norm):
             raise ValueError("norms that run as a pair read one copy of the stream, whole rows, with one eps")
         update = stream.update
         second = update.other if isinstance(update, SecondAddend) else None
-        normed = update if isinstance(update, NormedAddend) else None
+        normed = update if isinstance(update, NormedAddend) and update.plain() else None
         if update is not None and second is None and normed is None:
             raise ValueError(f"{type(self).__name__} cannot apply a pending {type(update).__name__}")
         n = stream.resid.shape[0] if rows is None else rows.shape[0]
@@ -119,6 +137,8 @@ class LayerNorm(Norm):
         return out
 
     def apply_stream(self, stream, read=None, rows=None, workspace=None, key="normed"):
+        if isinstance(stream.update, NormedAddend) and read is None:
+            return normed_addend_stream(self, stream, self.weight, self.bias, True, rows, workspace, key)
         T, W = stream.resid.shape[0], self.hidden_size
         copies = read.copies if read is not None else stream.copies
         init = None

@@ -99,9 +99,9 @@ class RotaryEncoding(PositionEncoding):
 
 
 def pair_rates(rot: int, base: float) -> torch.Tensor:
-    """f_i = base^(-2i / rot), i < rot / 2: made in 64 bits, kept as float32."""
+    """f_i = base^(-2i / rot), i < rot / 2, in 64 bits (the kernels take the angle in 64 bits)."""
     i = torch.arange(0, rot, 2, dtype=torch.float64)
-    return torch.pow(torch.tensor(float(base), dtype=torch.float64), -i / max(rot, 1)).to(torch.float32)
+    return torch.pow(torch.tensor(float(base), dtype=torch.float64), -i / max(rot, 1))
 
 
 @register_position_encoding("rotary_pairs")
@@ -113,9 +113,9 @@ class RotaryPairsEncoding(PositionEncoding):
     turn every head of queries and keys is divided by sqrt(mean(head^2) +
     unit_eps) (a norm without a weight).  ``values_are_keys``: the projection
     has no values of its own; the value pool receives the keys as projected,
-    before turn and norm.  No table: the angle (position times rate), sine and
-    cosine are computed in 32 bits from the step's own positions, so there is no
-    longest position.  ``head_dim`` is the real size of queries and keys; the
+    before turn and norm.  No table: the angle (position times rate, in 64 bits),
+    sine and cosine (in 32) are made from the step's own positions, so there is
+    no longest position.  ``head_dim`` is the real size of queries and keys; the
     heads the kernels see may be padded with zeros behind it."""
     padded_heads_ok = True
 
@@ -305,3 +305,103 @@ class NormedRotaryEncoding(PositionEncoding):
                               ctx.positions, ctx.request_of_token,
                               ctx.block_tables[kv.group] if kv is not None else ctx.block_tables[0], nh, nkv, hd,
                               kv.page_size if kv is not None else 1, write, ctx.status)
+
+
+@register_position_encoding("conv_rotary_pairs")
+class ConvRotaryPairsEncoding(PositionEncoding):
+    """What a projection may pass through on its way to the attention, in one
+    kernel with the cache write: biases on q, k and v (``bias_names``), a short
+    causal convolution over time on every channel of q, k and v (``taps`` taps,
+    the last one the current token's, zeros before the request's start; the
+    weights ``conv_names``, [channels, taps]), rotary positions on neighbouring
+    pairs of the first ``rot`` entries of every head of q and k, and with
+    ``unit_eps`` not None a division of those heads by sqrt(mean(head^2) +
+    unit_eps).  The last taps - 1 projected values of a request are state of
+    its own (``extra_state_needs``).
+
+    The convolution reads rows of earlier tokens, so queries do not stay in
+    place: ``encode_rows`` returns them in a buffer of their own.  Names of
+    keys and values that are None (both): the layer has queries only and reads
+    another layer's keys and values.  ``head_dim`` / ``value_dim`` are the real
+    sizes; the heads the kernels see may be padded with zeros behind them."""
+    padded_heads_ok = True
+
+    def __init__(self, num_heads: int, num_kv_heads: int, head_dim: int, rot: int, base: float, taps: int, conv_names: tuple,
+                 bias_names: tuple | None = None, unit_eps: float | None = None, value_dim: int | None = None):
+        self.num_heads, self.num_kv_heads, self.head_dim = int(num_heads), int(num_kv_heads), int(head_dim)
+        self.value_dim = int(value_dim) if value_dim else self.head_dim
+        self.rot, self.base, self.taps = int(rot), float(base), int(taps)
+        if self.rot % 2 or not 0 <= self.rot <= self.head_dim:
+            raise ValueError(f"rotary width {rot} must be even and at most the head size {head_dim}")
+        if not 1 <= self.taps <= ops.SHORT_CONV_MAX_TAPS:
+            raise ValueError(f"a short convolution takes 1..{ops.SHORT_CONV_MAX_TAPS} taps, got {taps}")
+        self.unit_eps = float(unit_eps) if unit_eps is not None else None
+        self.conv_names = tuple(conv_names)
+        self.bias_names = tuple(bias_names) if bias_names else None
+        self.queries_only = self.conv_names[1] is None
+        self.padded = self.head_dim
+        self.rates = self.bias = self.w_taps = None
+        self.runtime = None
+
+    def set_geometry(self, padded_head_dim: int) -> None:
+        """The head size of kernels and pages (at least the real sizes)."""
+        self.padded = int(padded_head_dim)
+
+    def _kinds(self):
+        """(heads, real size) of q and, unless the layer has none, k and v."""
+        q = [(self.num_heads, self.head_dim)]
+        return q if self.queries_only else q + [(self.num_kv_heads, self.head_dim), (self.num_kv_heads, self.value_dim)]
+
+    def channels(self) -> int:
+        return sum(heads for heads, _ in self._kinds()) * self.padded
+
+    def extra_state_needs(self):
+        from .base import StateNeed
+        return {"mixer_taps": StateNeed((self.taps - 1, self.channels()), torch.float32)} if self.taps > 1 else {}
+
+    def tile_sizes(self):
+        return [ops.SHORT_CONV_TILE]
+
+    def tensors(self):
+        from .base import TensorDecl
+        decls = []
+        for i, (heads, size) in enumerate(self._kinds()):
+            decls.append(TensorDecl(self.conv_names[i], (heads * size, self.taps), role="vector", init="taps"))
+            if self.bias_names:
+                decls.append(TensorDecl(self.bias_names[i], (heads * size,), role="vector", init="taps"))
+        return decls
+
+    def bind(self, get, runtime):
+        key = ("rotary_pairs", self.rot, self.base)
+        rates = runtime.shared.get(key)
+        if rates is None:
+            rates = runtime.shared[key] = pair_rates(max(self.rot, 2), self.base).to(runtime.device).contiguous()
+        self.rates = rates
+
+        def padded(t, heads, size):          # [heads * size, n] -> [heads * padded, n], zeros behind every head's entries
+            out = torch.zeros((heads, self.padded, t.shape[1]), dtype=torch.float32, device=t.device)
+            out[:, :size] = t.view(heads, size, t.shape[1])
+            return out.view(heads * self.padded, t.shape[1])
+
+        kinds = self._kinds()
+        self.w_taps = torch.cat([padded(get(n), *k) for n, k in zip(self.conv_names, kinds)]).t().contiguous()
+        if self.bias_names:
+            self.bias = torch.cat([padded(get(n)[:, None], *k) for n, k in zip(self.bias_names, kinds)]).view(-1).contiguous()
+        self.runtime = runtime
+
+    def encode_rows(self, qkv, geometry, ctx, cache):
+        """The queries as the attention reads them [T, heads * padded]; keys
+        and values go to the pages when the layer writes them."""
+        nh, nkv, hd = geometry
+        kv = cache.kv
+        write = cache.write and not self.queries_only
+        out = ctx.workspace.get("conv_queries", (qkv.shape[0], nh * hd), qkv.dtype)
+        if ctx.pure_decode:
+            tiles = (None, None, ctx.num_requests)       # one token per request: request b is row b
+        else:
+            tiles = ctx.tiles[ops.SHORT_CONV_TILE][:3]
+        ops.conv_turn_store(out, qkv, self.bias, self.w_taps, (cache.extra or {}).get("mixer_taps"), ctx.state_slots, ctx.cu_q,
+                            *tiles, self.rates, self.rot, 1.0, self.unit_eps, self.head_dim, kv.k if write else None,
+                            kv.v if write else None, ctx.positions, ctx.block_tables[kv.group], nh,
+                            0 if self.queries_only else nkv, hd, kv.page_size, write, ctx.status)
+        return out

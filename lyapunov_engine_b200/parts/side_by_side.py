@@ -30,6 +30,8 @@ class SideBySideMixer(Mixer):
         for m in self.mixers:
             if not all(hasattr(m, a) for a in ("forward_inner", "inner_width", "output_weight")):
                 raise ValueError(f"{type(m).__name__} cannot stand side by side: it does not hand on what its output projection reads")
+        if any(m.o_bias_name for m in self.mixers):
+            raise ValueError("mixers side by side share one output product, which adds no bias")
         if sum(m.cache_need() is not None for m in self.mixers) > 1:
             raise ValueError("of mixers side by side at most one keeps pages")
         # columns of the shared buffer, each mixer's start a 16-byte multiple

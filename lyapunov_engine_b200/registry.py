@@ -52,6 +52,7 @@ def _register_builtin() -> None:
     from .models.sulepel import sulepel_spec
     from .models.zepilix import zepilix_spec
     from .models.ribozen import ribozen_spec
+    from .models.zamizen import zamizen_spec
     from .models.zuzenex import zuzenex_spec
 
     register_architecture("LlamaForCausalLM", llama_spec)
@@ -61,6 +62,7 @@ def _register_builtin() -> None:
     register_architecture("Zepilix", zepilix_spec)
     register_architecture("Ribozen", ribozen_spec)
     register_architecture("Zuzenex", zuzenex_spec)
+    register_architecture("Zamizen", zamizen_spec)
 
 
 _register_builtin()
