@@ -2254,6 +2254,253 @@ def run_zuzenex(args):
     return 0
 
 
+# ---------------------------------------------------------------------------------------------- Zamizen
+ZAMIZEN_LATENT, ZAMIZEN_TURNED, ZAMIZEN_TAPS = 64, 64, 4
+
+
+def zamizen_config(llama: dict) -> dict:
+    """A Zamizen model with the width, feed-forward size, heads, head size, vocabulary and number of layers of the given
+    Llama shapes: latent attention, attention, latent attention, attention that reads the keys of the one before it, and
+    so on."""
+    nh, nkv, hd, W = llama["num_attention_heads"], llama["num_key_value_heads"], llama["head_dim"], llama["hidden_size"]
+    mlp = {"kind": "dense", "ff": llama["intermediate_size"]}
+    layers = []
+    for i in range(llama["num_hidden_layers"]):
+        if i % 2 == 0:
+            mixer = {"heads": nh, "dim": hd, "rot_dim": ZAMIZEN_TURNED, "vdim": hd, "kv_rank": ZAMIZEN_LATENT,
+                     "scale": (hd + ZAMIZEN_TURNED) ** -0.5,
+                     "rot": {"dims": ZAMIZEN_TURNED, "base": 500000.0,
+                             "scaling": {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}
+        else:
+            mixer = {"heads": nh, "kv_heads": nkv, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "conv": ZAMIZEN_TAPS,
+                     "rot": {"dims": hd // 2, "base": 500000.0}}
+            if i % 4 == 3:
+                mixer["kv_from"] = i - 2
+        layers.append({"type": "attention" if i % 2 else "latent_attention", "mixer": mixer, "mlp": mlp})
+    return {"architecture": "Zamizen", "vocab": llama["vocab_size"], "width": W, "norm": {"eps": 1e-5}, "residual_mult": 0.8,
+            "layers": layers}
+
+
+def zamizen_decode_bytes(cfg, batch, context):
+    """Bytes one decode step of a Zamizen model must move: the bfloat16 weights, each live request's keys and values (of
+    a layer that reads another's too: a long context does not stay in the L2) or latents, and the convolutions' state."""
+    W, V = cfg["width"], cfg["vocab"]
+    total = 2 * V * W + 8 * W
+    for layer in cfg["layers"]:
+        m, F = layer["mixer"], layer["mlp"]["ff"]
+        H, d, e = m["heads"], m["dim"], m["vdim"]
+        total += 2 * (3 * F * W + W * H * e) + 4 * 8 * W
+        if layer["type"] == "attention":
+            G = m["kv_heads"]
+            C = H * d + (0 if "kv_from" in m else G * (d + e))
+            total += 2 * C * W + 4 * C * (m["conv"] + 1) + batch * (2 * 4 * C * (m["conv"] - 1) + 2 * context * G * (d + e))
+        else:
+            r, t = m["kv_rank"], m["rot_dim"]
+            total += 2 * ((H * (d + t) + r + t + H * e) * W + H * (d + e) * r) + 2 * batch * context * (r + t)
+    return total
+
+
+def zamizen_prefill_flops(cfg, tokens):
+    """Flops of the matrix products and of the attentions as computed here (latent attention over the latents)."""
+    W, V = cfg["width"], cfg["vocab"]
+    flops, pairs = 2 * V * W, tokens * (tokens + 1) // 2
+    for layer in cfg["layers"]:
+        m, F = layer["mixer"], layer["mlp"]["ff"]
+        H, d, e = m["heads"], m["dim"], m["vdim"]
+        flops += 2 * tokens * (3 * F * W + W * H * e)
+        if layer["type"] == "attention":
+            C = H * d + (0 if "kv_from" in m else m["kv_heads"] * (d + e))
+            flops += 2 * tokens * C * W + 2 * H * (d + e) * pairs
+        else:
+            r, t = m["kv_rank"], m["rot_dim"]
+            flops += 2 * tokens * ((H * (d + t) + r + t + H * e) * W + H * (d + e) * r) + 2 * H * (2 * r + t) * pairs
+    return flops
+
+
+def zamizen_kernel_rows(pk, llama):
+    """Each kernel the design adds, alone, beside the like kernel of the closest existing path at the same sizes:
+    microseconds per launch inside a captured graph over rotating tensors and the share of the measured copy bandwidth
+    that the bytes it must move make."""
+    import torch
+
+    from lyapunov_engine_b200 import ops
+    from lyapunov_engine_b200.parts.rope import pair_rates, ramped_rates
+
+    dev = "cuda:0"
+    W, nh, nkv, hd = llama["hidden_size"], llama["num_attention_heads"], llama["num_key_value_heads"], llama["head_dim"]
+    r, t, taps, page = ZAMIZEN_LATENT, ZAMIZEN_TURNED, ZAMIZEN_TAPS, BLOCK_SIZE
+    rows = []
+
+    def row(kernel, like, tokens, nbytes, launch, sets):
+        us = graph_median_us(launch, sets)
+        rows.append({"kernel": kernel, "like": like, "tokens": tokens, "us": round(us, 2), "gbs": round(nbytes / us / 1e3, 1),
+                     "hbm_frac": round(nbytes / us / 1e3 / pk["hbm_gbs"], 3)})
+
+    def sets_for(nbytes):
+        return max(2, min(64, (256 << 20) // max(nbytes, 1) + 1))
+
+    bf = torch.bfloat16
+    status = ops.new_status(dev)
+    for T in (1, 8, 2048):
+        # norms around the addition
+        nbytes = T * W * (4 + 2 + 4 + 2) + 20 * W
+        n = sets_for(nbytes)
+        resid = [torch.randn(T, W, device=dev) for _ in range(n)]
+        parts = 4 if T <= 8 else 0        # (a decode step's outputs are partial sums)
+        addend = [(torch.randn(parts, T, W, device=dev) if parts else torch.randn(T, W, device=dev).to(bf)) for _ in range(n)]
+        nbytes += T * W * (4 * parts - 2 if parts else 0)
+        out = [torch.empty(T, W, device=dev, dtype=bf) for _ in range(n)]
+        w1, w2, b1, b2, b3 = (torch.randn(W, device=dev) for _ in range(5))
+        row("output's layer norm + addition + layer norm", "", T, nbytes,
+            lambda i: ops.addend_norm(out[i], resid[i], w1, b1, 1e-5, True, addend=addend[i], addend_bias=b3, addend_weight=w2,
+                                      addend_norm_bias=b2, addend_eps=1e-5, addend_centered=True), n)
+        row("output's rms norm + addition + rms norm (Zepilix)", "output's layer norm + addition + layer norm", T, nbytes,
+            lambda i: ops.rmsnorm_pair(out[i], None, resid[i], w1, None, 1e-5, addend=addend[i], addend_weight=w2, addend_eps=1e-5), n)
+        row("addition + layer norm (Kaditar)", "output's layer norm + addition + layer norm", T, nbytes,
+            lambda i: ops.stream_norm(out[i], resid[i].view(T, 1, W), w1, b1, 1e-5, delta=addend[i]), n)
+        row("addition + rms norm (Llama)", "output's layer norm + addition + layer norm", T, nbytes,
+            lambda i: ops.rmsnorm(out[i], resid[i], addend[i], w1, 1e-5), n)
+        del resid, addend, out
+        # queries, keys and values on their way to the attention
+        C = (nh + 2 * nkv) * hd
+        reqs = T if T <= 64 else 1
+        cu = torch.arange(0, T + 1, T // reqs, dtype=torch.int32, device=dev)
+        tiles = (None, None, reqs)
+        if T > 64:
+            q0 = torch.arange(0, T, ops.SHORT_CONV_TILE, dtype=torch.int32, device=dev)
+            tiles = (torch.zeros_like(q0), q0, q0.numel())
+        slots = torch.arange(reqs, dtype=torch.int32, device=dev)
+        pages = (T + page - 1) // page + 1
+        table = torch.arange(pages, dtype=torch.int32, device=dev).view(1, -1).repeat(reqs, 1).contiguous()
+        req = torch.zeros(T, dtype=torch.int32, device=dev) if T > 64 else torch.arange(T, dtype=torch.int32, device=dev)
+        pos = torch.arange(T, dtype=torch.int32, device=dev)
+        nbytes = T * C * 4
+        n = sets_for(nbytes)
+        src = [torch.randn(T, C, device=dev).to(bf) for _ in range(n)]
+        conv = [torch.empty(T, C, device=dev, dtype=bf) for _ in range(n)]
+        state = [torch.zeros(reqs + 1, taps - 1, C, device=dev) for _ in range(min(n, 8))]
+        wt, bias = torch.randn(taps, C, device=dev), torch.randn(C, device=dev)
+        kc = [torch.zeros(pages + 1, nkv, page, hd, device=dev, dtype=bf) for _ in range(n)]
+        vc = [torch.zeros_like(k) for k in kc]
+        rates, narrow = ramped_rates(hd // 2, 5e5, None)[0].to(dev), pair_rates(hd, 5e5).to(dev)
+        more = reqs * (taps - 1) * C * 8 + 4 * C * (taps + 1)
+        row("bias + convolution + turn + norm + cache write", "", T, nbytes + more,
+            lambda i: ops.conv_turn_store(conv[i][:, :nh * hd], src[i], bias, wt, state[i % len(state)], slots, cu, *tiles, rates,
+                                          hd // 2, 1.0, 1e-5, hd, kc[i], vc[i], pos, table, nh, nkv, hd, page, True, status), n)
+        wt_q = wt[:, :nh * hd].contiguous()
+        state_q = [torch.zeros(reqs + 1, taps - 1, nh * hd, device=dev) for _ in range(min(n, 8))]
+        row("queries alone: bias + convolution + turn + norm", "", T, T * nh * hd * 4 + more * nh * hd // C,
+            lambda i: ops.conv_turn_store(conv[i][:, :nh * hd], src[i], bias[:nh * hd], wt_q, state_q[i % len(state_q)], slots, cu,
+                                          *tiles, rates, hd // 2, 1.0, 1e-5, hd, None, None, pos, table, nh, 0, hd, page, False,
+                                          status), n)
+        row("turn of pairs + norm + cache write (Zepilix)", "bias + convolution + turn + norm + cache write", T, T * (nh + 2 * nkv) * hd * 4 - T * nkv * hd * 2,
+            lambda i: ops.rope_norm_store(src[i], kc[i], vc[i], narrow, pos, req, table, nh, nkv, hd, 0, hd, 1e-6, hd, page, True, True, status), n)
+        row("convolution, 4 taps + silu (Zepilix)", "bias + convolution + turn + norm + cache write", T, nbytes + more,
+            lambda i: ops.short_conv_general(conv[i], src[i], wt, state[i % len(state)], slots, cu, *tiles, add_input=False, silu=True), n)
+        del src, conv, kc, vc
+        # latent attention on its way to the attention
+        rp = r + t
+        width = nh * (hd + t) + rp + nh * hd
+        nbytes = T * (nh * t + rp) * 4
+        n = sets_for(T * width * 2)
+        proj = [torch.randn(T, width, device=dev).to(bf) for _ in range(n)]
+        ql = [torch.empty(T, nh * rp, device=dev, dtype=bf) for _ in range(n)]
+        pool = [torch.zeros(pages + 1, 1, page, rp, device=dev, dtype=bf) for _ in range(n)]
+        wl = torch.ones(r, device=dev)
+        rates = ramped_rates(t, 5e5, None)[0].to(dev)
+        place = (pos, req, table, page, status)
+        col = nh * (hd + t)
+        row("latent norm + turned keys and queries + cache write", "", T, nbytes,
+            lambda i: ops.latent_rope_store(proj[i], col, r, t, rp, wl, 1e-5, rates, pool[i], *place, magnitude=1.2,
+                                            queries=(hd, hd + t, nh, ql[i])), n)
+        narrow = pair_rates(t, 5e5).to(dev)
+        row("latent norm + turned keys + cache write (Zepilix)", "latent norm + turned keys and queries + cache write", T, T * rp * 4,
+            lambda i: ops.latent_rope_store(proj[i], col, r, t, rp, wl, 1e-5, narrow, pool[i], *place), n)
+        row("the queries' turn (Zepilix)", "latent norm + turned keys and queries + cache write", T, T * nh * rp * 4,
+            lambda i: ops.rope_norm_store(ql[i], None, None, narrow, pos, req, table, nh, 0, rp, r, t, None, rp, page, False, False, status), n)
+        into = [torch.randn(nh, r, hd, device=dev).to(bf) for _ in range(8)]
+        outof = [torch.randn(nh, hd, rp, device=dev).to(bf) for _ in range(8)]
+        heads = torch.empty(T, nh * hd, device=dev, dtype=bf)
+        if T <= 8:
+            nb = 2 * (nh * r * hd + T * nh * (hd + t + rp)) + T * rp * 4
+            row("latent prepare: product, turns, norm, cache write", "", T, nb,
+                lambda i: ops.latent_prepare(ql[i], proj[i], into[i % 8], col, r, wl, 1e-5, pool[i], *place, rot=t, rates=rates, magnitude=1.2), n)
+            into0 = [torch.randn(nh, rp, hd, device=dev).to(bf) for _ in range(8)]
+            wl0 = torch.ones(rp, device=dev)
+            row("latent prepare: product, norm, cache write (Sulepel)", "latent prepare: product, turns, norm, cache write", T,
+                2 * (nh * rp * hd + T * nh * (hd + rp)) + T * rp * 4,
+                lambda i: ops.latent_prepare(ql[i], proj[i], into0[i % 8], col, rp, wl0, 1e-5, pool[i], *place), n)
+            nb = 2 * (nh * rp * hd + T * nh * (rp + 2 * hd))
+            row("per-head product out of the latent space, gate per entry", "", T, nb,
+                lambda i: ops.gemm_heads(heads, ql[i], outof[i % 8], proj[i][:, col + rp:]), n)
+            row("per-head product out of the latent space, gate per head (Sulepel)", "per-head product out of the latent space, gate per entry",
+                T, nb, lambda i: ops.gemm_heads(heads, ql[i], outof[i % 8], proj[i][:, col + rp:col + rp + nh]), n)
+        else:
+            row("gate per entry", "", T, T * nh * hd * 6, lambda i: ops.sigmoid_gate(heads, heads, proj[i][:, col + rp:]), n)
+            row("gate per head (Sulepel)", "gate per entry", T, T * nh * hd * 4, lambda i: ops.head_gate(heads, proj[i][:, col + rp:col + rp + nh], nh, hd), n)
+        del proj, ql, pool
+    ops.check_status(status)
+    return rows
+
+
+def run_zamizen(args):
+    """--only zamizen: decode (1 and 8 requests at --context) and prefill (2,048 tokens) of a Zamizen model beside the
+    Zepilix model (the closest existing design: latent attention with a rotated part, attention with turned pairs and a
+    norm per head, short convolutions) and the Llama model of the same width, feed-forward size, heads, layers and
+    vocabulary (random weights, bfloat16), and the design's own kernels alone beside their likes."""
+    global BLOCK_SIZE
+    import torch
+
+    BLOCK_SIZE = args.page
+    pk = peaks()
+    context = args.context or CONTEXT
+    if args.profile_step:
+        llama = dict(SHAPES[args.shapes])
+        llama["num_hidden_layers"] = args.layers or 4
+        rig = make_rig(zamizen_config(llama), context, 8, args.page)
+        rig.runner.use_cuda_graphs = False
+        if args.profile_step == "decode":
+            ms, _, _ = rig.timed_decode(args.batch, 2, 2, context)
+        else:
+            ms = rig.timed_prefill(args.tokens or PREFILL_TOKENS, 1, 2)
+        print(json.dumps({"only": "zamizen", "profile_step": args.profile_step, "layers": llama["num_hidden_layers"], "ms": round(ms, 3)}))
+        return 0
+    out = {"only": "zamizen", "peaks": pk["source"], "context": context, "sizes": {}}
+    for name in ([args.shapes] if args.shapes != "1b" or args.layers else ["1b", "3b"]):
+        llama = dict(SHAPES[name])
+        if args.layers:
+            llama["num_hidden_layers"] = args.layers
+        res = {}
+        for label, cfg in (("zamizen", zamizen_config(llama)), ("zepilix", zepilix_config(llama)), ("llama", llama)):
+            rig = make_rig(cfg, context, 8, args.page)
+            for b in (1, 8):
+                rig.timed_decode(b, 3, 2, context - 200)
+                ms, graph_steps, _ = rig.timed_decode(b, 24, 6, context)
+                nbytes = {"zamizen": zamizen_decode_bytes, "zepilix": zepilix_decode_bytes, "llama": decode_bytes}[label](cfg, b, context - 12)
+                res[f"{label}_decode_b{b}_ms"] = round(ms, 4)
+                res[f"{label}_decode_b{b}_tokens_per_s"] = round(b * 1000.0 / ms, 1)
+                res[f"{label}_decode_b{b}_hbm_frac"] = round(nbytes / (ms * 1e-3) / 1e9 / pk["hbm_gbs"], 4)
+                res[f"{label}_decode_b{b}_graph_steps"] = graph_steps
+            ms = rig.timed_prefill(PREFILL_TOKENS, 3, 2)
+            flops = {"zamizen": zamizen_prefill_flops, "zepilix": lambda c, n: zepilix_prefill_flops(c, n)[0],
+                     "llama": prefill_flops}[label](cfg, PREFILL_TOKENS)
+            res[f"{label}_prefill_{PREFILL_TOKENS}_ms"] = round(ms, 3)
+            res[f"{label}_prefill_{PREFILL_TOKENS}_tokens_per_s"] = round(PREFILL_TOKENS * 1000.0 / ms, 1)
+            res[f"{label}_prefill_{PREFILL_TOKENS}_bf16_frac"] = round(flops / (ms * 1e-3) / 1e12 / pk["bf16_tflops"], 4)
+            rig.close()
+            del rig
+            torch.cuda.empty_cache()
+        out["sizes"][name] = res
+        for k, v in res.items():
+            print(f"{name}  {k} = {v}", file=sys.stderr)
+    rows = zamizen_kernel_rows(pk, dict(SHAPES["1b"]))
+    for r in rows:
+        print("  ".join(f"{k}={v}" for k, v in r.items() if v != ""), file=sys.stderr)
+    out["kernels"] = rows
+    print(json.dumps(out))
+    return 0
+
+
 def main():
     p = argparse.ArgumentParser()
     p.add_argument("--gpus", type=int, default=1)
@@ -2261,7 +2508,7 @@ def main():
     p.add_argument("--warmup", type=int, default=16)
     p.add_argument("--impl", default="ours", choices=["ours", "reference"])
     p.add_argument("--layers", type=int, default=0, help="fewer layers than the model has (named in config)")
-    p.add_argument("--only", choices=["decode", "prefill", "mixed", "serving", "kernels", "sulepel", "kaditar", "zepilix", "ribozen", "zuzenex"], default=None,
+    p.add_argument("--only", choices=["decode", "prefill", "mixed", "serving", "kernels", "sulepel", "kaditar", "zepilix", "ribozen", "zuzenex", "zamizen"], default=None,
                    help="run one kind of step and exit (for profilers and for further sizes); mixed = --batch decoding "
                         "requests beside one --tokens portion of a prompt in every step; serving = the reference's "
                         "serving benchmark (small model, prompts of 128 tokens, 32 generated: TTFT, ITL, tokens/s); "
@@ -2269,7 +2516,8 @@ def main():
                         "sulepel = the Sulepel design beside Llama at equal sizes (decode, prefill, its kernels alone); "
                         "kaditar = the same for the Kaditar design; zepilix = the Zepilix design beside Sulepel and Llama; "
                         "ribozen = the Ribozen design beside Zepilix and Llama; "
-                        "zuzenex = the Zuzenex design beside Ribozen and Llama")
+                        "zuzenex = the Zuzenex design beside Ribozen and Llama; "
+                        "zamizen = the Zamizen design beside Zepilix and Llama")
     p.add_argument("--batch-sizes", nargs="+", type=int, default=[1, 4, 8, 16], help="with --only serving")
     p.add_argument("--shapes", choices=sorted(SHAPES), default="1b", help="with --only: layer sizes of Llama-3.2-1B, 3.2-3B or 3.1-8B")
     p.add_argument("--batch", type=int, default=8, help="batch of --only decode")
@@ -2283,7 +2531,7 @@ def main():
     p.add_argument("--without", choices=["norms", "qkv", "attention", "o", "gate_up", "down", "head"], default=None,
                    help="with --only decode (batches up to 16): time the step with this kind of kernel left out")
     p.add_argument("--profile-step", choices=["decode", "prefill"], default=None,
-                   help="with --only sulepel, kaditar, zepilix, ribozen or zuzenex: run a few steps of that kind launch by launch (no captured graph) on a model of "
+                   help="with --only sulepel, kaditar, zepilix, ribozen, zuzenex or zamizen: run a few steps of that kind launch by launch (no captured graph) on a model of "
                         "--layers layers (4 by default) and exit; for profilers")
     p.add_argument("--points", choices=["all", "1b"], default="all",
                    help="all: also decode, prefill and the mixed step at the 3B and 8B shapes (context 8192) in `points`")
@@ -2307,6 +2555,8 @@ def main():
         return run_ribozen(args)
     if args.only == "zuzenex" and args.impl == "ours":
         return run_zuzenex(args)
+    if args.only == "zamizen" and args.impl == "ours":
+        return run_zamizen(args)
     if args.impl == "reference":
         return run_reference(args)
     return run_ours(args)

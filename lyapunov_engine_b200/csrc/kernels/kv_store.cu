@@ -113,7 +113,7 @@ LE_API int le_kv_store(const void *src, int64_t src_stride, int k_col, int v_col
 // le_latent_norm_store (rot 0) or le_latent_rope_store does (cache null: not stored).
 LE_API int le_latent_prepare(const void *src, int64_t src_stride, int num_tokens, int heads, int head_dim, const void *w_into,
                              void *q_latent, int64_t q_latent_stride, int col, int rank, int rot, int padded_rank,
-                             const float *weight, float eps, const double *rates, float magnitude, void *cache, int dtype,
+                             const float *weight, float eps, const void *rates, int rates_wide, float magnitude, void *cache, int dtype,
                              const int32_t *positions, const int32_t *request_of_token, const int32_t *block_table,
                              int max_blocks, int page_size, int num_pages, int *status, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
@@ -126,7 +126,7 @@ LE_API int le_latent_prepare(const void *src, int64_t src_stride, int num_tokens
   const dim3 grid((padded_rank + le_heads::GR_WARPS * le_heads::GR_COLS - 1) / (le_heads::GR_WARPS * le_heads::GR_COLS),
                   heads + (rot > 0 ? 2 : 1), (num_tokens + le_heads::GR_ROWS - 1) / le_heads::GR_ROWS);
   LE_DISPATCH_DTYPE(dtype, T, {
-    le_latent::Args<T> a{static_cast<const T *>(src), src_stride, col, rank, rot, padded_rank, weight, eps, rates, magnitude,
+    le_latent::Args<T> a{static_cast<const T *>(src), src_stride, col, rank, rot, padded_rank, weight, eps, le::Rates{rates, rates_wide}, magnitude,
                          static_cast<T *>(cache), positions, request_of_token, block_table, max_blocks, page_size, num_pages,
                          status, head_dim, head_dim + rot, heads, static_cast<T *>(q_latent), q_latent_stride, 0};
     a.q_pairs = le_latent::pairs_together(a);
@@ -144,7 +144,7 @@ LE_API int le_latent_norm_store(const void *src, int64_t src_stride, int col, in
   if (rank < 1 || padded_rank < rank) return le::invalid("le_latent_norm_store: rank %d, padded rank %d", rank, padded_rank);
   const int threads = rank >= 512 ? 256 : 128;
   LE_DISPATCH_DTYPE(dtype, T, {
-    const le_latent::Args<T> a{static_cast<const T *>(src), src_stride, col, rank, 0, padded_rank, weight, eps, nullptr, 1.0f,
+    const le_latent::Args<T> a{static_cast<const T *>(src), src_stride, col, rank, 0, padded_rank, weight, eps, le::Rates{nullptr, 0}, 1.0f,
                                static_cast<T *>(cache), positions, request_of_token, block_table, max_blocks, page_size,
                                num_pages, status, 0, 0, 0, nullptr, 0, 0};
     return le::launch_chained(latent_norm_store_kernel<T>, dim3(num_tokens), dim3(threads), 0, stream, a);

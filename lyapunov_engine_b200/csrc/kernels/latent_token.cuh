@@ -17,7 +17,7 @@ struct Args {
   int col, rank, rot, padded;       // the latent at columns [col, col + rank), its rotated part in the rot columns behind it
   const float *weight;              // [rank]
   float eps;
-  const double *rates;              // [rot / 2]
+  le::Rates rates;                  // [rot / 2]
   float magnitude;                  // on cosines and sines
   T *cache;                         // [pages, 1, page, padded] or null: nothing is stored
   const int32_t *positions, *request_of_token, *block_table;
@@ -34,7 +34,7 @@ struct Args {
 // Needs no result of the kernel before this one.
 template <typename T>
 __device__ __forceinline__ void make_turns(float2 *turn, const Args<T> &a, int t) {
-  for (int i = threadIdx.x; i < (a.rot >> 1); i += blockDim.x) turn[i] = le::turn_of(a.positions[t], a.rates[i], a.magnitude);
+  for (int i = threadIdx.x; i < (a.rot >> 1); i += blockDim.x) turn[i] = le::turn_of(a.positions[t], a.rates, i, a.magnitude);
 }
 
 // The whole block; `turn` is made, `scratch` holds 33 floats.

@@ -18,8 +18,8 @@
 // `values_are_keys`, the value heads [kv_heads][head_dim] behind the keys as
 // they are when `store_values`, else nothing.  A warp takes a head, a lane up to eight
 // pairs of it; a token's sines and cosines are made once per block, the angle
-// (position times a 64-bit rate) in 64 bits, the rest in 32; the result is
-// rounded once.
+// (position times rate) in 64 bits where the rates are, all else in 32; the
+// result is rounded once.
 //
 // latent_rope_store_kernel.  Columns [col, col + rank) of a token's row are a
 // latent: normed with a weight over `rank`; the `rot` columns behind it are one
@@ -82,7 +82,7 @@ __device__ __forceinline__ void store_pair(T *p, bool together, float u, float v
 template <typename T>
 __global__ void __launch_bounds__(128)
 rope_norm_store_kernel(T *__restrict__ rows, int64_t row_stride, T *__restrict__ k_cache, T *__restrict__ v_cache,
-                       const double *__restrict__ rates, const int32_t *__restrict__ positions,
+                       const le::Rates rates, const int32_t *__restrict__ positions,
                        const int32_t *__restrict__ request_of_token, const int32_t *__restrict__ block_table,
                        int max_blocks, int heads, int kv_heads, int head_dim, int rot_col, int rot, int unit, float eps,
                        int norm_dim, int page_size, int num_pages, int write_kv, int values_are_keys, int heads_per_block,
@@ -93,7 +93,7 @@ rope_norm_store_kernel(T *__restrict__ rows, int64_t row_stride, T *__restrict__
   const int t = blockIdx.x;
   const int pos = positions[t];
   for (int i = threadIdx.x; i < (rot >> 1); i += blockDim.x) {
-    const float2 cs = le::turn_of(pos, rates[i], extras.magnitude);
+    const float2 cs = le::turn_of(pos, rates, i, extras.magnitude);
     turn[2 * i] = cs.y, turn[2 * i + 1] = cs.x;
   }
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
@@ -195,7 +195,7 @@ struct Piece<float> {
 template <typename T>
 __global__ void __launch_bounds__(128)
 rope_norm_store_pieces_kernel(T *__restrict__ rows, int64_t row_stride, T *__restrict__ k_cache, T *__restrict__ v_cache,
-                              const double *__restrict__ rates, const int32_t *__restrict__ positions,
+                              const le::Rates rates, const int32_t *__restrict__ positions,
                               const int32_t *__restrict__ request_of_token, const int32_t *__restrict__ block_table,
                               int max_blocks, int heads, int kv_heads, int head_dim, int rot_col, int rot, int unit, float eps,
                               int norm_dim, int page_size, int num_pages, int write_kv, int values_are_keys,
@@ -208,7 +208,7 @@ rope_norm_store_pieces_kernel(T *__restrict__ rows, int64_t row_stride, T *__res
   const int t = blockIdx.x;
   const int pos = positions[t];
   for (int i = threadIdx.x; i < (rot >> 1); i += blockDim.x) {
-    const float2 cs = le::turn_of(pos, rates[i], extras.magnitude);
+    const float2 cs = le::turn_of(pos, rates, i, extras.magnitude);
     turn[2 * i] = cs.y, turn[2 * i + 1] = cs.x;
   }
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
@@ -313,8 +313,8 @@ latent_rope_store_kernel(const le_latent::Args<T> a, int col2, int rank2, const 
 
 // rows: [tokens] rows of row_stride elements, queries then keys, heads of head_dim entries (even, at most 512).
 // k_cache / v_cache: [pages, kv_heads, page, head_dim].  write_kv 0: queries only (the keys' columns are not read).
-// rates: float64.  w_q / w_k: float32 [head_dim] or null; temp_every 0: no query temperature; store_values: value heads lie behind the keys.
-LE_API int le_rope_norm_store(void *rows, int64_t row_stride, int dtype, void *k_cache, void *v_cache, const double *rates,
+// rates: float64 (rates_wide) or float32.  w_q / w_k: float32 [head_dim] or null; temp_every 0: no query temperature; store_values: value heads lie behind the keys.
+LE_API int le_rope_norm_store(void *rows, int64_t row_stride, int dtype, void *k_cache, void *v_cache, const void *rates, int rates_wide,
                               const int32_t *positions, const int32_t *request_of_token, const int32_t *block_table,
                               int max_blocks, int num_tokens, int heads, int kv_heads, int head_dim, int rot_col, int rot,
                               int unit, float eps, int norm_dim, int page_size, int num_pages, int write_kv,
@@ -343,22 +343,22 @@ LE_API int le_rope_norm_store(void *rows, int64_t row_stride, int dtype, void *k
     LE_DISPATCH_DTYPE(dtype, T,
                       return le::launch_chained(rope_norm_store_pieces_kernel<T>, grid, dim3(128), smem, stream,
                                                 static_cast<T *>(rows), row_stride, static_cast<T *>(k_cache),
-                                                static_cast<T *>(v_cache), rates, positions, request_of_token, block_table,
+                                                static_cast<T *>(v_cache), le::Rates{rates, rates_wide}, positions, request_of_token, block_table,
                                                 max_blocks, heads, kv_heads, head_dim, rot_col, rot, unit, eps, norm_dim,
                                                 page_size, num_pages, write_kv, values_are_keys, per_block, lph, extras, status));
   }
   LE_DISPATCH_DTYPE(dtype, T,
                     return le::launch_chained(rope_norm_store_kernel<T>, grid, dim3(128), smem, stream,
                                               static_cast<T *>(rows), row_stride, static_cast<T *>(k_cache),
-                                              static_cast<T *>(v_cache), rates, positions, request_of_token, block_table,
+                                              static_cast<T *>(v_cache), le::Rates{rates, rates_wide}, positions, request_of_token, block_table,
                                               max_blocks, heads, kv_heads, head_dim, rot_col, rot, unit, eps, norm_dim,
                                               page_size, num_pages, write_kv, values_are_keys, per_block, together, extras, status));
 }
 
 // cache: [pages, 1, page, padded] or null (nothing is stored); out2 null: no second latent; q_out null: no queries are
-// turned (else rows of q_stride elements, heads * padded wide: see latent_token.cuh); rates: float64.
+// turned (else rows of q_stride elements, heads * padded wide: see latent_token.cuh); rates: float64 (rates_wide) or float32.
 LE_API int le_latent_rope_store(const void *src, int64_t src_stride, int dtype, int col, int rank, int rot, int padded,
-                                const float *weight, float eps, const double *rates, float magnitude, void *cache, int col2,
+                                const float *weight, float eps, const void *rates, int rates_wide, float magnitude, void *cache, int col2,
                                 int rank2, const float *weight2, void *out2, int64_t out2_stride, int q_col, int q_head,
                                 int heads, void *q_out, int64_t q_stride, const int32_t *positions,
                                 const int32_t *request_of_token, const int32_t *block_table, int max_blocks, int num_tokens,
@@ -367,7 +367,7 @@ LE_API int le_latent_rope_store(const void *src, int64_t src_stride, int dtype, 
   if (rank < 1 || rot < 0 || rot % 2 || rot > 2 * le_latent::MAX_PAIRS || padded < rank + rot)
     return le::invalid("le_latent_rope_store: rank %d, %d turned entries, padded %d", rank, rot, padded);
   LE_DISPATCH_DTYPE(dtype, T, {
-    le_latent::Args<T> a{static_cast<const T *>(src), src_stride, col, rank, rot, padded, weight, eps, rates, magnitude,
+    le_latent::Args<T> a{static_cast<const T *>(src), src_stride, col, rank, rot, padded, weight, eps, le::Rates{rates, rates_wide}, magnitude,
                          static_cast<T *>(cache), positions, request_of_token, block_table, max_blocks, page_size, num_pages,
                          status, q_col, q_head, heads, static_cast<T *>(q_out), q_stride, 0};
     a.q_pairs = le_latent::pairs_together(a);

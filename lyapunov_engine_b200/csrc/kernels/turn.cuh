@@ -15,6 +15,18 @@ __device__ __forceinline__ float2 turn_of(int position, double rate, float magni
   return make_float2(c * magnitude, s * magnitude);
 }
 
+// Rates in either width: float64 ones as above; float32 ones give the angle position * rate in 32 bits.
+struct Rates {
+  const void *data;
+  int wide;           // 1: float64, 0: float32
+};
+__device__ __forceinline__ float2 turn_of(int position, const Rates &rates, int i, float magnitude) {
+  if (rates.wide) return turn_of(position, static_cast<const double *>(rates.data)[i], magnitude);
+  float s, c;
+  sincosf(static_cast<float>(position) * static_cast<const float *>(rates.data)[i], &s, &c);
+  return make_float2(c * magnitude, s * magnitude);
+}
+
 // Neighbouring entries (u, v) turned.
 __device__ __forceinline__ void turn_pair(float &u, float &v, const float2 &cs) {
   const float nu = u * cs.x - v * cs.y, nv = v * cs.x + u * cs.y;

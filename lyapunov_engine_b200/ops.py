@@ -90,10 +90,10 @@ _CORE_SIGNATURES = {
                             c_float, c_float, c_void_p, c_void_p],
     "le_head_norm_gate": [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_int, c_void_p, c_float, c_int, c_int,
                           c_int, c_int, c_int, c_float, c_void_p],
-    "le_rope_norm_store": [c_void_p, c_int64, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+    "le_rope_norm_store": [c_void_p, c_int64, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
                            c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_int, c_int, c_int,
                            c_void_p, c_void_p, c_float, c_int, c_int, c_float, c_void_p, c_void_p],
-    "le_latent_rope_store": [c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_float,
+    "le_latent_rope_store": [c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_float,
                              c_void_p, c_int, c_int, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_int64,
                              c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
     "le_conv_turn_store": [c_void_p, c_int64, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
@@ -130,7 +130,7 @@ _CORE_SIGNATURES = {
     "le_latent_norm_store": [c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p,
                              c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
     "le_latent_prepare": [c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int,
-                          c_void_p, c_float, c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                          c_void_p, c_float, c_void_p, c_int, c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int,
                           c_int, c_void_p, c_void_p],
     "le_gemm_heads": [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int,
                       c_int, c_int64, c_int64, c_void_p],
@@ -471,13 +471,18 @@ def latent_prepare(q_latent, src, w_into, col, rank, weight, eps, cache, positio
         pages = cache.shape[0]
     _check(core().le_latent_prepare(_ptr(src), src.stride(0), T, heads, head_dim, _ptr(w_into), _ptr(q_latent),
                                     q_latent.stride(0), col, rank, int(rot), padded, _ptr(weight), float(eps), _ptr(rates),
-                                    float(magnitude), _ptr(cache), dtype_code(src.dtype), _ptr(positions),
+                                    _wide(rates), float(magnitude), _ptr(cache), dtype_code(src.dtype), _ptr(positions),
                                     _ptr(request_of_token), _ptr(block_table), block_table.shape[1], page_size, pages,
                                     _ptr(status), _stream()), "le_latent_prepare")
 
 
 def _check_rates(rates, rot: int) -> None:
-    assert rot == 0 or (rates is not None and rates.dtype == torch.float64 and rates.is_contiguous() and rates.numel() >= rot // 2)
+    assert rot == 0 or (rates is not None and rates.dtype in (torch.float64, torch.float32) and rates.is_contiguous()
+                        and rates.numel() >= rot // 2)
+
+
+def _wide(rates) -> int:
+    return 1 if rates is not None and rates.dtype == torch.float64 else 0
 
 
 def gemm_heads(out, a, w, gate=None, a_head: int | None = None, out_head: int | None = None) -> None:
@@ -1404,8 +1409,8 @@ def rope_norm_store(rows, k_cache, v_cache, rates, positions, request_of_token, 
                     temperature=None, store_values: bool = False, magnitude: float = 1.0) -> None:
     """Rows hold query heads, then key heads, ``head_dim`` entries each.  The
     entries (rot_col + 2i, rot_col + 2i + 1) below rot_col + ``rot`` of every
-    head turn by position * rates[i] (``rates`` float64: the angle is taken in
-    64 bits; cosine and sine times ``magnitude``); with ``unit_eps`` not None the head is then divided by sqrt(mean over its first ``norm_dim`` entries of x^2 +
+    head turn by position * rates[i] (``rates`` float64 or float32: the angle is
+    taken in that width; cosine and sine times ``magnitude``); with ``unit_eps`` not None the head is then divided by sqrt(mean over its first ``norm_dim`` entries of x^2 +
     unit_eps).  Queries are rewritten in place, keys go to ``k_cache``, and
     ``v_cache`` receives the keys as they were projected when
     ``values_are_keys``.  ``write_kv`` False: the queries only.  ``w_q`` /
@@ -1428,7 +1433,7 @@ def rope_norm_store(rows, k_cache, v_cache, rates, positions, request_of_token, 
         assert not (values_are_keys or store_values) or (v_cache.shape == k_cache.shape and v_cache.is_contiguous())
         pages = k_cache.shape[0]
     _check(core().le_rope_norm_store(_ptr(rows), rows.stride(0), dtype_code(rows.dtype), _ptr(k_cache) if write_kv else None,
-                                     _ptr(v_cache) if write_kv and (values_are_keys or store_values) else None, _ptr(rates),
+                                     _ptr(v_cache) if write_kv and (values_are_keys or store_values) else None, _ptr(rates), _wide(rates),
                                      _ptr(positions),
                                      _ptr(request_of_token), _ptr(block_table), block_table.shape[1], T, heads, kv_heads,
                                      head_dim, rot_col, rot, 0 if unit_eps is None else 1,
@@ -1441,8 +1446,8 @@ def latent_rope_store(src, col, rank, rot, padded, weight, eps, rates, cache, po
                       page_size, status, second=None, magnitude: float = 1.0, queries=None) -> None:
     """The latent at columns [col, col + rank) of ``src`` is normed (weight
     [rank]) and the ``rot`` columns behind it are turned in neighbouring pairs
-    by position * rates[i] (``rates`` float64; cosine and sine times
-    ``magnitude``); both go to ``cache`` [pages, 1, page, padded] (None: nothing
+    by position * rates[i] (``rates`` float64 or float32: the angle is taken in
+    that width; cosine and sine times ``magnitude``); both go to ``cache`` [pages, 1, page, padded] (None: nothing
     is stored).  ``second`` = (col2, rank2, weight2, out2): a second latent of
     the row is normed into ``out2``.  ``queries`` = (q_col, q_head, heads,
     q_out): the rot columns from q_col + h * q_head of every head h are turned
@@ -1464,7 +1469,7 @@ def latent_rope_store(src, col, rank, rot, padded, weight, eps, rates, cache, po
         assert q_out.dtype == src.dtype and q_out.stride(1) == 1 and q_out.shape == (T, heads * padded)
         assert src.shape[1] >= q_col + (heads - 1) * q_head + rot
     _check(core().le_latent_rope_store(_ptr(src), src.stride(0), dtype_code(src.dtype), col, rank, rot, padded, _ptr(weight),
-                                       float(eps), _ptr(rates), float(magnitude), _ptr(cache), col2, rank2, _ptr(weight2),
+                                       float(eps), _ptr(rates), _wide(rates), float(magnitude), _ptr(cache), col2, rank2, _ptr(weight2),
                                        _ptr(out2), out2.stride(0) if out2 is not None else 0, q_col, q_head, heads, _ptr(q_out),
                                        q_out.stride(0) if q_out is not None else 0, _ptr(positions), _ptr(request_of_token),
                                        _ptr(block_table), block_table.shape[1], T, page_size, pages, _ptr(status), _stream()),
@@ -1497,6 +1502,7 @@ def conv_turn_store(q_out, src, bias, w_taps, state, state_slots, cu_q, tile_req
     assert w_taps.shape[1] == channels and block_table.dtype == torch.int32 and block_table.is_contiguous()
     assert bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == channels)
     _check_rates(rates, rot)
+    assert rot == 0 or _wide(rates)
     rows = pages = 0
     if taps > 1:
         assert state is not None and state.dtype == torch.float32 and state.is_contiguous()

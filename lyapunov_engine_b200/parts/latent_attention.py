@@ -55,7 +55,7 @@ from .. import ops
 from . import attention_kernels
 from .attention import signed_scale
 from .base import KVNeed, Mixer, TensorDecl, register_mixer
-from .rope import ramped_rates
+from .rope import pair_rates, ramped_rates
 
 LIBRARY_ROWS = 64       # bfloat16 steps with more rows than this run the per-head products in the library
 # The most ways a decoded token's latents are cut.  (Capping it at 8, the most that merge inside a thread-block
@@ -143,7 +143,11 @@ class LatentAttentionMixer(Mixer):
         self.q_norm_weight = get(self.q_names[1]) if self.q_rank else None
         self.rates, self.magnitude = None, 1.0
         if rd:
-            rates, self.magnitude = ramped_rates(rd, self.rot_base, self.rot_scaling)
+            # (plain pairs: rates, and so angles, of 32 bits)
+            if self.rot_halves or self.rot_scaling:
+                rates, self.magnitude = ramped_rates(rd, self.rot_base, self.rot_scaling)
+            else:
+                rates = pair_rates(rd, self.rot_base)
             self.rates = rates.to(runtime.device).contiguous()
         # the latent's columns start on a 16-byte boundary of the projection's rows, and so do the gate's
         self.latent_col = (self.q_width + 7) // 8 * 8

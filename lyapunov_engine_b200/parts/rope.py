@@ -99,9 +99,9 @@ class RotaryEncoding(PositionEncoding):
 
 
 def pair_rates(rot: int, base: float) -> torch.Tensor:
-    """f_i = base^(-2i / rot), i < rot / 2, in 64 bits (the kernels take the angle in 64 bits)."""
+    """f_i = base^(-2i / rot), i < rot / 2: made in 64 bits, kept as float32."""
     i = torch.arange(0, rot, 2, dtype=torch.float64)
-    return torch.pow(torch.tensor(float(base), dtype=torch.float64), -i / max(rot, 1))
+    return torch.pow(torch.tensor(float(base), dtype=torch.float64), -i / max(rot, 1)).to(torch.float32)
 
 
 @register_position_encoding("rotary_pairs")
@@ -113,9 +113,9 @@ class RotaryPairsEncoding(PositionEncoding):
     turn every head of queries and keys is divided by sqrt(mean(head^2) +
     unit_eps) (a norm without a weight).  ``values_are_keys``: the projection
     has no values of its own; the value pool receives the keys as projected,
-    before turn and norm.  No table: the angle (position times rate, in 64 bits),
-    sine and cosine (in 32) are made from the step's own positions, so there is
-    no longest position.  ``head_dim`` is the real size of queries and keys; the
+    before turn and norm.  No table: the angle (position times rate), sine and
+    cosine are computed in 32 bits from the step's own positions, so there is no
+    longest position.  ``head_dim`` is the real size of queries and keys; the
     heads the kernels see may be padded with zeros behind it."""
     padded_heads_ok = True
 
@@ -372,11 +372,11 @@ class ConvRotaryPairsEncoding(PositionEncoding):
         return decls
 
     def bind(self, get, runtime):
-        key = ("rotary_pairs", self.rot, self.base)
+        key = ("conv_rotary_pairs", self.rot, self.base)
         rates = runtime.shared.get(key)
         if rates is None:
-            rates = runtime.shared[key] = pair_rates(max(self.rot, 2), self.base).to(runtime.device).contiguous()
-        self.rates = rates
+            rates = runtime.shared[key] = ramped_rates(self.rot, self.base, None)[0].to(runtime.device).contiguous()
+        self.rates = rates                   # (64-bit: the kernel takes the angle in 64 bits)
 
         def padded(t, heads, size):          # [heads * size, n] -> [heads * padded, n], zeros behind every head's entries
             out = torch.zeros((heads, self.padded, t.shape[1]), dtype=torch.float32, device=t.device)

@@ -118,7 +118,6 @@ def test_convolution_turn_norm_and_store_under_every_cut(sizes, rot, taps, unit,
     the taps, over the kernel's tiles) on state rows that others left full;
     queries, stored keys and values equal those of the whole sequences."""
     from lyapunov_engine_b200 import ops
-    from lyapunov_engine_b200.parts.rope import pair_rates
     H, G, d, e = sizes
     hd = (max(d, e) + 15) // 16 * 16
     base, eps, page = 3e3, 1e-5, 8
@@ -139,7 +138,7 @@ def test_convolution_turn_norm_and_store_under_every_cut(sizes, rot, taps, unit,
     order = torch.randperm(pages - 1, generator=g).view(4, 9).to(torch.int32)
     kc = torch.full((pages, G, page, hd), 3.0, dtype=dtype, device=DEV)
     vc = torch.full_like(kc, 3.0)
-    rates = pair_rates(max(rot, 2), base).to(DEV)
+    rates = pz.plain_rates(max(rot, 2), base).to(DEV)
     status = ops.new_status(DEV)
     at = [0] * 4
     got_q = [[] for _ in range(4)]
@@ -191,14 +190,13 @@ def test_queries_alone_rows_of_no_request_and_a_page_outside_the_pool(taps, dtyp
     -1 see zeros before them and keep nothing.  A page outside the pool is
     refused, not followed."""
     from lyapunov_engine_b200 import ops
-    from lyapunov_engine_b200.parts.rope import pair_rates
     H, hd, rot, T = 3, 32, 16, 4
     g = torch.Generator().manual_seed(taps)
     u = torch.randn(T, H * hd, generator=g).to(dtype)
     w = torch.randn(taps, H * hd, generator=g)
     state = torch.randn(3, max(taps - 1, 1), H * hd, generator=g).to(DEV) if taps > 1 else None
     before = state.clone() if taps > 1 else None
-    rates = pair_rates(rot, 100.0).to(DEV)
+    rates = pz.plain_rates(rot, 100.0).to(DEV)
     status = ops.new_status(DEV)
     table = torch.zeros(T, 2, dtype=torch.int32, device=DEV)
     q = torch.empty(T, H * hd, dtype=dtype, device=DEV)
