@@ -28,6 +28,7 @@ namespace {
 
 constexpr int CT_TILE = 16;        // tokens of a tile in the step's lists
 constexpr int CT_THREADS = 128;
+constexpr int CT_WALK = 4;         // tokens that a lane of the form over 16-byte pieces works on at a time
 constexpr int CT_MAX_TAPS = CT_TILE + 1;
 constexpr int CT_MAX_PAIRS = 8;    // pairs a lane of the general form holds: heads of up to 512 entries
 
@@ -74,18 +75,25 @@ __device__ __forceinline__ void make_turns(float2 *turn, const ConvTurnArgs<T> &
     turn[i] = le::turn_of(a.positions[s.first + s.q0 + t], a.rates[j], a.magnitude);
   }
 }
-// Where head `h` (a key head or, behind those, a value head) of the token at `pos` of request b is stored; null: nowhere.
+// Where the stretch's tokens are stored: places[t] is the token's row of its page's first head, in rows of head_dim
+// entries from the pool's start (-1: nowhere).  A head further on is page_size rows further.
 template <typename T>
-__device__ __forceinline__ T *page_place(const ConvTurnArgs<T> &a, int b, int pos, int h) {
+__device__ __forceinline__ void find_places(int64_t *places, const ConvTurnArgs<T> &a, const Stretch &s) {
+  for (int t = threadIdx.x; t < s.n; t += CT_THREADS) {
+    const int pos = a.positions[s.first + s.q0 + t];
+    const int page = pos >= 0 ? a.block_table[static_cast<int64_t>(s.b) * a.max_blocks + pos / a.page_size] : -1;
+    const bool bad = page < 0 || page >= a.num_pages;
+    if (bad) atomicOr(a.status, LE_STATUS_BAD_PAGE);
+    places[t] = bad ? -1 : static_cast<int64_t>(page) * a.kv_heads * a.page_size + pos % a.page_size;
+  }
+}
+// The start of head `h` (a key head or, behind those, a value head) at such a place; null: nowhere.
+template <typename T>
+__device__ __forceinline__ T *page_place(const ConvTurnArgs<T> &a, int64_t place, int h) {
+  if (place < 0) return nullptr;
   const bool is_value = h >= a.heads + a.kv_heads;
   const int kvh = h - a.heads - (is_value ? a.kv_heads : 0);
-  const int page = pos >= 0 ? a.block_table[static_cast<int64_t>(b) * a.max_blocks + pos / a.page_size] : -1;
-  if (page < 0 || page >= a.num_pages) {
-    atomicOr(a.status, LE_STATUS_BAD_PAGE);
-    return nullptr;
-  }
-  return (is_value ? a.v_cache : a.k_cache) +
-         ((static_cast<int64_t>(page) * a.kv_heads + kvh) * a.page_size + pos % a.page_size) * a.head_dim;
+  return (is_value ? a.v_cache : a.k_cache) + (place + static_cast<int64_t>(kvh) * a.page_size) * a.head_dim;
 }
 
 template <int N>
@@ -102,14 +110,41 @@ __device__ __forceinline__ void store_floats(float *p, const float (&s)[N]) {
   for (int i = 0; i < N; i += 4) *reinterpret_cast<float4 *>(p + i) = make_float4(s[i], s[i + 1], s[i + 2], s[i + 3]);
 }
 
+// 16 bytes of a row as floats, and back.
+template <int N>
+__device__ __forceinline__ void open_piece(float (&d)[N], const uint4 &r) {
+  const uint32_t w[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    if constexpr (N == 8) d[2 * i] = __uint_as_float(w[i] << 16), d[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+    else d[i] = __uint_as_float(w[i]);
+  }
+}
+template <int N>
+__device__ __forceinline__ uint4 close_piece(const float (&v)[N], float f) {
+  uint32_t w[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    if constexpr (N == 8) {
+      const __nv_bfloat162 two = __floats2bfloat162_rn(v[2 * i] * f, v[2 * i + 1] * f);
+      w[i] = *reinterpret_cast<const uint32_t *>(&two);
+    } else {
+      w[i] = __float_as_uint(v[i] * f);
+    }
+  }
+  return make_uint4(w[0], w[1], w[2], w[3]);
+}
+
 // 16 bytes of a head per lane (heads of at most 32 such pieces, 2 to 4 taps, everything on 16-byte addresses): a head
-// belongs to `lph` neighbouring lanes (a power of two), so a block takes CT_THREADS / lph heads of its stretch of at most
-// WALK tokens.  A lane keeps its weights and the last TAPS - 1 inputs in registers and asks for all its rows at once.
-template <typename T, int TAPS, int WALK>
+// belongs to `lph` neighbouring lanes (a power of two), so a block takes CT_THREADS / lph heads of its stretch.  A lane
+// keeps its weights and the last TAPS - 1 inputs in registers, walks its tokens CT_WALK at a time, and asks for the next
+// ones' rows before it works on these.
+template <typename T, int TAPS>
 __global__ void __launch_bounds__(CT_THREADS)
 conv_turn_pieces_kernel(const ConvTurnArgs<T> a, int lph) {
   constexpr int N = le::Piece16<T>::COUNT, KEEP = TAPS - 1;
   extern __shared__ float2 turn[];       // [tokens of the stretch][rot / 2]: cosine, sine
+  __shared__ int64_t places[CT_TILE];
   le::let_successor_start();
   const Stretch s = stretch_of(a);
   if (s.n <= 0) return;
@@ -118,6 +153,7 @@ conv_turn_pieces_kernel(const ConvTurnArgs<T> a, int lph) {
   const int at = (threadIdx.x % lph) * N;                   // first entry of the head that this lane holds
   const bool live = h < a.heads + 2 * a.kv_heads && at < a.head_dim;
   const bool is_query = h < a.heads, is_value = h >= a.heads + a.kv_heads;
+  const int turned = is_value || !live ? 0 : a.rot - at;     // this lane's entries below it turn
   const int c = live ? h * a.head_dim + at : 0;
   float w[TAPS][N], bias[N];
 #pragma unroll
@@ -126,6 +162,7 @@ conv_turn_pieces_kernel(const ConvTurnArgs<T> a, int lph) {
   for (int e = 0; e < N; ++e) bias[e] = 0.0f;
   if (a.bias != nullptr) load_floats<N>(bias, a.bias + c);
   make_turns(turn, a, s);
+  if (a.write_kv) find_places(places, a, s);
   float *mine = nullptr;
   if (s.q0 == 0 && live) {
     const int slot = a.state_slots[s.b];
@@ -133,83 +170,91 @@ conv_turn_pieces_kernel(const ConvTurnArgs<T> a, int lph) {
   }
   le::wait_for_predecessor();
   const T *rows = a.src + static_cast<int64_t>(s.first) * a.src_stride + c;
-  uint4 raw[WALK];
+  auto fetch = [&](uint4 (&raw)[CT_WALK], int i0) {
 #pragma unroll
-  for (int i = 0; i < WALK; ++i)
-    if (i < s.n) raw[i] = *reinterpret_cast<const uint4 *>(rows + (s.q0 + i) * a.src_stride);
+    for (int i = 0; i < CT_WALK; ++i)
+      if (i0 + i < s.n) raw[i] = *reinterpret_cast<const uint4 *>(rows + (s.q0 + i0 + i) * a.src_stride);
+  };
+  uint4 next[CT_WALK];
+  fetch(next, 0);
   float past[KEEP][N];
+  auto fetch_past = [&](int q) {         // the KEEP inputs before token q of the step
 #pragma unroll
-  for (int j = 0; j < KEEP; ++j) {
-    if (s.q0 > 0) {                      // (a stretch that is not the first begins at a multiple of WALK >= KEEP)
-      le::load_piece16<T>(past[j], rows + (s.q0 - KEEP + j) * a.src_stride);
+    for (int j = 0; j < KEEP; ++j) {
+      open_piece<N>(past[j], *reinterpret_cast<const uint4 *>(rows + (q - KEEP + j) * a.src_stride));
 #pragma unroll
       for (int e = 0; e < N; ++e) past[j][e] += bias[e];
-    } else if (mine != nullptr) {
-      load_floats<N>(past[j], mine + static_cast<int64_t>(j) * channels);
-    } else {
+    }
+  };
+  if (s.q0 > 0) {                        // (a stretch that is not the first begins at a multiple of CT_WALK >= KEEP)
+    fetch_past(s.q0);
+  } else {
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
 #pragma unroll
       for (int e = 0; e < N; ++e) past[j][e] = 0.0f;
+      if (mine != nullptr) load_floats<N>(past[j], mine + static_cast<int64_t>(j) * channels);
     }
   }
-  __syncthreads();                       // the turns are there
+  __syncthreads();                       // turns and places are there
+  const float2 *my_turn = turn + (at >> 1);
   const int half = a.rot >> 1;
+  const float count = 1.0f / static_cast<float>(a.norm_dim);
+  T *q_row = a.q_out + static_cast<int64_t>(s.first + s.q0) * a.q_stride + c;
+#pragma unroll 1
+  for (int i0 = 0; i0 < s.n; i0 += CT_WALK) {
+    uint4 raw[CT_WALK];
 #pragma unroll
-  for (int i = 0; i < WALK; ++i) {
-    if (i < s.n) {                       // (the same for the whole block)
-      float u[N], y[N];
-      const T *raw_e = reinterpret_cast<const T *>(&raw[i]);
+    for (int i = 0; i < CT_WALK; ++i) raw[i] = next[i];
+    fetch(next, i0 + CT_WALK);
 #pragma unroll
-      for (int e = 0; e < N; ++e) {
-        u[e] = le::to_f32(raw_e[e]) + bias[e];
-        float acc = w[0][e] * past[0][e];
+    for (int i = 0; i < CT_WALK; ++i) {
+      if (i0 + i < s.n) {                // (the same for the whole block)
+        float u[N], y[N];
+        open_piece<N>(u, raw[i]);
 #pragma unroll
-        for (int j = 1; j < KEEP; ++j) acc = fmaf(w[j][e], past[j][e], acc);
-        y[e] = fmaf(w[KEEP][e], u[e], acc);
-      }
+        for (int e = 0; e < N; ++e) {
+          u[e] += bias[e];
+          float acc = w[0][e] * past[0][e];
 #pragma unroll
-      for (int e = 0; e < N; ++e) {
-#pragma unroll
-        for (int j = 0; j + 1 < KEEP; ++j) past[j][e] = past[j + 1][e];
-        past[KEEP - 1][e] = u[e];
-      }
-      float ss = 0.0f;
-      if (live) {
-#pragma unroll
-        for (int e = 0; e < N; e += 2) {
-          if (!is_value && at + e + 1 < a.rot) le::turn_pair(y[e], y[e + 1], turn[i * half + ((at + e) >> 1)]);
-          ss = fmaf(y[e], y[e], fmaf(y[e + 1], y[e + 1], ss));
+          for (int j = 1; j < KEEP; ++j) acc = fmaf(w[j][e], past[j][e], acc);
+          y[e] = fmaf(w[KEEP][e], u[e], acc);
         }
-      }
-      float inv = 1.0f;
-      if (a.unit) {
-        for (int o = 1; o < lph; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-        if (!is_value) inv = rsqrtf(ss / static_cast<float>(a.norm_dim) + a.eps);
-      }
-      T *dst = nullptr;
-      const int t = s.first + s.q0 + i;
-      if (live && is_query) dst = a.q_out + static_cast<int64_t>(t) * a.q_stride + c;
-      else if (live && a.write_kv) {
-        dst = page_place(a, s.b, a.positions[t], h);
-        if (dst != nullptr) dst += at;
-      }
-      if (dst != nullptr) {
-        uint4 packed;
-        T *o = reinterpret_cast<T *>(&packed);
 #pragma unroll
-        for (int e = 0; e < N; ++e) o[e] = le::from_f32<T>(y[e] * inv);
-        *reinterpret_cast<uint4 *>(dst) = packed;
+        for (int e = 0; e < N; ++e) {
+#pragma unroll
+          for (int j = 0; j + 1 < KEEP; ++j) past[j][e] = past[j + 1][e];
+          past[KEEP - 1][e] = u[e];
+        }
+        if (turned > 0) {
+#pragma unroll
+          for (int e = 0; e < N; e += 2)
+            if (e < turned) le::turn_pair(y[e], y[e + 1], my_turn[(e >> 1)]);
+        }
+        my_turn += half;
+        float inv = 1.0f;
+        if (a.unit) {
+          float ss = 0.0f;
+          if (live) {
+#pragma unroll
+            for (int e = 0; e < N; ++e) ss = fmaf(y[e], y[e], ss);
+          }
+          for (int o = 1; o < lph; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+          if (!is_value) inv = rsqrtf(fmaf(ss, count, a.eps));
+        }
+        T *dst = nullptr;
+        if (live && is_query) dst = q_row;
+        else if (live && a.write_kv) {
+          dst = page_place(a, places[i0 + i], h);
+          if (dst != nullptr) dst += at;
+        }
+        q_row += a.q_stride;
+        if (dst != nullptr) *reinterpret_cast<uint4 *>(dst) = close_piece<N>(y, inv);
       }
     }
   }
   if (mine == nullptr) return;
-  if (s.q_len > s.n) {                   // the request goes on beyond this stretch: its last inputs are further down the rows
-#pragma unroll
-    for (int j = 0; j < KEEP; ++j) {
-      le::load_piece16<T>(past[j], rows + (s.q_len - KEEP + j) * a.src_stride);
-#pragma unroll
-      for (int e = 0; e < N; ++e) past[j][e] += bias[e];
-    }
-  }
+  if (s.q_len > s.n) fetch_past(s.q_len);       // the request goes on beyond this stretch: its last inputs are further down the rows
 #pragma unroll
   for (int j = 0; j < KEEP; ++j) store_floats<N>(mine + static_cast<int64_t>(j) * channels, past[j]);
 }
@@ -220,11 +265,13 @@ template <typename T>
 __global__ void __launch_bounds__(CT_THREADS)
 conv_turn_kernel(const ConvTurnArgs<T> a) {
   extern __shared__ float2 turn[];
+  __shared__ int64_t places[CT_TILE];
   le::let_successor_start();
   const Stretch s = stretch_of(a);
   if (s.n <= 0) return;
   const int channels = (a.heads + 2 * a.kv_heads) * a.head_dim, keep = a.taps - 1, half = a.rot >> 1;
   make_turns(turn, a, s);
+  if (a.write_kv) find_places(places, a, s);
   le::wait_for_predecessor();
   __syncthreads();
   const int lane = threadIdx.x & 31;
@@ -266,7 +313,7 @@ conv_turn_kernel(const ConvTurnArgs<T> a) {
     T *dst = nullptr;
     const int t = s.first + s.q0 + i;
     if (is_query) dst = a.q_out + static_cast<int64_t>(t) * a.q_stride + static_cast<int64_t>(h) * a.head_dim;
-    else if (a.write_kv) dst = page_place(a, s.b, a.positions[t], h);
+    else if (a.write_kv) dst = page_place(a, places[i], h);
     if (dst == nullptr) continue;
 #pragma unroll
     for (int k = 0; k < CT_MAX_PAIRS; ++k) {
@@ -294,7 +341,7 @@ conv_turn_kernel(const ConvTurnArgs<T> a) {
 // written; k_cache / v_cache: [num_pages, kv_heads, page_size, head_dim].
 LE_API int le_conv_turn_store(const void *src, int64_t src_stride, int dtype, const float *bias, const float *taps_w, int taps,
                               float *state, int state_rows, const int32_t *state_slots, const int32_t *cu_q,
-                              const int32_t *tile_request, const int32_t *tile_q0, int num_tiles, int tile, int num_tokens,
+                              const int32_t *tile_request, const int32_t *tile_q0, int num_tiles, int tile,
                               const double *rates, int rot, float magnitude, int unit, float eps, int norm_dim, void *q_out,
                               int64_t q_stride, void *k_cache, void *v_cache, const int32_t *positions,
                               const int32_t *block_table, int max_blocks, int heads, int kv_heads, int head_dim, int page_size,
@@ -317,9 +364,10 @@ LE_API int le_conv_turn_store(const void *src, int64_t src_stride, int dtype, co
                       on16(k_cache) && on16(v_cache);
   int lph = 1;
   while (lph * piece < head_dim) lph <<= 1;
-  // many tokens: longer walks (fewer inputs fetched twice); few: more blocks
-  const int walk = tile_request == nullptr ? 4 : (pieces ? (num_tokens >= 1024 ? 8 : 4) : CT_TILE);
   const int per_block = pieces ? CT_THREADS / lph : CT_THREADS / 32;
+  // a whole tile to a block where that leaves every multiprocessor a block, else shorter stretches and more blocks
+  const bool many = static_cast<int64_t>(num_tiles) * ((all + per_block - 1) / per_block) >= 148;
+  const int walk = pieces && !many ? CT_WALK : CT_TILE;
   const dim3 grid(num_tiles * (tile_request == nullptr ? 1 : CT_TILE / walk), (all + per_block - 1) / per_block);
   if (grid.y > 65535) return le::invalid("le_conv_turn_store: %d heads are too many for one launch", all);
   const size_t smem = sizeof(float2) * (tile_request == nullptr ? 1 : walk) * (rot > 0 ? rot / 2 : 1);
@@ -333,10 +381,7 @@ LE_API int le_conv_turn_store(const void *src, int64_t src_stride, int dtype, co
     a.unit = unit, a.norm_dim = norm_dim, a.page_size = page_size, a.num_pages = num_pages, a.write_kv = write_kv;
     a.walk = walk, a.magnitude = magnitude, a.eps = eps;
     if (!pieces) return le::launch_chained(conv_turn_kernel<T>, grid, dim3(CT_THREADS), smem, stream, a);
-    auto kernel = walk == 8 ? (taps == 2 ? conv_turn_pieces_kernel<T, 2, 8> : taps == 3 ? conv_turn_pieces_kernel<T, 3, 8>
-                                                                                          : conv_turn_pieces_kernel<T, 4, 8>)
-                            : (taps == 2 ? conv_turn_pieces_kernel<T, 2, 4> : taps == 3 ? conv_turn_pieces_kernel<T, 3, 4>
-                                                                                          : conv_turn_pieces_kernel<T, 4, 4>);
+    auto kernel = taps == 2 ? conv_turn_pieces_kernel<T, 2> : taps == 3 ? conv_turn_pieces_kernel<T, 3> : conv_turn_pieces_kernel<T, 4>;
     return le::launch_chained(kernel, grid, dim3(CT_THREADS), smem, stream, a, lph);
   });
 }

@@ -97,7 +97,7 @@ _CORE_SIGNATURES = {
                              c_void_p, c_int, c_int, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_void_p, c_int64,
                              c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
     "le_conv_turn_store": [c_void_p, c_int64, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
-                           c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_float, c_int, c_float, c_int, c_void_p, c_int64,
+                           c_void_p, c_int, c_int, c_void_p, c_int, c_float, c_int, c_float, c_int, c_void_p, c_int64,
                            c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
                            c_void_p],
     "le_addend_norm": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int64, c_void_p, c_void_p, c_void_p, c_float, c_int,
@@ -1514,7 +1514,7 @@ def conv_turn_store(q_out, src, bias, w_taps, state, state_slots, cu_q, tile_req
         pages = k_cache.shape[0]
     _check(core().le_conv_turn_store(_ptr(src), src.stride(0), dtype_code(src.dtype), _ptr(bias), _ptr(w_taps), taps,
                                      _ptr(state) if taps > 1 else None, rows, _ptr(state_slots), _ptr(cu_q),
-                                     _ptr(tile_request), _ptr(tile_q0), num_tiles, SHORT_CONV_TILE, T, _ptr(rates), int(rot),
+                                     _ptr(tile_request), _ptr(tile_q0), num_tiles, SHORT_CONV_TILE, _ptr(rates), int(rot),
                                      float(magnitude), 0 if unit_eps is None else 1,
                                      0.0 if unit_eps is None else float(unit_eps), int(norm_dim), _ptr(q_out), q_out.stride(0),
                                      _ptr(k_cache) if write_kv else None, _ptr(v_cache) if write_kv else None,

@@ -37,7 +37,8 @@ def plain_addend_norm(x, y, b_in, wy, by, eps_y, centered_y, w, b, eps, centered
 
 @BOTH
 @pytest.mark.parametrize("rows,W", [(1, 64), (3, 100), (5, 33), (7, 1024), (2, 2048), (150, 2048), (9, 3072), (200, 3072), (3, 5000),
-                                    (2, 8192), (160, 8192), (2, 9000), (4, 4)])
+                                    (2, 8192), (160, 8192), (2, 9000), (4, 4),
+                                    (300, 1000), (4600, 600), (2300, 2048)])
 def test_output_norm_addition_and_next_norm(rows, W, dtype):
     """Layer norms and root mean square norms in every combination, with and
     without biases, outputs as one tensor and as 1 to 5 partial sums, for all
@@ -117,6 +118,16 @@ def test_convolution_turn_norm_and_store_under_every_cut(sizes, rot, taps, unit,
     """Four requests in cuts of unequal sizes (down to one token, shorter than
     the taps, over the kernel's tiles) on state rows that others left full;
     queries, stored keys and values equal those of the whole sequences."""
+    run_conv_turn(sizes, rot, taps, unit, dtype, [[1, 1, 2, 1, 33, 1, 31], [2, 1, 1, 1], [40, 1], [16, 2]], [2, 0, 4, 3])
+
+
+@BOTH
+@pytest.mark.parametrize("sizes,rot,taps", [((32, 8, 64, 64), 32, 4), ((24, 4, 80, 64), 64, 3)])
+def test_the_same_with_enough_tokens_for_whole_tiles_to_a_block(sizes, rot, taps, dtype):
+    run_conv_turn(sizes, rot, taps, True, dtype, [[450, 3, 467], [1, 2, 330], [18, 1, 29]], [4, 2, 0])
+
+
+def run_conv_turn(sizes, rot, taps, unit, dtype, cuts, slots_of):
     from lyapunov_engine_b200 import ops
     H, G, d, e = sizes
     hd = (max(d, e) + 15) // 16 * 16
@@ -124,26 +135,26 @@ def test_convolution_turn_norm_and_store_under_every_cut(sizes, rot, taps, unit,
     g = torch.Generator().manual_seed(H * 100 + d + taps)
     real = H * d + G * (d + e)
     w, bias = 0.6 * torch.randn(real, taps, generator=g), 0.5 * torch.randn(real, generator=g)
-    lens = (70, 5, 41, 18)
-    cuts = [[1, 1, 2, 1, 33, 1, 31], [2, 1, 1, 1], [40, 1], [16, 2]]
+    lens = [sum(c) for c in cuts]
     u = [torch.randn(n, real, generator=g).to(dtype) for n in lens]
     want = [plain_conv_turn(x.double(), bias.double(), w.double(), sizes, rot, base, eps if unit else None) for x in u]
     wide = [padded_channels(x.t().contiguous(), sizes, hd).t().contiguous() for x in u]
     C = (H + 2 * G) * hd
     w_dev = padded_channels(w, sizes, hd).t().contiguous().to(DEV)
     bias_dev = padded_channels(bias[:, None], sizes, hd).view(-1).contiguous().to(DEV)
-    slots_of = [2, 0, 4, 3]
+    R = len(cuts)
     state = torch.full((6, max(taps - 1, 1), C), 7.0, device=DEV) if taps > 1 else None
-    pages = 4 * 9 + 1
-    order = torch.randperm(pages - 1, generator=g).view(4, 9).to(torch.int32)
+    per = (max(lens) + page - 1) // page
+    pages = R * per + 1
+    order = torch.randperm(pages - 1, generator=g).view(R, per).to(torch.int32)
     kc = torch.full((pages, G, page, hd), 3.0, dtype=dtype, device=DEV)
     vc = torch.full_like(kc, 3.0)
     rates = pz.plain_rates(max(rot, 2), base).to(DEV)
     status = ops.new_status(DEV)
-    at = [0] * 4
-    got_q = [[] for _ in range(4)]
+    at = [0] * R
+    got_q = [[] for _ in range(R)]
     for step in range(max(map(len, cuts))):
-        live = [r for r in (2, 0, 3, 1) if step < len(cuts[r])]
+        live = [r for r in (2, 0, 3, 1) if r < R and step < len(cuts[r])]
         q_lens = [cuts[r][step] for r in live]
         src = torch.cat([wide[r][at[r]:at[r] + n] for r, n in zip(live, q_lens)])
         src = torch.cat([src, torch.zeros(src.shape[0], 8, dtype=dtype)], dim=1).to(DEV)     # (rows wider than the channels)
@@ -171,11 +182,11 @@ def test_convolution_turn_norm_and_store_under_every_cut(sizes, rot, taps, unit,
         q = torch.cat(got_q[r])
         torch.testing.assert_close(q[..., :d], want[r][0].float(), **tol)
         assert float(q[..., d:].abs().sum()) == 0.0
-        for t in range(n):
-            pg = int(order[r, t // page])
-            torch.testing.assert_close(kc[pg, :, t % page, :d].float().cpu(), want[r][1][t].float(), **tol)
-            torch.testing.assert_close(vc[pg, :, t % page, :e].float().cpu(), want[r][2][t].float(), **tol)
-            assert float(kc[pg, :, t % page, d:].float().abs().sum()) == 0.0 == float(vc[pg, :, t % page, e:].float().abs().sum())
+        pg = order[r, torch.arange(n) // page].long()
+        keys, values = (p[pg.to(DEV), :, (torch.arange(n) % page).to(DEV)].float().cpu() for p in (kc, vc))
+        torch.testing.assert_close(keys[..., :d], want[r][1].float(), **tol)
+        torch.testing.assert_close(values[..., :e], want[r][2].float(), **tol)
+        assert float(keys[..., d:].abs().sum()) == 0.0 == float(values[..., e:].abs().sum())
         if taps > 1:
             tail = torch.cat([torch.zeros(taps, C), wide[r].float() + bias_dev.cpu()[None]])[-(taps - 1):]
             torch.testing.assert_close(state[slots_of[r]].cpu(), tail, atol=1e-6, rtol=1e-6)
