@@ -65,24 +65,31 @@ __device__ __forceinline__ void gemm_heads_rows_block(T *__restrict__ out, int64
       }
     }
   }
+  // The 32 sums over the warp, each in the order of a butterfly over offsets 16, 8, 4, 2, 1; at each offset a lane keeps
+  // the half of them that its bit names and hands the other half over, so that lane l ends with sum l (31 exchanges
+  // instead of 160).
+  static_assert(GR_ROWS * GR_COLS == 32, "a sum per lane");
+  float v[32];
 #pragma unroll
-  for (int r = 0; r < GR_ROWS; ++r)
+  for (int i = 0; i < 32; ++i) v[i] = acc[i / GR_COLS][i % GR_COLS];
 #pragma unroll
-    for (int c = 0; c < GR_COLS; ++c) acc[r][c] = le::warp_sum(acc[r][c]);
-  if (lane < GR_COLS && n0 + lane < N) {
-    for (int r = 0; r < rows; ++r) {
-      float g = 1.0f;
-      if (gate) {
-        const int64_t i = (m0 + r) * gate_stride + (at.gate_entries ? static_cast<int64_t>(head) * N + n0 + lane : head);
-        g = 1.0f / (1.0f + expf(-le::to_f32(gate[i])));
-      }
-      float v = acc[r][0];
+  for (int o = 16; o > 0; o >>= 1) {
+    const bool upper = lane & o;
 #pragma unroll
-      for (int c = 1; c < GR_COLS; ++c) v = lane == c ? acc[r][c] : v;
-      out[(m0 + r) * out_stride + head * at.out_head + n0 + lane] = le::from_f32<T>(v * g);
+    for (int i = 0; i < o; ++i) {
+      const float keep = upper ? v[i + o] : v[i], give = upper ? v[i] : v[i + o];
+      v[i] = keep + __shfl_xor_sync(0xffffffffu, give, o);
     }
   }
+  const int r = lane / GR_COLS, n = n0 + lane % GR_COLS;
+  if (r < rows && n < N) {
+    float g = 1.0f;
+    if (gate) {
+      const int64_t i = (m0 + r) * gate_stride + (at.gate_entries ? static_cast<int64_t>(head) * N + n : head);
+      g = 1.0f / (1.0f + expf(-le::to_f32(gate[i])));
+    }
+    out[(m0 + r) * out_stride + head * at.out_head + n] = le::from_f32<T>(v[0] * g);
+  }
 }
-
 
 }  // namespace le_heads
