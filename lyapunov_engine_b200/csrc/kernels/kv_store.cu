@@ -75,7 +75,11 @@ latent_prepare_kernel(const le_latent::Args<T> a, int num_tokens, int head_dim, 
   if (waits) le::wait_for_predecessor();
   if (part == 0 && a.cache == nullptr) return;
   bool waited = waits;
-  for (int t = blockIdx.z * gridDim.x + blockIdx.x; t < num_tokens; t += gridDim.x * gridDim.z) {
+  // a token to a block, or, of the queries' turns, to as many blocks as there are for it
+  const int blocks = gridDim.x * gridDim.z, mine = blockIdx.z * gridDim.x + blockIdx.x;
+  const int per = part == 0 ? 1 : max(1, blocks / num_tokens);
+  if (mine >= blocks / per * per) return;
+  for (int t = mine / per; t < num_tokens; t += blocks / per) {
     if (a.rot > 0) {
       __syncthreads();             // (the last token's turns are done with)
       le_latent::make_turns(turn, a, t);
@@ -84,7 +88,7 @@ latent_prepare_kernel(const le_latent::Args<T> a, int num_tokens, int head_dim, 
       __syncthreads();
     }
     if (part == 0) le_latent::store_latent(a, t, turn, scratch);
-    else le_latent::turn_queries(a, t, turn);
+    else le_latent::turn_queries(a, t, turn, mine % per, per);
   }
 }
 

@@ -70,13 +70,14 @@ __device__ __forceinline__ void store_latent(const Args<T> &a, int t, const floa
   }
 }
 
-// The whole block; `turn` is made.
+// The whole block, block `mine` of `blocks` that share the token's work; `turn` is made.
 template <typename T>
-__device__ __forceinline__ void turn_queries(const Args<T> &a, int t, const float2 *turn) {
+__device__ __forceinline__ void turn_queries(const Args<T> &a, int t, const float2 *turn, int mine = 0, int blocks = 1) {
   const T *row = a.src + static_cast<int64_t>(t) * a.src_stride + a.q_col;
   T *out = a.q_out + static_cast<int64_t>(t) * a.q_stride + a.rank;
   const int half = a.rot >> 1, tail = a.padded - a.rank - a.rot;
-  for (int i = threadIdx.x; i < a.heads * half; i += blockDim.x) {
+  const int first = mine * blockDim.x + threadIdx.x, step = blocks * blockDim.x;
+  for (int i = first; i < a.heads * half; i += step) {
     const int h = i / half, j = i - h * half;
     const T *p = row + static_cast<int64_t>(h) * a.q_head + 2 * j;
     T *o = out + static_cast<int64_t>(h) * a.padded + 2 * j;
@@ -97,7 +98,7 @@ __device__ __forceinline__ void turn_queries(const Args<T> &a, int t, const floa
       o[0] = le::from_f32<T>(u), o[1] = le::from_f32<T>(v);
     }
   }
-  for (int i = threadIdx.x; i < a.heads * tail; i += blockDim.x)
+  for (int i = first; i < a.heads * tail; i += step)
     out[static_cast<int64_t>(i / tail) * a.padded + a.rot + i % tail] = le::from_f32<T>(0.0f);
 }
 

@@ -17,7 +17,10 @@ Interfaces (all tensors are CUDA tensors; T tokens in the step, H width):
 ``PositionEncoding``
     ``encode_and_store(qkv, geometry, ctx, kv, write)``: encodes the queries
     (in place) and keys of the fused projection rows and, if ``write``, stores
-    keys and values in the paged cache ``kv``.
+    keys and values in the paged cache ``kv``.  One that cannot work in place
+    (a convolution over time reads earlier rows) offers ``encode_rows(qkv,
+    geometry, ctx, cache) -> queries`` instead, with ``extra_state_needs()``
+    and ``tile_sizes()`` as a mixer has them.
 ``Mixer``
     ``cache_need() -> KVNeed | None`` and ``state_need() -> StateNeed | None``
     say what the cache manager must hold for it; ``forward(x, ctx, cache) ->
